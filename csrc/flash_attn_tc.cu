@@ -21,6 +21,7 @@
 #include "gemm_tcgen05.cuh"
 #include "attn_tc_common.cuh"
 #include "ptx.cuh"
+#include "score_mod.cuh"
 
 #include <type_traits>
 
@@ -42,6 +43,9 @@ struct TcParams {
     // WIN instantiation only: sliding window with kept first keys and a linear distance bias (causal)
     int window, keep_first;      // window <= 0: no window
     const float* slopes;         // [Hq] or NULL; the bias is -slope * (query position - key position)
+    const float* sinks;          // [Hq] or NULL: exp(sink) joins the softmax denominator
+    ScoreMod mod;                // output gate; SCORE instantiations: soft cap, logarithmic bias, sigmoid weights
+    int bias_entries;            // SCORE: distances in the shared-memory bias table; 0: no bias, -1: evaluated per score
 };
 
 template <int D>
@@ -62,7 +66,11 @@ struct TcSmem {
 // (`tile(j)` maps the j-th visited tile to its index; every role derives it from the same two numbers), the masked path
 // also hides keys below the window that are not kept, and scores get the scale and the distance bias before the running
 // max (which is then kept in log2 units).  The barrier protocol and the MMA issue are the same for both instantiations.
-template <int D, bool CAUSAL, bool DROP, bool WIN = false>
+// SCORE (with WIN): 1 = soft cap and / or logarithmic distance bias ahead of the softmax, 2 = sigmoid weights (no running max,
+// no denominator).  The distance bias of a head is a table over the distances in shared memory, filled once per CTA (lanes are
+// query rows, so a warp reads 32 consecutive entries); the soft cap takes the tanh series unless a score of the warp's tile
+// is too large for it.
+template <int D, bool CAUSAL, bool DROP, bool WIN = false, int SCORE = 0>
 __global__ void __launch_bounds__(kThreadsTc, 2)
 fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_constant__ CUtensorMap tmap_k,
                  const __grid_constant__ CUtensorMap tmap_v, const __grid_constant__ CUtensorMap tmap_o,
@@ -118,6 +126,15 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         ptx::fence_barrier_init();
     }
     if (warp == 1) ptx::tmem_alloc<1>(tmem_ptr_smem, L::kTmemCols);
+    float* dtab = reinterpret_cast<float*>(sP);          // bias table (SCORE): the P staging area is free, P lives in TMEM
+    constexpr float kL2e = score::kLog2e;
+    const float r1 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r1[hq] * kL2e : 0.f;
+    const float r2 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r2[hq] : 0.f;
+    if (SCORE > 0 && p.bias_entries > 0) {
+        const float sl = p.slopes != nullptr ? p.slopes[hq] * kL2e : 0.f;
+        const int n = min(p.bias_entries, m0 + kBM + offset);
+        for (int i = threadIdx.x; i < n; i += kThreadsTc) dtab[i] = r1 * __log2f(fmaf(r2, (float)i, 1.f)) + sl * (float)i;
+    }
     ptx::tcgen05_fence_before();
     __syncthreads();
     ptx::tcgen05_fence_after();
@@ -212,6 +229,9 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         // FFMA per element: s * scale_log2 - m * scale_log2.
         float m_run = -INFINITY, l_run = 0.f;
         const float sc = WIN ? 1.f : p.scale_log2;                   // WIN: scores are converted to log2 units up front
+        const float cap_in = (SCORE > 0 && p.mod.cap > 0.f) ? p.scale_log2 / (kL2e * p.mod.cap) : 0.f;
+        const float cap_out = p.mod.cap * kL2e;
+        const float pb2 = SCORE == 2 ? p.mod.pb[hq] * kL2e : 0.f;
         const float slope2 = (WIN && p.slopes != nullptr) ? p.slopes[hq] * 1.4426950408889634f : 0.f;
         // one tile of the online softmax; MASK is instantiated only for tiles on the causal diagonal / past Sk
         auto tile_softmax = [&](auto mask_tag, int j) {
@@ -223,7 +243,46 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
             ptx::tcgen05_fence_before();
             ptx::mbar_arrive(s_empty);
             const int n0 = tile(j) * kBN;
-            if (WIN) {
+            if (SCORE > 0) {
+                if (cap_in > 0.f) {
+                    float am0 = 0.f, am1 = 0.f;
+#pragma unroll
+                    for (int c = 0; c < kBN; c += 2) {
+                        am0 = fmaxf(am0, fabsf(__uint_as_float(sr[c])));
+                        am1 = fmaxf(am1, fabsf(__uint_as_float(sr[c + 1])));
+                    }
+                    if (__any_sync(0xffffffffu, fmaxf(am0, am1) * cap_in >= score::kSeriesLimit)) {
+#pragma unroll
+                        for (int c = 0; c < kBN; ++c)
+                            sr[c] = __float_as_uint(cap_out * score::tanh_exp(__uint_as_float(sr[c]) * cap_in));
+                    } else {
+#pragma unroll
+                        for (int c = 0; c < kBN; ++c)
+                            sr[c] = __float_as_uint(cap_out * score::tanh_series(__uint_as_float(sr[c]) * cap_in));
+                    }
+                } else {
+#pragma unroll
+                    for (int c = 0; c < kBN; ++c) sr[c] = __float_as_uint(__uint_as_float(sr[c]) * p.scale_log2);
+                }
+                const int d0 = grow + offset - n0;                          // distance of column 0
+                if (p.bias_entries > 0) {
+                    if (MASK) {
+#pragma unroll
+                        for (int c = 0; c < kBN; ++c)
+                            sr[c] = __float_as_uint(__uint_as_float(sr[c]) - dtab[min(max(d0 - c, 0), p.bias_entries - 1)]);
+                    } else {
+                        const float* tb = dtab + d0;
+#pragma unroll
+                        for (int c = 0; c < kBN; ++c) sr[c] = __float_as_uint(__uint_as_float(sr[c]) - tb[-c]);
+                    }
+                } else if (p.bias_entries < 0) {
+#pragma unroll
+                    for (int c = 0; c < kBN; ++c) {
+                        const float dist = (float)max(d0 - c, 0);
+                        sr[c] = __float_as_uint(__uint_as_float(sr[c]) - r1 * __log2f(fmaf(r2, dist, 1.f)) - slope2 * dist);
+                    }
+                }
+            } else if (WIN) {
                 // log2 units: s * scale - slope * (query position - key position)
                 const float base = -slope2 * (float)(grow + offset - n0);
 #pragma unroll
@@ -241,6 +300,27 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
                 for (int c = 0; c < kBN; ++c)
                     if (c >= first_bad || (WIN && c < first_good && c >= kept)) sr[c] = 0xff800000u;   // -inf
             }
+            uint32_t pk[kBN / 2];
+            if constexpr (SCORE == 2) {
+                // sigmoid(x) = 1 / (1 + 2^-x2); one reciprocal serves two weights (the clamp keeps the product finite)
+#pragma unroll
+                for (int c = 0; c < kBN; c += 2) {
+                    const float x0 = __uint_as_float(sr[c]) + pb2, x1 = __uint_as_float(sr[c + 1]) + pb2;
+                    const float a = 1.f + ex2_approx(fminf(-x0, 60.f)), bq = 1.f + ex2_approx(fminf(-x1, 60.f));
+                    const float r = __fdividef(1.f, a * bq);
+                    float p0 = r * bq, p1 = r * a;
+                    if (MASK) {
+                        if (x0 == -INFINITY) p0 = 0.f;
+                        if (x1 == -INFINITY) p1 = 0.f;
+                    }
+                    pk[c >> 1] = pack_bf16x2(p0, p1);
+                }
+                l_run = 1.f;
+                if (j > 0) {
+                    ptx::mbar_wait(pv_done, ((uint32_t)(j - 1)) & 1u);  // P buffer free
+                    ptx::tcgen05_fence_after();
+                }
+            } else {
             float mx0 = __uint_as_float(sr[0]), mx1 = __uint_as_float(sr[1]), mx2 = __uint_as_float(sr[2]),
                   mx3 = __uint_as_float(sr[3]);
 #pragma unroll
@@ -264,7 +344,6 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
             }
             const float neg_m = (m_run == -INFINITY) ? 0.f : -m_run * sc;
             float rs0 = 0.f, rs1 = 0.f;
-            uint32_t pk[kBN / 2];
 #pragma unroll
             for (int c = 0; c < kBN; c += 2) {
                 const float p0 = ex2_approx(fmaf(__uint_as_float(sr[c]), sc, neg_m));
@@ -298,6 +377,7 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
                     tmem_st_wait();
                 }
             }
+            }
             // P goes to TENSOR MEMORY (this thread's row, 64 keys = 32 packed words): the A operand of the P V MMA never
             // touches shared memory (no 16 KB store + re-read per tile, no async-proxy fence)
             tmem_st_32x32b_x16(tmem_p + lane_off, pk);
@@ -323,7 +403,9 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
             ptx::mbar_wait(pv_done, ((uint32_t)(n_tiles - 1)) & 1u);
             ptx::tcgen05_fence_after();
         }
-        const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+        if (WIN && SCORE != 2 && p.sinks != nullptr && m_run != -INFINITY) l_run += ex2_approx(p.sinks[hq] * kL2e - m_run);
+        float inv = l_run > 0.f ? 1.f / l_run : 0.f;
+        if (WIN && grow < p.Sq) inv *= score::out_gate<bf16>(p.mod, (long long)b * p.Sq + grow, hq);
         if (p.lse && grow < p.Sq)
             p.lse[((long long)b * p.Hq + hq) * p.Sq + grow] = l_run > 0.f ? m_run * sc + log2f(l_run) : INFINITY;
         // every MMA that read Q has completed: reuse the Q tile as staging (warp q owns rows [32q, 32q+32) of
@@ -391,15 +473,15 @@ int launch_fwd_tc(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMa
                 : launch_fwd_tc_one<D, false, false>(tq, tk, tv, to, p, st);
 }
 
-template <int D>
+template <int D, int SCORE>
 int launch_fwd_tc_win(const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, const CUtensorMap& to,
                       const TcParams& p, cudaStream_t st) {
     using L = TcSmem<D>;
     dim3 grid(p.Hq, p.B, (p.Sq + kBM - 1) / kBM);
-    static cudaError_t once = cudaFuncSetAttribute(fa_fwd_tc_kernel<D, true, false, true>,
+    static cudaError_t once = cudaFuncSetAttribute(fa_fwd_tc_kernel<D, true, false, true, SCORE>,
                                                    cudaFuncAttributeMaxDynamicSharedMemorySize, L::kBytes);
     NXD_CHECK_CUDA(once);
-    fa_fwd_tc_kernel<D, true, false, true><<<grid, kThreadsTc, L::kBytes, st>>>(tq, tk, tv, to, p);
+    fa_fwd_tc_kernel<D, true, false, true, SCORE><<<grid, kThreadsTc, L::kBytes, st>>>(tq, tk, tv, to, p);
     NXD_LAUNCH_CHECK();
     return 0;
 }
@@ -452,9 +534,14 @@ NXD_API int nxd_flash_attn_fwd_tc_dropout(const void* q, const void* k, const vo
 
 // Causal attention with a sliding window (window <= 0: none), `keep_first` first keys that stay visible, and a linear
 // distance bias -slopes[h] * (i - j) (slopes NULL: none); tensors and strides as nxd_flash_attn_fwd_tc, no lse output.
-NXD_API int nxd_flash_attn_fwd_tc_window(const void* q, const void* k, const void* v, void* o, const long long* strides,
+// sinks [Hq] or NULL; softcap, log_r1 / log_r2, sigmoid_bias, gate as in nxd_scored_attn_prefill (score_mod.cuh).
+NXD_API int nxd_flash_attn_fwd_tc_scored(const void* q, const void* k, const void* v, void* o, const long long* strides,
                                          int B, int Hq, int Hkv, int Sq, int Sk, int D, float scale, int window,
-                                         int keep_first, const float* slopes, void* stream) {
+                                         int keep_first, const float* slopes, const float* sinks, float softcap,
+                                         const float* log_r1, const float* log_r2, const float* sigmoid_bias,
+                                         const void* gate, long long gate_ld, void* stream) {
+    NXD_REQUIRE((log_r1 == nullptr) == (log_r2 == nullptr), "flash_attn_tc: the logarithmic bias needs %s", "both vectors");
+    NXD_REQUIRE(sigmoid_bias == nullptr || sinks == nullptr, "flash_attn_tc: sigmoid weights have no %s", "sink");
     NXD_REQUIRE(D == 64 || D == 128, "flash_attn_tc_window: head dim %d not supported (64 or 128)", D);
     NXD_REQUIRE(B > 0 && Hq > 0 && Hkv > 0 && Sq > 0 && Sk >= Sq && Hq % Hkv == 0, "flash_attn_tc_window: bad problem");
     for (int i = 0; i < 12; ++i)
@@ -471,12 +558,28 @@ NXD_API int nxd_flash_attn_fwd_tc_window(const void* q, const void* k, const voi
     p.window = window;
     p.keep_first = keep_first > 0 ? keep_first : 0;
     p.slopes = slopes;
+    p.sinks = sinks;
+    p.mod = ScoreMod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld};
+    const int mode = p.mod.mode();
+    if (mode > 0 && (log_r1 != nullptr || slopes != nullptr)) {
+        const int span = (window > 0 && window < Sk && p.keep_first == 0) ? window : Sk;      // distances that can be visible
+        p.bias_entries = span <= TcSmem<64>::kPBytes / 4 ? span : -1;
+    }
     CUtensorMap tq, tk, tv, to;
     int rc;
     if ((rc = make_tmap_bhsd(&tq, q, D, Sq, Hq, B, strides[2], strides[1], strides[0], kBM, p.pos_q))) return rc;
     if ((rc = make_tmap_bhsd(&tk, k, D, Sk, Hkv, B, strides[5], strides[4], strides[3], kBN, p.pos_k))) return rc;
     if ((rc = make_tmap_bhsd(&tv, v, D, Sk, Hkv, B, strides[8], strides[7], strides[6], kBN, p.pos_v))) return rc;
     if ((rc = make_tmap_bhsd(&to, o, D, Sq, Hq, B, strides[11], strides[10], strides[9], 32, p.pos_o))) return rc;
-    return D == 64 ? launch_fwd_tc_win<64>(tq, tk, tv, to, p, (cudaStream_t)stream)
-                   : launch_fwd_tc_win<128>(tq, tk, tv, to, p, (cudaStream_t)stream);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (mode == 2) return D == 64 ? launch_fwd_tc_win<64, 2>(tq, tk, tv, to, p, st) : launch_fwd_tc_win<128, 2>(tq, tk, tv, to, p, st);
+    if (mode == 1) return D == 64 ? launch_fwd_tc_win<64, 1>(tq, tk, tv, to, p, st) : launch_fwd_tc_win<128, 1>(tq, tk, tv, to, p, st);
+    return D == 64 ? launch_fwd_tc_win<64, 0>(tq, tk, tv, to, p, st) : launch_fwd_tc_win<128, 0>(tq, tk, tv, to, p, st);
+}
+
+NXD_API int nxd_flash_attn_fwd_tc_window(const void* q, const void* k, const void* v, void* o, const long long* strides,
+                                         int B, int Hq, int Hkv, int Sq, int Sk, int D, float scale, int window,
+                                         int keep_first, const float* slopes, void* stream) {
+    return nxd_flash_attn_fwd_tc_scored(q, k, v, o, strides, B, Hq, Hkv, Sq, Sk, D, scale, window, keep_first, slopes, nullptr,
+                                        0.f, nullptr, nullptr, nullptr, nullptr, 0, stream);
 }

@@ -1,0 +1,53 @@
+// What an attention kernel may do to a score after the scaled product, next to the mask and the linear distance bias, and to
+// the head output after the value product:
+//
+//   soft cap         s <- cap * tanh(s / cap)                                        (cap > 0)
+//   log distance     s <- s - r1_h * ln(1 + r2_h * (i - j))                          (r1, r2 != NULL)
+//   sigmoid weights  weight = sigmoid(s + pb_h), not normalised over the keys        (pb != NULL; no softmax, no sink)
+//   output gate      o <- o * sigmoid(gate[row, h])                                  (gate != NULL; one number per head)
+//
+// tanh in fp32 for |x| < 0.4 is the odd power series up to x^9 (next term below 1e-6 of the value), beyond that
+// 1 - 2 / (1 + exp(2 |x|)); the kernels choose once per tile where they can.
+#pragma once
+#include "common.cuh"
+
+struct ScoreMod {
+    float cap;
+    const float* r1;
+    const float* r2;
+    const float* pb;
+    const void* gate;        // activation dtype; pre-activation of (row n, head h) at gate[n * gate_ld + h]
+    long long gate_ld;
+    __host__ __device__ int mode() const { return pb != nullptr ? 2 : ((cap > 0.f || r1 != nullptr) ? 1 : 0); }
+};
+
+namespace score {
+
+constexpr float kSeriesLimit = 0.4f;
+constexpr float kLog2e = 1.4426950408889634f;
+
+__device__ __forceinline__ float tanh_series(float x) {
+    const float z = x * x;
+    float p = fmaf(z, 62.f / 2835.f, -17.f / 315.f);
+    p = fmaf(z, p, 2.f / 15.f);
+    p = fmaf(z, p, -1.f / 3.f);
+    return fmaf(x * z, p, x);
+}
+__device__ __forceinline__ float tanh_exp(float x) {
+    const float e = exp2f(2.f * kLog2e * fabsf(x));
+    return copysignf(1.f - __fdividef(2.f, 1.f + fminf(e, 1e30f)), x);
+}
+__device__ __forceinline__ float tanh_any(float x) { return fabsf(x) < kSeriesLimit ? tanh_series(x) : tanh_exp(x); }
+
+// sigmoid(x) for x given in log2 units (x * log2 e); the clamp keeps 1 + 2^-x finite
+__device__ __forceinline__ float sigmoid_log2(float x2) { return __fdividef(1.f, 1.f + exp2f(fminf(-x2, 100.f))); }
+__device__ __forceinline__ float sigmoid(float x) { return sigmoid_log2(x * kLog2e); }
+
+__device__ __forceinline__ float ldg(const float* p) { return *p; }
+__device__ __forceinline__ float ldg(const bf16* p) { return __bfloat162float(*p); }
+template <typename T>
+__device__ __forceinline__ float out_gate(const ScoreMod& m, long long row, int h) {
+    return m.gate == nullptr ? 1.f : sigmoid(ldg(reinterpret_cast<const T*>(m.gate) + row * m.gate_ld + h));
+}
+
+}  // namespace score

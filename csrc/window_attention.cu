@@ -6,6 +6,8 @@
 //   score(i, j)   = scale * <q_i, k_j> - slope_h * (i - j)            (slopes == NULL: no bias)
 //   softmax denominator = sum over visible j of exp(score) (+ exp(sink_h) with sinks != NULL: a learned per-head
 //                   logit attached to no position that only takes probability mass)
+// After the scaled product a score may be soft-capped and lose a logarithmic distance bias, the weights may be sigmoids
+// instead of a softmax, and the head output may be gated (score_mod.cuh).
 // Chunk boundaries sit at absolute multiples of the chunk size.  The value rows may be a column range of the key rows (one
 // cache tensor, value row pitch = key row pitch): the latent cache of a compressed key/value projection.
 //
@@ -22,6 +24,7 @@
 // The cache is contiguous [lines, G, S, D] or paged [pages, G, page, D] with a block table [lines, cols].
 #include "common.cuh"
 #include "mma_sync.cuh"
+#include "score_mod.cuh"
 
 namespace {
 
@@ -49,18 +52,18 @@ __device__ __forceinline__ void stf(bf16* p, float v) { *p = __float2bfloat16_rn
 // 1 / rms over all query heads (stat[2n]) and over all key heads (stat[2n + 1]) of projection row n: one warp per row
 template <typename T>
 __global__ void qk_row_stat_kernel(const T* __restrict__ qkv, long long ld, float* __restrict__ stat, long long rows, int nq,
-                                   int nk, float eps) {
+                                   int nk, float eps, const float* __restrict__ bias) {
     const int lane = threadIdx.x & 31;
     const long long n = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (n >= rows) return;
     const T* row = qkv + n * ld;
     float sq = 0.f, sk = 0.f;
     for (int i = lane; i < nq; i += 32) {
-        const float v = ldf(row + i);
+        const float v = ldf(row + i) + (bias != nullptr ? bias[i] : 0.f);
         sq += v * v;
     }
     for (int i = lane; i < nk; i += 32) {
-        const float v = ldf(row + nq + i);
+        const float v = ldf(row + nq + i) + (bias != nullptr ? bias[nq + i] : 0.f);
         sk += v * v;
     }
     sq = warp_sum(sq);
@@ -80,7 +83,8 @@ __global__ void qk_norm_cache_write_kernel(const T* __restrict__ qkv, long long 
                                            const float* __restrict__ q_weight, const float* __restrict__ k_weight,
                                            const float* __restrict__ rope_cos, const float* __restrict__ rope_sin,
                                            int rope_dims, int value_from_key, int Gv, int rope_halves,
-                                           int whole_norm, const float* __restrict__ row_stat) {
+                                           int whole_norm, const float* __restrict__ row_stat,
+                                           const float* __restrict__ bias, int value_norm) {
     const int lane = threadIdx.x & 31;
     const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (unit >= units) return;
@@ -103,6 +107,8 @@ __global__ void qk_norm_cache_write_kernel(const T* __restrict__ qkv, long long 
         src = qkv + n * ld + (long long)(H + G) * D + (long long)(hd - H - G) * Dv;
         dim = Dv;
     }
+    // bias [columns of the row] fp32 or NULL: added to the projection ahead of everything else
+    const float* bsrc = bias != nullptr ? bias + (src - (qkv + n * ld)) : nullptr;
     T* dst;
     if (hd < H) {
         dst = q_out + (n * H + hd) * D;
@@ -121,17 +127,26 @@ __global__ void qk_norm_cache_write_kernel(const T* __restrict__ qkv, long long 
         // weight has that size; else over the head alone, with a weight of D values shared by the heads
         const T* stat = whole_norm ? (hd < H ? qkv + n * ld : qkv + n * ld + (long long)H * D) : src;
         const int cnt = whole_norm ? (hd < H ? H : G) * D : dim;
+        const float* bstat = bias != nullptr ? bias + (stat - (qkv + n * ld)) : nullptr;
         float ss = 0.f;
         for (int i = lane; i < cnt; i += 32) {
-            const float v = ldf(stat + i);
+            const float v = ldf(stat + i) + (bstat != nullptr ? bstat[i] : 0.f);
             ss += v * v;
         }
         ss = warp_sum(ss);
         r = 1.f / sqrtf(ss / (float)cnt + eps);
+    } else if (hd >= H + G && value_norm) {      // unit-RMS values, every head on its own, no weight
+        float ss = 0.f;
+        for (int i = lane; i < dim; i += 32) {
+            const float v = ldf(src + i) + (bsrc != nullptr ? bsrc[i] : 0.f);
+            ss += v * v;
+        }
+        r = 1.f / sqrtf(warp_sum(ss) / (float)dim + eps);
     }
-    // writeback: the normalised keys also replace the raw ones in the projection buffer, so that a kernel that reads
-    // q / k / v as strided views of that buffer (prefill from position 0) sees what the cache holds
-    T* back = (writeback && hd >= H && hd < H + G) ? const_cast<T*>(src) : nullptr;
+    // writeback: the keys (and, where a bias or a norm changes them, the values) as cached also replace the raw ones in
+    // the projection buffer, so that a kernel that reads q / k / v as strided views of that buffer (prefill from position
+    // 0) sees what the cache holds
+    T* back = (writeback && hd >= H && (hd < H + G || bias != nullptr || value_norm)) ? const_cast<T*>(src) : nullptr;
     const float* wgt = hd < H ? q_weight : (hd < H + G ? k_weight : nullptr);
     if (wgt != nullptr && whole_norm) wgt += (long long)(hd < H ? hd : hd - H) * D;
     const int rot = (hd < H + G && rope_cos != nullptr) ? rope_dims : 0;
@@ -143,7 +158,8 @@ __global__ void qk_norm_cache_write_kernel(const T* __restrict__ qkv, long long 
         const float* sn = rope_sin + pos * (rope_dims / 2);
         for (int i = lane; i < rot / 2; i += 32) {
             const int iu = rope_halves ? i : 2 * i, iv = rope_halves ? i + rot / 2 : 2 * i + 1;
-            float u = ldf(src + iu) * r, v = ldf(src + iv) * r;
+            float u = (ldf(src + iu) + (bsrc != nullptr ? bsrc[iu] : 0.f)) * r;
+            float v = (ldf(src + iv) + (bsrc != nullptr ? bsrc[iv] : 0.f)) * r;
             if (wgt != nullptr) {
                 u *= wgt[iu];
                 v *= wgt[iv];
@@ -154,7 +170,7 @@ __global__ void qk_norm_cache_write_kernel(const T* __restrict__ qkv, long long 
         }
     }
     for (int i = rot + lane; i < dim; i += 32) {
-        float v = ldf(src + i) * r;
+        float v = (ldf(src + i) + (bsrc != nullptr ? bsrc[i] : 0.f)) * r;
         if (wgt != nullptr) v *= wgt[i];
         stf(dst + i, v);
         if (back != nullptr) stf(back + i, v);
@@ -170,7 +186,7 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
                            CacheAddr ka, CacheAddr va, T* __restrict__ out, const int* __restrict__ q_start,
                            const int* __restrict__ n_new, const int* __restrict__ seq_ids,
                            const float* __restrict__ slopes, int Tn, int H, int G, int D, int Dv, float scale, int window,
-                           int keep_first, int chunk, const float* __restrict__ sinks) {
+                           int keep_first, int chunk, const float* __restrict__ sinks, const ScoreMod mod) {
     extern __shared__ float smem[];
     float* Qs = smem;                       // [BQ][D]
     float* Ks = Qs + BQ * D;                // [BK][D + 1]
@@ -198,6 +214,9 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
     const int p_lo = start + q0;
     const int p_hi = start + min(q0 + BQ, nb) - 1;
     const float slope = slopes != nullptr ? slopes[h] : 0.f;
+    const float r1 = mod.r1 != nullptr ? mod.r1[h] : 0.f, r2 = mod.r1 != nullptr ? mod.r2[h] : 0.f;
+    const bool sig = mod.pb != nullptr;
+    const float pb = sig ? mod.pb[h] : 0.f;
 
     for (int idx = tid; idx < BQ * D; idx += PF_THREADS) {
         const int r = idx / D, c = idx - r * D;
@@ -244,17 +263,19 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
             const int dist = p_i - j;
             const bool vis = row_ok && dist >= 0 && (window <= 0 || dist < window || j < keep_first) &&
                              (chunk <= 0 || p_i / chunk == j / chunk);
+            if (mod.cap > 0.f) d = mod.cap * score::tanh_any(d / mod.cap);
+            if (r1 != 0.f) d -= r1 * logf(1.f + r2 * (float)max(dist, 0));
             s[m] = vis ? d - slope * (float)dist : -INFINITY;
             tmax = fmaxf(tmax, s[m]);
         }
 #pragma unroll
         for (int o = 1; o < 8; o <<= 1) tmax = fmaxf(tmax, __shfl_xor_sync(0xffffffffu, tmax, o));
-        const float m_new = fmaxf(m_i, tmax);
-        const float alpha = (m_new == -INFINITY) ? 1.f : expf(m_i - m_new);
+        const float m_new = sig ? 0.f : fmaxf(m_i, tmax);           // sigmoid weights need no running maximum
+        const float alpha = (m_new == -INFINITY || sig) ? 1.f : expf(m_i - m_new);
         float tsum = 0.f;
 #pragma unroll
         for (int m = 0; m < 4; ++m) {
-            const float p = (s[m] == -INFINITY) ? 0.f : expf(s[m] - m_new);
+            const float p = (s[m] == -INFINITY) ? 0.f : (sig ? score::sigmoid(s[m] + pb) : expf(s[m] - m_new));
             Ps[qi * BK + sub + 8 * m] = p;
             tsum += p;
         }
@@ -278,7 +299,8 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
     }
     if (sinks != nullptr) l_i += expf(sinks[h] - (m_i == -INFINITY ? 0.f : m_i));
     if (q0 + qi < Tn) {
-        const float inv = (row_ok && l_i > 0.f) ? 1.f / l_i : 0.f;
+        float inv = (row_ok && l_i > 0.f) ? (sig ? 1.f : 1.f / l_i) : 0.f;
+        if (row_ok) inv *= score::out_gate<T>(mod, (long long)b * Tn + q0 + qi, h);
 #pragma unroll
         for (int m = 0; m < MAXC; ++m) {
             if (m < nc) {
@@ -297,19 +319,23 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
 // tiles visited are the ones that hold kept first tokens plus the ones the window of some query of the tile reaches.
 constexpr int MQ = 64, MK = 64, M_THREADS = 128;
 
-template <int D, int DV>
+// MODE: 0 = softmax of the (linearly biased) scores, 1 = soft cap and / or logarithmic bias ahead of the softmax, 2 = sigmoid
+// weights.  The distance biases of modes 1 and 2 come from a table of the tile's 127 distances in shared memory.
+template <int D, int DV, int MODE>
 __global__ void __launch_bounds__(M_THREADS)
 window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache_k,
                                const bf16* __restrict__ cache_v, CacheAddr ka, CacheAddr va, bf16* __restrict__ out,
                                const int* __restrict__ q_start, const int* __restrict__ n_new,
                                const int* __restrict__ seq_ids, const float* __restrict__ slopes, int Tn, int H, int G,
-                               float scale, int window, int keep_first, int chunk, const float* __restrict__ sinks) {
+                               float scale, int window, int keep_first, int chunk, const float* __restrict__ sinks,
+                               const ScoreMod mod) {
     constexpr int LDK = D + 8, LDV = DV + 8, CK = D / 8, CV = DV / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);       // [MQ][LDK]
     bf16* Ks = Qs + MQ * LDK;                           // [2][MK][LDK]
     bf16* Vs = Ks + 2 * MK * LDK;                       // [2][MK][LDV]
     __shared__ long long koff[2][MK], voff[2][MK];
+    __shared__ float dbias[MODE > 0 ? MQ + MK : 1];
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int q0 = blockIdx.x * MQ, h = blockIdx.y, b = blockIdx.z;
@@ -381,6 +407,11 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     uint32_t qf[D / 16][4];
+    const bool biased = MODE > 0 && (mod.r1 != nullptr || slopes != nullptr);
+    const float r1 = (MODE > 0 && mod.r1 != nullptr) ? mod.r1[h] * LOG2E : 0.f;
+    const float r2 = (MODE > 0 && mod.r1 != nullptr) ? mod.r2[h] : 0.f;
+    const float pb2 = MODE == 2 ? mod.pb[h] * LOG2E : 0.f;
+    const float cap_in = (MODE > 0 && mod.cap > 0.f) ? scale / mod.cap : 0.f, cap_out = mod.cap * LOG2E;
 
     for (int n = 0; n < n_tiles; ++n) {
         const int buf = n & 1;
@@ -389,6 +420,11 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
             mma::cp_async_wait<1>();
         } else {
             mma::cp_async_wait<0>();
+        }
+        if (MODE > 0 && biased) {                         // distance of entry e: (first query - last key of the tile) + e
+            const int kt_b = n < n_sink_tiles ? n : t_win + (n - n_sink_tiles);
+            const float dist = (float)max(p_lo - kt_b * MK - (MK - 1) + tid, 0);
+            dbias[tid] = r1 * __log2f(fmaf(r2, dist, 1.f)) + sl2 * dist;
         }
         __syncthreads();
         if (n == 0) {
@@ -418,7 +454,57 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
         const bool full = q0 + MQ <= nb && k0 + MK - 1 <= p_lo &&
                           (window <= 0 || p_hi - k0 < window || k0 + MK <= keep_first) &&
                           (chunk <= 0 || k0 / chunk == p_hi / chunk);
-        if (full) {
+        if (MODE > 0) {
+            if (cap_in > 0.f) {
+                float am = 0.f;
+#pragma unroll
+                for (int i = 0; i < MK / 8; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) am = fmaxf(am, fabsf(s[i][e]));
+                if (__any_sync(0xffffffffu, am * cap_in >= score::kSeriesLimit)) {
+#pragma unroll
+                    for (int i = 0; i < MK / 8; ++i)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) s[i][e] = cap_out * score::tanh_exp(s[i][e] * cap_in);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < MK / 8; ++i)
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) s[i][e] = cap_out * score::tanh_series(s[i][e] * cap_in);
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < MK / 8; ++i)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[i][e] *= sc2;
+            }
+            if (biased) {
+                const float* tb = dbias + r_lo + (MK - 1) - (lane & 3) * 2;      // entry of (row r_lo, column (lane & 3) * 2)
+#pragma unroll
+                for (int i = 0; i < MK / 8; ++i) {
+                    s[i][0] -= tb[-8 * i];
+                    s[i][1] -= tb[-8 * i - 1];
+                    s[i][2] -= tb[8 - 8 * i];
+                    s[i][3] -= tb[8 - 8 * i - 1];
+                }
+            }
+#pragma unroll
+            for (int i = 0; i < MK / 8; ++i) {
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    if (!full) {
+                        const int j = k0 + i * 8 + (lane & 3) * 2 + (e & 1);
+                        const int pi = (e & 2) ? pi1 : pi0;
+                        const int dist = pi - j;
+                        const bool vis = ((e & 2) ? ok1 : ok0) && dist >= 0 &&
+                                         (window <= 0 || dist < window || j < keep_first) &&
+                                         (chunk <= 0 || pi / chunk == j / chunk);
+                        if (!vis) s[i][e] = -INFINITY;
+                    }
+                    if (e & 2) mx1 = fmaxf(mx1, s[i][e]); else mx0 = fmaxf(mx0, s[i][e]);
+                }
+            }
+        } else if (full) {
             const float jb = (float)(k0 + (lane & 3) * 2);
             const float c0 = sl2 * (jb - (float)pi0), c1 = sl2 * (jb - (float)pi1);     // -slope * (i - j) at column 0
 #pragma unroll
@@ -448,31 +534,39 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
                 }
             }
         }
-        mx0 = mma::quad_max(mx0);
-        mx1 = mma::quad_max(mx1);
-        const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-        const float ms0 = mn0 == -INFINITY ? 0.f : mn0, ms1 = mn1 == -INFINITY ? 0.f : mn1;
-        const float a0 = exp2f(m0 - ms0), a1 = exp2f(m1 - ms1);
-        m0 = mn0;
-        m1 = mn1;
-        float ps0 = 0.f, ps1 = 0.f;
+        if (MODE == 2) {                                  // sigmoid weights: no maximum, no denominator
 #pragma unroll
-        for (int i = 0; i < MK / 8; ++i) {
-            s[i][0] = exp2f(s[i][0] - ms0);
-            s[i][1] = exp2f(s[i][1] - ms0);
-            s[i][2] = exp2f(s[i][2] - ms1);
-            s[i][3] = exp2f(s[i][3] - ms1);
-            ps0 += s[i][0] + s[i][1];
-            ps1 += s[i][2] + s[i][3];
-        }
-        l0 = l0 * a0 + ps0;
-        l1 = l1 * a1 + ps1;
+            for (int i = 0; i < MK / 8; ++i)
 #pragma unroll
-        for (int i = 0; i < DV / 8; ++i) {
-            o[i][0] *= a0;
-            o[i][1] *= a0;
-            o[i][2] *= a1;
-            o[i][3] *= a1;
+                for (int e = 0; e < 4; ++e)
+                    s[i][e] = s[i][e] == -INFINITY ? 0.f : score::sigmoid_log2(s[i][e] + pb2);
+        } else {
+            mx0 = mma::quad_max(mx0);
+            mx1 = mma::quad_max(mx1);
+            const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+            const float ms0 = mn0 == -INFINITY ? 0.f : mn0, ms1 = mn1 == -INFINITY ? 0.f : mn1;
+            const float a0 = exp2f(m0 - ms0), a1 = exp2f(m1 - ms1);
+            m0 = mn0;
+            m1 = mn1;
+            float ps0 = 0.f, ps1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < MK / 8; ++i) {
+                s[i][0] = exp2f(s[i][0] - ms0);
+                s[i][1] = exp2f(s[i][1] - ms0);
+                s[i][2] = exp2f(s[i][2] - ms1);
+                s[i][3] = exp2f(s[i][3] - ms1);
+                ps0 += s[i][0] + s[i][1];
+                ps1 += s[i][2] + s[i][3];
+            }
+            l0 = l0 * a0 + ps0;
+            l1 = l1 * a1 + ps1;
+#pragma unroll
+            for (int i = 0; i < DV / 8; ++i) {
+                o[i][0] *= a0;
+                o[i][1] *= a0;
+                o[i][2] *= a1;
+                o[i][3] *= a1;
+            }
         }
         const uint32_t vb_addr = vs_addr + buf * MK * LDV * 2;
 #pragma unroll
@@ -500,7 +594,12 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
         l0 += exp2f(sk - (m0 == -INFINITY ? 0.f : m0));
         l1 += exp2f(sk - (m1 == -INFINITY ? 0.f : m1));
     }
-    const float i0 = (ok0 && l0 > 0.f) ? 1.f / l0 : 0.f, i1 = (ok1 && l1 > 0.f) ? 1.f / l1 : 0.f;
+    float i0 = (ok0 && l0 > 0.f) ? 1.f / l0 : 0.f, i1 = (ok1 && l1 > 0.f) ? 1.f / l1 : 0.f;
+    if (MODE == 2) i0 = ok0 ? 1.f : 0.f, i1 = ok1 ? 1.f : 0.f;
+    if (mod.gate != nullptr) {
+        if (ok0) i0 *= score::out_gate<bf16>(mod, (long long)b * Tn + q0 + r_lo, h);
+        if (ok1) i1 *= score::out_gate<bf16>(mod, (long long)b * Tn + q0 + r_lo + 8, h);
+    }
     bf16* out0 = out + (((long long)b * Tn + q0 + r_lo) * H + h) * DV + (lane & 3) * 2;
     bf16* out1 = out0 + (long long)8 * H * DV;
 #pragma unroll
@@ -510,16 +609,17 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
     }
 }
 
-template <int D, int DV>
+template <int D, int DV, int MODE = 0>
 int launch_prefill_mma(const void* q, const void* ck, const void* cv, CacheAddr ka, CacheAddr va, void* out,
                        const int* q_start, const int* n_new, const int* seq_ids, const float* slopes, int B, int Tn, int H,
-                       int G, float scale, int window, int keep_first, int chunk, const float* sinks, cudaStream_t st) {
+                       int G, float scale, int window, int keep_first, int chunk, const float* sinks, const ScoreMod& mod,
+                       cudaStream_t st) {
     const size_t smem = (size_t)(MQ * (D + 8) + 2 * MK * (D + 8) + 2 * MK * (DV + 8)) * sizeof(bf16);
-    auto kern = window_attn_prefill_mma_kernel<D, DV>;
+    auto kern = window_attn_prefill_mma_kernel<D, DV, MODE>;
     if (smem > 32 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     dim3 grid((Tn + MQ - 1) / MQ, H, B);
     kern<<<grid, M_THREADS, smem, st>>>((const bf16*)q, (const bf16*)ck, (const bf16*)cv, ka, va, (bf16*)out, q_start,
-                                        n_new, seq_ids, slopes, Tn, H, G, scale, window, keep_first, chunk, sinks);
+                                        n_new, seq_ids, slopes, Tn, H, G, scale, window, keep_first, chunk, sinks, mod);
     NXD_LAUNCH_CHECK();
     return 0;
 }
@@ -533,7 +633,7 @@ window_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ cache_k
                           CacheAddr ka, CacheAddr va, T* __restrict__ out, const int* __restrict__ positions,
                           const int* __restrict__ seq_ids, const float* __restrict__ slopes, int H, int G, int D, int Dv,
                           float scale, int window, int keep_first, int chunk, const float* __restrict__ sinks,
-                          int groups_per_kv) {
+                          int groups_per_kv, const ScoreMod mod) {
     extern __shared__ float smem[];
     const int R_all = H / G;
     const int g = blockIdx.x / groups_per_kv, sub_group = blockIdx.x % groups_per_kv;
@@ -555,13 +655,17 @@ window_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ cache_k
     const int lo = max(window > 0 ? max(0, p - window + 1) : 0, c_lo);
     const int n_sink = max(0, min(keep_first, lo) - c_lo);         // kept first tokens below the window, inside the chunk
     const int nk = n_sink + (p - lo + 1);
-    float m_r[DEC_R], l_r[DEC_R], sl[DEC_R];
+    const bool sig = mod.pb != nullptr;
+    float m_r[DEC_R], l_r[DEC_R], sl[DEC_R], r1[DEC_R], r2[DEC_R], pb[DEC_R];
     float acc[DEC_R][DEC_MV];
 #pragma unroll
     for (int r = 0; r < DEC_R; ++r) {
         m_r[r] = -INFINITY;
         l_r[r] = 0.f;
         sl[r] = (slopes != nullptr && r < R) ? slopes[h0 + r] : 0.f;
+        r1[r] = (mod.r1 != nullptr && r < R) ? mod.r1[h0 + r] : 0.f;
+        r2[r] = (mod.r1 != nullptr && r < R) ? mod.r2[h0 + r] : 0.f;
+        pb[r] = (sig && r < R) ? mod.pb[h0 + r] : 0.f;
 #pragma unroll
         for (int m = 0; m < DEC_MV; ++m) acc[r][m] = 0.f;
     }
@@ -588,10 +692,13 @@ window_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ cache_k
 #pragma unroll
         for (int r = 0; r < DEC_R; ++r) {
             if (r < R) {
-                const float s = warp_sum(d[r]) - sl[r] * dist;
-                const float m_new = fmaxf(m_r[r], s);
-                const float alpha = expf(m_r[r] - m_new);      // exp(-inf) = 0 on the first key
-                const float pw = expf(s - m_new);
+                float s = warp_sum(d[r]);
+                if (mod.cap > 0.f) s = mod.cap * score::tanh_any(s / mod.cap);
+                s -= sl[r] * dist;
+                if (mod.r1 != nullptr) s -= r1[r] * logf(1.f + r2[r] * dist);
+                const float m_new = sig ? 0.f : fmaxf(m_r[r], s);
+                const float alpha = sig ? 1.f : expf(m_r[r] - m_new);      // exp(-inf) = 0 on the first key
+                const float pw = sig ? score::sigmoid(s + pb[r]) : expf(s - m_new);
                 l_r[r] = l_r[r] * alpha + pw;
                 m_r[r] = m_new;
 #pragma unroll
@@ -630,7 +737,9 @@ window_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ cache_k
             den = fmaf(f, src[Dv + 1], den);
         }
         if (sinks != nullptr) den += expf(sinks[h0 + r] - (mx == -INFINITY ? 0.f : mx));
-        stf(out + ((long long)b * H + h0 + r) * Dv + c, den > 0.f ? num / den : 0.f);
+        if (sig) den = 1.f;
+        const float y = den > 0.f ? num / den : 0.f;
+        stf(out + ((long long)b * H + h0 + r) * Dv + c, y * score::out_gate<T>(mod, b, h0 + r));
     }
 }
 
@@ -645,13 +754,13 @@ constexpr int DM_THREADS = 128, DM_ROWS = 16;
 // gridDim.z CTAs: each recomputes the scores of its 16 query heads and accumulates its own VS output columns, so the
 // accumulator stays in registers; the other slices' reads of the same key rows hit L2.  QS: the query fragments are
 // re-read from shared memory at every step of the key dimension instead of living in registers (large D).
-template <int D, int DV, int VS, bool QS>
+template <int D, int DV, int VS, bool QS, int MODE>
 __global__ void __launch_bounds__(DM_THREADS)
 window_attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict__ cache_k,
                               const bf16* __restrict__ cache_v, CacheAddr ka, CacheAddr va, bf16* __restrict__ out,
                               const int* __restrict__ positions, const int* __restrict__ seq_ids,
                               const float* __restrict__ slopes, int H, int G, float scale, int window, int keep_first,
-                              int chunk, const float* __restrict__ sinks, int groups_per_kv) {
+                              int chunk, const float* __restrict__ sinks, int groups_per_kv, const ScoreMod mod) {
     constexpr int LDK = D + 8, LDV = VS + 8, CK = D / 8, CV = VS / 8;
     extern __shared__ __align__(16) unsigned char smem_raw[];
     bf16* Qs = reinterpret_cast<bf16*>(smem_raw);       // [DM_ROWS][LDK]
@@ -715,6 +824,16 @@ window_attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict
     const bool ok0 = r_lo < R, ok1 = r_lo + 8 < R;
     const float sl0 = (slopes != nullptr && ok0 ? slopes[h0 + r_lo] : 0.f) * LOG2E;
     const float sl1 = (slopes != nullptr && ok1 ? slopes[h0 + r_lo + 8] : 0.f) * LOG2E;
+    const float cap_in = (MODE > 0 && mod.cap > 0.f) ? scale / mod.cap : 0.f, cap_out = mod.cap * LOG2E;
+    float ra0 = 0.f, ra1 = 0.f, rb0 = 0.f, rb1 = 0.f, pb0 = 0.f, pb1 = 0.f;      // logarithmic bias, sigmoid offset per row
+    if (MODE > 0 && mod.r1 != nullptr) {
+        if (ok0) ra0 = mod.r1[h0 + r_lo] * LOG2E, rb0 = mod.r2[h0 + r_lo];
+        if (ok1) ra1 = mod.r1[h0 + r_lo + 8] * LOG2E, rb1 = mod.r2[h0 + r_lo + 8];
+    }
+    if (MODE == 2) {
+        if (ok0) pb0 = mod.pb[h0 + r_lo] * LOG2E;
+        if (ok1) pb1 = mod.pb[h0 + r_lo + 8] * LOG2E;
+    }
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     float o[VS / 8][4];
 #pragma unroll
@@ -758,30 +877,44 @@ window_attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict
                 const int dist = p - j;
                 const bool vis = ((e & 2) ? ok1 : ok0) && dist >= 0 &&
                                  (window <= 0 || dist < window || j < keep_first) && (chunk <= 0 || p / chunk == j / chunk);
-                const float v = vis ? s[i][e] * sc2 - ((e & 2) ? sl1 : sl0) * (float)dist : -INFINITY;
+                float t = s[i][e] * sc2;
+                if (MODE > 0 && cap_in > 0.f) t = cap_out * score::tanh_any(s[i][e] * cap_in);
+                if (MODE > 0 && mod.r1 != nullptr)
+                    t -= ((e & 2) ? ra1 : ra0) * __log2f(fmaf((e & 2) ? rb1 : rb0, (float)max(dist, 0), 1.f));
+                const float v = vis ? t - ((e & 2) ? sl1 : sl0) * (float)dist : -INFINITY;
                 s[i][e] = v;
                 if (e & 2) mx1 = fmaxf(mx1, v); else mx0 = fmaxf(mx0, v);
             }
         }
-        mx0 = mma::quad_max(mx0);
-        mx1 = mma::quad_max(mx1);
-        const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-        const float ms0 = mn0 == -INFINITY ? 0.f : mn0, ms1 = mn1 == -INFINITY ? 0.f : mn1;
-        const float a0 = exp2f(m0 - ms0), a1 = exp2f(m1 - ms1);
-        m0 = mn0;
-        m1 = mn1;
-        float ps0 = 0.f, ps1 = 0.f;
+        float a0 = 1.f, a1 = 1.f;
+        if (MODE == 2) {                                  // sigmoid weights: no maximum, no denominator
+            m0 = m1 = 0.f;
 #pragma unroll
-        for (int i = 0; i < 2; ++i) {
-            s[i][0] = exp2f(s[i][0] - ms0);
-            s[i][1] = exp2f(s[i][1] - ms0);
-            s[i][2] = exp2f(s[i][2] - ms1);
-            s[i][3] = exp2f(s[i][3] - ms1);
-            ps0 += s[i][0] + s[i][1];
-            ps1 += s[i][2] + s[i][3];
+            for (int i = 0; i < 2; ++i)
+#pragma unroll
+                for (int e = 0; e < 4; ++e)
+                    s[i][e] = s[i][e] == -INFINITY ? 0.f : score::sigmoid_log2(s[i][e] + ((e & 2) ? pb1 : pb0));
+        } else {
+            mx0 = mma::quad_max(mx0);
+            mx1 = mma::quad_max(mx1);
+            const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+            const float ms0 = mn0 == -INFINITY ? 0.f : mn0, ms1 = mn1 == -INFINITY ? 0.f : mn1;
+            a0 = exp2f(m0 - ms0), a1 = exp2f(m1 - ms1);
+            m0 = mn0;
+            m1 = mn1;
+            float ps0 = 0.f, ps1 = 0.f;
+#pragma unroll
+            for (int i = 0; i < 2; ++i) {
+                s[i][0] = exp2f(s[i][0] - ms0);
+                s[i][1] = exp2f(s[i][1] - ms0);
+                s[i][2] = exp2f(s[i][2] - ms1);
+                s[i][3] = exp2f(s[i][3] - ms1);
+                ps0 += s[i][0] + s[i][1];
+                ps1 += s[i][2] + s[i][3];
+            }
+            l0 = l0 * a0 + ps0;
+            l1 = l1 * a1 + ps1;
         }
-        l0 = l0 * a0 + ps0;
-        l1 = l1 * a1 + ps1;
         uint32_t pa[4];
         pa[0] = mma::pack2(s[0][0], s[0][1]);
         pa[1] = mma::pack2(s[0][2], s[0][3]);
@@ -844,22 +977,24 @@ window_attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict
             den = fmaf(f, src[VS + 1], den);
         }
         if (sinks != nullptr) den += exp2f(sinks[h0 + r] * LOG2E - (mx == -INFINITY ? 0.f : mx));
-        out[((long long)b * H + h0 + r) * DV + vz + c] = __float2bfloat16_rn(den > 0.f ? num / den : 0.f);
+        if (MODE == 2) den = 1.f;
+        const float y = den > 0.f ? num / den : 0.f;
+        out[((long long)b * H + h0 + r) * DV + vz + c] = __float2bfloat16_rn(y * score::out_gate<bf16>(mod, b, h0 + r));
     }
 }
 
-template <int D, int DV, int VS = DV>
+template <int D, int DV, int VS = DV, int MODE = 0>
 int launch_decode_mma(const void* q, const void* ck, const void* cv, CacheAddr ka, CacheAddr va, void* out,
                       const int* positions, const int* seq_ids, const float* slopes, int B, int H, int G, float scale,
-                      int window, int keep_first, int chunk, const float* sinks, cudaStream_t st) {
+                      int window, int keep_first, int chunk, const float* sinks, const ScoreMod& mod, cudaStream_t st) {
     const int groups = (H / G + DM_ROWS - 1) / DM_ROWS;
     static_assert(DV % VS == 0 && VS % 16 == 0, "value slices");
     const size_t smem = (size_t)(DM_ROWS * (D + 8) + 2 * MK * (D + 8) + 2 * MK * (VS + 8)) * sizeof(bf16);
-    auto kern = window_attn_decode_mma_kernel<D, DV, VS, (D > 256)>;
+    auto kern = window_attn_decode_mma_kernel<D, DV, VS, (D > 256), MODE>;
     if (smem > 32 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     dim3 grid(G * groups, B, DV / VS);
     kern<<<grid, DM_THREADS, smem, st>>>((const bf16*)q, (const bf16*)ck, (const bf16*)cv, ka, va, (bf16*)out, positions,
-                                         seq_ids, slopes, H, G, scale, window, keep_first, chunk, sinks, groups);
+                                         seq_ids, slopes, H, G, scale, window, keep_first, chunk, sinks, groups, mod);
     NXD_LAUNCH_CHECK();
     return 0;
 }
@@ -911,13 +1046,13 @@ template <typename T>
 int launch_prefill(const void* q, const void* ck, const void* cv, CacheAddr ka, CacheAddr va, void* out,
                    const int* q_start, const int* n_new, const int* seq_ids, const float* slopes, int B, int Tn, int H,
                    int G, int D, int Dv, float scale, int window, int keep_first, int chunk, const float* sinks,
-                   cudaStream_t st) {
+                   const ScoreMod& mod, cudaStream_t st) {
     const size_t smem = (size_t)(BQ * D + BK * (D + 1) + BK * Dv + BQ * BK) * sizeof(float);
     auto kern = window_attn_prefill_kernel<T>;
     if (smem > 32 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     dim3 grid((Tn + BQ - 1) / BQ, H, B);
     kern<<<grid, PF_THREADS, smem, st>>>((const T*)q, (const T*)ck, (const T*)cv, ka, va, (T*)out, q_start, n_new,
-                                         seq_ids, slopes, Tn, H, G, D, Dv, scale, window, keep_first, chunk, sinks);
+                                         seq_ids, slopes, Tn, H, G, D, Dv, scale, window, keep_first, chunk, sinks, mod);
     NXD_LAUNCH_CHECK();
     return 0;
 }
@@ -925,7 +1060,8 @@ int launch_prefill(const void* q, const void* ck, const void* cv, CacheAddr ka, 
 template <typename T, int DEC_R, int DEC_MV>
 int launch_decode_rm(const void* q, const void* ck, const void* cv, CacheAddr ka, CacheAddr va, void* out,
                      const int* positions, const int* seq_ids, const float* slopes, int B, int H, int G, int D, int Dv,
-                     float scale, int window, int keep_first, int chunk, const float* sinks, cudaStream_t st) {
+                     float scale, int window, int keep_first, int chunk, const float* sinks, const ScoreMod& mod,
+                     cudaStream_t st) {
     const int R_all = H / G;
     const int groups = (R_all + DEC_R - 1) / DEC_R;
     const size_t smem = (size_t)(DEC_R * D + DEC_WARPS * DEC_R * (Dv + 2)) * sizeof(float);
@@ -933,7 +1069,7 @@ int launch_decode_rm(const void* q, const void* ck, const void* cv, CacheAddr ka
     if (smem > 32 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     dim3 grid(G * groups, B);
     kern<<<grid, DEC_WARPS * 32, smem, st>>>((const T*)q, (const T*)ck, (const T*)cv, ka, va, (T*)out, positions, seq_ids,
-                                             slopes, H, G, D, Dv, scale, window, keep_first, chunk, sinks, groups);
+                                             slopes, H, G, D, Dv, scale, window, keep_first, chunk, sinks, groups, mod);
     NXD_LAUNCH_CHECK();
     return 0;
 }
@@ -941,12 +1077,13 @@ int launch_decode_rm(const void* q, const void* ck, const void* cv, CacheAddr ka
 template <typename T>
 int launch_decode(const void* q, const void* ck, const void* cv, CacheAddr ka, CacheAddr va, void* out,
                   const int* positions, const int* seq_ids, const float* slopes, int B, int H, int G, int D, int Dv,
-                  float scale, int window, int keep_first, int chunk, const float* sinks, cudaStream_t st) {
+                  float scale, int window, int keep_first, int chunk, const float* sinks, const ScoreMod& mod,
+                  cudaStream_t st) {
     if (Dv <= 256)
         return launch_decode_rm<T, 8, 8>(q, ck, cv, ka, va, out, positions, seq_ids, slopes, B, H, G, D, Dv, scale, window,
-                                         keep_first, chunk, sinks, st);
+                                         keep_first, chunk, sinks, mod, st);
     return launch_decode_rm<T, 4, 16>(q, ck, cv, ka, va, out, positions, seq_ids, slopes, B, H, G, D, Dv, scale, window,
-                                      keep_first, chunk, sinks, st);      // wide value rows: fewer heads per CTA
+                                      keep_first, chunk, sinks, mod, st);      // wide value rows: fewer heads per CTA
 }
 
 }  // namespace
@@ -961,20 +1098,25 @@ int launch_decode(const void* q, const void* ck, const void* cv, CacheAddr ka, C
 // key heads) of a row at once and q_weight / k_weight hold H * D / G * D values; row_stat [B * Tn, 2] fp32 scratch (or NULL:
 // every head's warp computes the row statistic itself).
 // value_from_key: the row has no value columns, the cached value is the raw key projection (taken ahead of the norm and the rotation).
-NXD_API int nxd_qk_prep_cache_write(int dtype, const void* qkv, long long ld, void* q_out, void* cache_k, void* cache_v,
+// bias [columns of the row] fp32 or NULL: added to the projection first; value_norm: every value head is divided by its
+// root mean square (eps inside the root, no weight) before it is cached.
+NXD_API int nxd_qkv_prep_cache_write(int dtype, const void* qkv, long long ld, void* q_out, void* cache_k, void* cache_v,
                                     long long k_stride_line, long long k_stride_head, long long v_stride_line,
                                     long long v_stride_head, const int* block_table, int page_size, int table_cols,
                                     const int* q_start, const int* n_new, const int* seq_ids, int B, int Tn, int H, int G,
                                     int D, int Dv, int has_kv, int normalize, float eps, int max_pos, int writeback,
                                     const float* q_weight, const float* k_weight, const float* rope_cos,
                                     const float* rope_sin, int rope_dims, int value_from_key, int value_heads,
-                                    int rope_halves, int whole_norm, float* row_stat, void* stream) {
+                                    int rope_halves, int whole_norm, float* row_stat, const float* bias, int value_norm,
+                                    void* stream) {
     const int Gv = value_heads > 0 ? value_heads : G;
     const long long units = (long long)B * Tn * (H + (has_kv ? G + Gv : 0));
     if (units == 0) return 0;
     NXD_REQUIRE(!value_from_key || Gv == G, "values taken from the keys need as many value heads (%d) as key heads (%d)", Gv, G);
     NXD_REQUIRE(rope_cos == nullptr || (rope_dims % 2 == 0 && rope_dims <= D), "rotation over %d of %d dimensions", rope_dims, D);
     NXD_REQUIRE(!value_from_key || Dv == D, "values taken from the keys need equal sizes (%d, %d)", D, Dv);
+    NXD_REQUIRE(!(value_from_key && (bias != nullptr || value_norm)), "values taken from the keys: no bias or norm of their %s", "own");
+    NXD_REQUIRE(!(writeback && whole_norm && normalize && row_stat == nullptr), "write-back under a whole-row norm needs %s", "row_stat");
     NXD_REQUIRE(!(writeback && rope_cos != nullptr), "write-back of rotated keys is not %s", "supported");
     const CacheAddr ka = make_addr(k_stride_line, k_stride_head, block_table, page_size, table_cols, D);
     const CacheAddr va = make_addr(v_stride_line, v_stride_head, block_table, page_size, table_cols, Dv);
@@ -986,24 +1128,39 @@ NXD_API int nxd_qk_prep_cache_write(int dtype, const void* qkv, long long ld, vo
         const unsigned sb = (unsigned)((rows + wpb - 1) / wpb);
         if (dtype == 0)
             qk_row_stat_kernel<bf16><<<sb, wpb * 32, 0, (cudaStream_t)stream>>>((const bf16*)qkv, ld, row_stat, rows, H * D,
-                                                                                has_kv ? G * D : 0, eps);
+                                                                                has_kv ? G * D : 0, eps, bias);
         else
             qk_row_stat_kernel<float><<<sb, wpb * 32, 0, (cudaStream_t)stream>>>((const float*)qkv, ld, row_stat, rows, H * D,
-                                                                                 has_kv ? G * D : 0, eps);
+                                                                                 has_kv ? G * D : 0, eps, bias);
         NXD_LAUNCH_CHECK();
     }
     if (dtype == 0)
         qk_norm_cache_write_kernel<bf16><<<blocks, wpb * 32, 0, (cudaStream_t)stream>>>(
             (const bf16*)qkv, ld, (bf16*)q_out, (bf16*)cache_k, (bf16*)cache_v, ka, va, q_start, n_new, seq_ids, units, Tn,
             H, G, D, Dv, has_kv, normalize, eps, max_pos, writeback, q_weight, k_weight, rope_cos, rope_sin, rope_dims,
-            value_from_key, Gv, rope_halves, whole_norm, row_stat);
+            value_from_key, Gv, rope_halves, whole_norm, row_stat, bias, value_norm);
     else
         qk_norm_cache_write_kernel<float><<<blocks, wpb * 32, 0, (cudaStream_t)stream>>>(
             (const float*)qkv, ld, (float*)q_out, (float*)cache_k, (float*)cache_v, ka, va, q_start, n_new, seq_ids, units,
             Tn, H, G, D, Dv, has_kv, normalize, eps, max_pos, writeback, q_weight, k_weight, rope_cos, rope_sin, rope_dims,
-            value_from_key, Gv, rope_halves, whole_norm, row_stat);
+            value_from_key, Gv, rope_halves, whole_norm, row_stat, bias, value_norm);
     NXD_LAUNCH_CHECK();
     return 0;
+}
+
+NXD_API int nxd_qk_prep_cache_write(int dtype, const void* qkv, long long ld, void* q_out, void* cache_k, void* cache_v,
+                                    long long k_stride_line, long long k_stride_head, long long v_stride_line,
+                                    long long v_stride_head, const int* block_table, int page_size, int table_cols,
+                                    const int* q_start, const int* n_new, const int* seq_ids, int B, int Tn, int H, int G,
+                                    int D, int Dv, int has_kv, int normalize, float eps, int max_pos, int writeback,
+                                    const float* q_weight, const float* k_weight, const float* rope_cos,
+                                    const float* rope_sin, int rope_dims, int value_from_key, int value_heads,
+                                    int rope_halves, int whole_norm, float* row_stat, void* stream) {
+    return nxd_qkv_prep_cache_write(dtype, qkv, ld, q_out, cache_k, cache_v, k_stride_line, k_stride_head, v_stride_line,
+                                    v_stride_head, block_table, page_size, table_cols, q_start, n_new, seq_ids, B, Tn, H,
+                                    G, D, Dv, has_kv, normalize, eps, max_pos, writeback, q_weight, k_weight, rope_cos,
+                                    rope_sin, rope_dims, value_from_key, value_heads, rope_halves, whole_norm, row_stat,
+                                    nullptr, 0, stream);
 }
 
 NXD_API int nxd_qk_norm_cache_write(int dtype, const void* qkv, long long ld, void* q_out, void* cache_k, void* cache_v,
@@ -1023,13 +1180,20 @@ NXD_API int nxd_qk_norm_cache_write(int dtype, const void* qkv, long long ld, vo
 // chunk <= 0: no chunks; sinks [H] fp32 or NULL.  k_row / v_row: elements between consecutive cache rows (D / Dv for
 // tensors of their own; v_row == k_row when the values are columns of the key rows).
 // impl: 0 = choose, 1 = the generic kernel, 2 = the tensor-core kernel (an error when it does not apply).
-NXD_API int nxd_masked_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v,
+// softcap <= 0: none; log_r1 / log_r2 [H] fp32 or NULL: logarithmic distance bias; sigmoid_bias [H] fp32 or NULL: sigmoid
+// weights instead of the softmax; gate (activation dtype, rows gate_ld elements apart) or NULL: output gate per head.
+NXD_API int nxd_scored_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v,
                                     long long k_stride_line, long long k_stride_head, long long k_row,
                                     long long v_stride_line, long long v_stride_head, long long v_row,
                                     const int* block_table, int page_size, int table_cols, void* out, const int* q_start,
                                     const int* n_new, const int* seq_ids, const float* slopes, const float* sinks, int B,
                                     int Tn, int H, int G, int D, int Dv, float scale, int window, int keep_first, int chunk,
-                                    int impl, int value_heads, void* stream) {
+                                    int impl, int value_heads, float softcap, const float* log_r1, const float* log_r2,
+                                    const float* sigmoid_bias, const void* gate, long long gate_ld, void* stream) {
+    NXD_REQUIRE((log_r1 == nullptr) == (log_r2 == nullptr), "attention: the logarithmic bias needs %s", "both vectors");
+    NXD_REQUIRE(sigmoid_bias == nullptr || sinks == nullptr, "attention: sigmoid weights have no %s", "sink");
+    const ScoreMod mod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld};
+    const int mode = mod.mode();
     NXD_REQUIRE(G > 0 && H % G == 0, "attention: %d query heads over %d key/value heads", H, G);
     NXD_REQUIRE(Dv <= MAXC * 8, "attention: value size %d above %d", Dv, MAXC * 8);
     if (B * Tn == 0) return 0;
@@ -1043,29 +1207,54 @@ NXD_API int nxd_masked_attn_prefill(int dtype, const void* q, const void* cache_
         (k_stride_line % 8) == 0 && (v_stride_line % 8) == 0 && (k_row % 8) == 0 && (v_row % 8) == 0 &&
         ((uintptr_t)cache_k % 16) == 0 && ((uintptr_t)cache_v % 16) == 0) {
 #define NXD_WA_CASE(DD, DDV)                                                                                          \
-    if (D == DD && Dv == DDV)                                                                                         \
+    if (mode == 0 && D == DD && Dv == DDV)                                                                            \
         return launch_prefill_mma<DD, DDV>(q, cache_k, cache_v, ka, va, out, q_start, n_new, seq_ids, slopes, B, Tn, H, \
-                                           G, scale, window, keep_first, chunk, sinks, st)
-        NXD_WA_CASE(32, 32);
-        NXD_WA_CASE(64, 64);
-        NXD_WA_CASE(96, 96);
-        NXD_WA_CASE(128, 128);
-        NXD_WA_CASE(64, 128);
-        NXD_WA_CASE(128, 64);
+                                           G, scale, window, keep_first, chunk, sinks, mod, st)
+#define NXD_WS_CASE(DD, DDV)                                                                                          \
+    NXD_WA_CASE(DD, DDV);                                                                                             \
+    if (mode == 1 && D == DD && Dv == DDV)                                                                            \
+        return launch_prefill_mma<DD, DDV, 1>(q, cache_k, cache_v, ka, va, out, q_start, n_new, seq_ids, slopes, B, Tn, \
+                                              H, G, scale, window, keep_first, chunk, sinks, mod, st);                \
+    if (mode == 2 && D == DD && Dv == DDV)                                                                            \
+        return launch_prefill_mma<DD, DDV, 2>(q, cache_k, cache_v, ka, va, out, q_start, n_new, seq_ids, slopes, B, Tn, \
+                                              H, G, scale, window, keep_first, chunk, sinks, mod, st)
+        NXD_WS_CASE(32, 32);
+        NXD_WS_CASE(64, 64);
+        NXD_WS_CASE(96, 96);
+        NXD_WS_CASE(128, 128);
+        NXD_WS_CASE(64, 128);
+        NXD_WS_CASE(128, 64);
         NXD_WA_CASE(96, 64);      // key size = un-rotated + rotated dimensions of an expanded latent head
         NXD_WA_CASE(192, 128);
         NXD_WA_CASE(32, 64);      // two attention maps of half the value size (differential attention)
         NXD_WA_CASE(48, 96);
         NXD_WA_CASE(96, 192);
         NXD_WA_CASE(128, 256);
+        NXD_WA_CASE(32, 48);      // expanded latent heads whose value is half as wide again as the key
+        NXD_WA_CASE(64, 96);
+        NXD_WA_CASE(128, 192);
+#undef NXD_WS_CASE
 #undef NXD_WA_CASE
     }
     NXD_REQUIRE(impl != 2, "attention: no tensor-core kernel for bf16=%d D=%d Dv=%d", dtype == 0, D, Dv);
     if (dtype == 0)
         return launch_prefill<bf16>(q, cache_k, cache_v, ka, va, out, q_start, n_new, seq_ids, slopes, B, Tn, H, G, D, Dv,
-                                    scale, window, keep_first, chunk, sinks, st);
+                                    scale, window, keep_first, chunk, sinks, mod, st);
     return launch_prefill<float>(q, cache_k, cache_v, ka, va, out, q_start, n_new, seq_ids, slopes, B, Tn, H, G, D, Dv,
-                                 scale, window, keep_first, chunk, sinks, st);
+                                 scale, window, keep_first, chunk, sinks, mod, st);
+}
+
+NXD_API int nxd_masked_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v,
+                                    long long k_stride_line, long long k_stride_head, long long k_row,
+                                    long long v_stride_line, long long v_stride_head, long long v_row,
+                                    const int* block_table, int page_size, int table_cols, void* out, const int* q_start,
+                                    const int* n_new, const int* seq_ids, const float* slopes, const float* sinks, int B,
+                                    int Tn, int H, int G, int D, int Dv, float scale, int window, int keep_first, int chunk,
+                                    int impl, int value_heads, void* stream) {
+    return nxd_scored_attn_prefill(dtype, q, cache_k, cache_v, k_stride_line, k_stride_head, k_row, v_stride_line,
+                                   v_stride_head, v_row, block_table, page_size, table_cols, out, q_start, n_new, seq_ids,
+                                   slopes, sinks, B, Tn, H, G, D, Dv, scale, window, keep_first, chunk, impl, value_heads,
+                                   0.f, nullptr, nullptr, nullptr, nullptr, 0, stream);
 }
 
 NXD_API int nxd_window_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v,
@@ -1080,13 +1269,18 @@ NXD_API int nxd_window_attn_prefill(int dtype, const void* q, const void* cache_
 }
 
 // q [B, H, D] of one new token per row at positions[b] (its key and value already in the cache) -> out [B, H, Dv].
-NXD_API int nxd_masked_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v,
+NXD_API int nxd_scored_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v,
                                    long long k_stride_line, long long k_stride_head, long long k_row,
                                    long long v_stride_line, long long v_stride_head, long long v_row,
                                    const int* block_table, int page_size, int table_cols, void* out, const int* positions,
                                    const int* seq_ids, const float* slopes, const float* sinks, int B, int H, int G, int D,
                                    int Dv, float scale, int window, int keep_first, int chunk, int impl, int value_heads,
-                                   void* stream) {
+                                   float softcap, const float* log_r1, const float* log_r2, const float* sigmoid_bias,
+                                   const void* gate, long long gate_ld, void* stream) {
+    NXD_REQUIRE((log_r1 == nullptr) == (log_r2 == nullptr), "attention: the logarithmic bias needs %s", "both vectors");
+    NXD_REQUIRE(sigmoid_bias == nullptr || sinks == nullptr, "attention: sigmoid weights have no %s", "sink");
+    const ScoreMod mod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld};
+    const int mode = mod.mode();
     NXD_REQUIRE(G > 0 && H % G == 0, "attention: %d query heads over %d key/value heads", H, G);
     NXD_REQUIRE(Dv <= 512, "attention: value size %d above %d", Dv, 512);
     if (B == 0) return 0;
@@ -1098,34 +1292,56 @@ NXD_API int nxd_masked_attn_decode(int dtype, const void* q, const void* cache_k
         (v_stride_line % 8) == 0 && (k_row % 8) == 0 && (v_row % 8) == 0 && ((uintptr_t)cache_k % 16) == 0 &&
         ((uintptr_t)cache_v % 16) == 0) {
 #define NXD_WD_CASE(DD, DDV)                                                                                          \
-    if (D == DD && Dv == DDV)                                                                                         \
+    if (mode == 0 && D == DD && Dv == DDV)                                                                            \
         return launch_decode_mma<DD, DDV>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G, scale, \
-                                          window, keep_first, chunk, sinks, st)
-        NXD_WD_CASE(32, 32);
-        NXD_WD_CASE(64, 64);
-        NXD_WD_CASE(96, 96);
-        NXD_WD_CASE(128, 128);
-        NXD_WD_CASE(64, 128);
-        NXD_WD_CASE(128, 64);
+                                          window, keep_first, chunk, sinks, mod, st)
+#define NXD_WDS_CASE(DD, DDV)                                                                                         \
+    NXD_WD_CASE(DD, DDV);                                                                                             \
+    if (mode == 1 && D == DD && Dv == DDV)                                                                            \
+        return launch_decode_mma<DD, DDV, DDV, 1>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G, \
+                                                  scale, window, keep_first, chunk, sinks, mod, st);                  \
+    if (mode == 2 && D == DD && Dv == DDV)                                                                            \
+        return launch_decode_mma<DD, DDV, DDV, 2>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G, \
+                                                  scale, window, keep_first, chunk, sinks, mod, st)
+        NXD_WDS_CASE(32, 32);
+        NXD_WDS_CASE(64, 64);
+        NXD_WDS_CASE(96, 96);
+        NXD_WDS_CASE(128, 128);
+        NXD_WDS_CASE(64, 128);
+        NXD_WDS_CASE(128, 64);
         NXD_WD_CASE(160, 128);    // latent rows: compressed key/value + shared rotated key part; value = the compressed part
         NXD_WD_CASE(32, 64);      // two attention maps of half the value size (differential attention)
         NXD_WD_CASE(48, 96);
         NXD_WD_CASE(96, 192);
         NXD_WD_CASE(128, 256);
+#undef NXD_WDS_CASE
 #undef NXD_WD_CASE
-        if (D == 288 && Dv == 256)                   // wide latent rows: the value columns are split over CTAs
+        if (mode == 0 && D == 288 && Dv == 256)                   // wide latent rows: the value columns are split over CTAs
             return launch_decode_mma<288, 256, 128>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G,
-                                                    scale, window, keep_first, chunk, sinks, st);
-        if (D == 576 && Dv == 512)
+                                                    scale, window, keep_first, chunk, sinks, mod, st);
+        if (mode == 0 && D == 576 && Dv == 512)
             return launch_decode_mma<576, 512, 128>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G,
-                                                    scale, window, keep_first, chunk, sinks, st);
+                                                    scale, window, keep_first, chunk, sinks, mod, st);
     }
     NXD_REQUIRE(impl != 2, "attention decode: no tensor-core kernel for bf16=%d D=%d Dv=%d", dtype == 0, D, Dv);
     if (dtype == 0)
         return launch_decode<bf16>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G, D, Dv, scale,
-                                   window, keep_first, chunk, sinks, st);
+                                   window, keep_first, chunk, sinks, mod, st);
     return launch_decode<float>(q, cache_k, cache_v, ka, va, out, positions, seq_ids, slopes, B, H, G, D, Dv, scale,
-                                window, keep_first, chunk, sinks, st);
+                                window, keep_first, chunk, sinks, mod, st);
+}
+
+NXD_API int nxd_masked_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v,
+                                   long long k_stride_line, long long k_stride_head, long long k_row,
+                                   long long v_stride_line, long long v_stride_head, long long v_row,
+                                   const int* block_table, int page_size, int table_cols, void* out, const int* positions,
+                                   const int* seq_ids, const float* slopes, const float* sinks, int B, int H, int G, int D,
+                                   int Dv, float scale, int window, int keep_first, int chunk, int impl, int value_heads,
+                                   void* stream) {
+    return nxd_scored_attn_decode(dtype, q, cache_k, cache_v, k_stride_line, k_stride_head, k_row, v_stride_line,
+                                  v_stride_head, v_row, block_table, page_size, table_cols, out, positions, seq_ids, slopes,
+                                  sinks, B, H, G, D, Dv, scale, window, keep_first, chunk, impl, value_heads, 0.f, nullptr,
+                                  nullptr, nullptr, nullptr, 0, stream);
 }
 
 NXD_API int nxd_window_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v,

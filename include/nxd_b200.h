@@ -330,6 +330,39 @@ int nxd_masked_attn_decode(int dtype, const void* q, const void* cache_k, const 
                            const int* positions, const int* seq_ids, const float* slopes, const float* sinks, int B, int H,
                            int G, int D, int Dv, float scale, int window, int keep_first, int chunk, int impl,
                            int value_heads, void* stream);
+/* The attention entry points with changes to the score and the head output (csrc/score_mod.cuh): softcap (<= 0: none),
+ * logarithmic distance bias log_r1_h * ln(1 + log_r2_h * (i - j)) (fp32 [H], both or neither), sigmoid_bias (fp32 [H]: weights
+ * sigmoid(score + b_h) instead of the softmax), gate (activation dtype, rows gate_ld apart: head h times sigmoid(gate)). */
+int nxd_scored_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v, long long k_stride_line,
+                            long long k_stride_head, long long k_row, long long v_stride_line, long long v_stride_head,
+                            long long v_row, const int* block_table, int page_size, int table_cols, void* out,
+                            const int* q_start, const int* n_new, const int* seq_ids, const float* slopes,
+                            const float* sinks, int B, int Tn, int H, int G, int D, int Dv, float scale, int window,
+                            int keep_first, int chunk, int impl, int value_heads, float softcap, const float* log_r1,
+                            const float* log_r2, const float* sigmoid_bias, const void* gate, long long gate_ld,
+                            void* stream);
+int nxd_scored_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v, long long k_stride_line,
+                           long long k_stride_head, long long k_row, long long v_stride_line, long long v_stride_head,
+                           long long v_row, const int* block_table, int page_size, int table_cols, void* out,
+                           const int* positions, const int* seq_ids, const float* slopes, const float* sinks, int B, int H,
+                           int G, int D, int Dv, float scale, int window, int keep_first, int chunk, int impl,
+                           int value_heads, float softcap, const float* log_r1, const float* log_r2,
+                           const float* sigmoid_bias, const void* gate, long long gate_ld, void* stream);
+/* nxd_qk_prep_cache_write with a projection bias (fp32, one number per column of the row, or NULL) and unit-RMS values */
+int nxd_qkv_prep_cache_write(int dtype, const void* qkv, long long ld, void* q_out, void* cache_k, void* cache_v,
+                             long long k_stride_line, long long k_stride_head, long long v_stride_line,
+                             long long v_stride_head, const int* block_table, int page_size, int table_cols,
+                             const int* q_start, const int* n_new, const int* seq_ids, int B, int Tn, int H, int G, int D,
+                             int Dv, int has_kv, int normalize, float eps, int max_pos, int writeback, const float* q_weight,
+                             const float* k_weight, const float* rope_cos, const float* rope_sin, int rope_dims,
+                             int value_from_key, int value_heads, int rope_halves, int whole_norm, float* row_stat,
+                             const float* bias, int value_norm, void* stream);
+/* tcgen05 attention forward from position 0 (tensors / strides as nxd_flash_attn_fwd_tc_window) with the same changes */
+int nxd_flash_attn_fwd_tc_scored(const void* q, const void* k, const void* v, void* o, const long long* strides, int B, int Hq,
+                                 int Hkv, int Sq, int Sk, int D, float scale, int window, int keep_first,
+                                 const float* slopes, const float* sinks, float softcap, const float* log_r1,
+                                 const float* log_r2, const float* sigmoid_bias, const void* gate, long long gate_ld,
+                                 void* stream);
 /* differential attention: maps [N, 2 * H, Dv] (first H heads = map 1, last H = map 2) -> out [N, H * Dv] =
  * rms_head(a1 - lambda * a2) * (1 - diff), lambda = exp(<lq1, lk1>) - exp(<lq2, lk2>) + diff (vectors fp32 [D]) */
 int nxd_diff_attn_combine(int dtype, const void* maps, void* out, const float* lq1, const float* lk1, const float* lq2,
@@ -344,7 +377,14 @@ int nxd_latent_prep(int dtype, const void* proj, long long ld, int q_off, int kv
  * [B, H, nsplit, Dv + 2]; returns 2 when no kernel is compiled for (D, Dv) */
 int nxd_latent_decode(const void* q, const void* cache, long long stride_line, long long row_pitch, const int* block_table,
                       int page_size, int table_cols, void* out, float* partial, const int* positions, const int* seq_ids,
-                      const float* sinks, int B, int H, int D, int Dv, float scale, int nsplit, void* stream);
+                      const float* sinks, int B, int H, int D, int Dv, float scale, int nsplit, int window,
+                      const void* gate, long long gate_ld, void* stream);
+/* latent projection without positions: normalised query latents -> cq, normalised key/value latents -> cache rows (and
+ * c_rows [B * Tn, rank] or NULL) */
+int nxd_latent_norms(int dtype, const void* proj, long long ld, int q_off, int kv_off, void* cq, void* c_rows, void* cache,
+                     long long stride_line, long long row_pitch, const int* block_table, int page_size, int table_cols,
+                     const float* q_weight, const float* c_weight, const int* q_start, const int* n_new, const int* seq_ids,
+                     int B, int Tn, int q_rank, int rank, float eps, int max_pos, void* stream);
 int nxd_mlstm_chunk_states(float* u, const float* ftot, const float* mloc, const float* s0, const float* m0, float* s_out,
                            float* m_start, float* m_out, long long BH, int NC, long long E, void* stream);
 /* recurrent matrix memory: fp32 gates (soft cap, log-sigmoid forget gate), scan over a step on the line's fp32 state,
@@ -434,6 +474,13 @@ int nxd_retention_chunkwise(int dtype, const void* proj, long long ld, int q_off
 int nxd_hc_step(int y_dtype, int h_dtype, float* X, const void* ya, const void* yb, const float* wa, const float* wb,
                 const float* mix, const float* outw, const float* inw, const float* wn, void* h, long long N, int S, int W,
                 float eps, void* stream);
+/* fp32 residual stream of plain pre-norm decoders (csrc/stream_norm.cu): x += y (+ bias) and the RMS norm that follows;
+ * token embedding (+ sinusoidal position vectors) with a norm of its own, and the norm that follows */
+int nxd_residual_norm(int y_dtype, int h_dtype, float* x, const void* y, const float* bias, const float* w, void* h,
+                      long long rows, int W, float eps, void* stream);
+int nxd_embed_norm(int e_dtype, int h_dtype, const void* table, const long long* ids, const long long* pos,
+                   const double* freq, const float* w_embed, const float* w_next, float* x, void* h, long long rows, int W,
+                   int vocab, float eps, void* stream);
 
 #ifdef __cplusplus
 }

@@ -1,5 +1,5 @@
 """Hybrid families (recurrent mixers next to attention over the cache) over the framework's step function: Rasodra and,
-further down, Gogalix and Vufasun.
+further down, Gogalix, Vufasun and Tidavik (windowed attention of several kinds, no recurrence).
 
 Rasodra over the framework's step function: chunked attention, latent attention and the recurrent matrix memory on
 one KV cache / state manager.
@@ -30,9 +30,11 @@ import torch
 
 from ..models.gogalix import UNIT_NORM_EPS, GogalixConfig, GogalixForCausalLM
 from ..models.rasodra import RasodraConfig, RasodraForCausalLM
+from ..models.tidavik import POSITION_BASE, TidavikConfig, TidavikForCausalLM
 from ..models.vufasun import VufasunConfig, VufasunForCausalLM
 from ..ops import activation as act_ops
 from ..ops import attention as attn_ops
+from ..ops import backend, decode_fused
 from ..ops import delta_rule as delta_ops
 from ..ops import hyper_connection as hc_ops
 from ..ops import latent_attention as la_ops
@@ -41,6 +43,7 @@ from ..ops import moe_sparse as moe_ops
 from ..ops import norm as norm_ops
 from ..ops import retention as ret_ops
 from ..ops import rope as rope_ops
+from ..ops import stream_norm as sn_ops
 from ..ops import window_attention as wa_ops
 from ..ops.linear import gemm_nt
 from .config import InferenceConfig
@@ -48,7 +51,40 @@ from .kv_cache import KVCache
 from .model import KVCacheInferenceMixin
 
 
-class RasodraInferenceModel(KVCacheInferenceMixin, RasodraForCausalLM):
+class CacheRowsMixin:
+    """What the families with a latent cache ask of the KV cache inside a step."""
+
+    def _paged(self) -> dict:
+        kc = self.kv_cache
+        return dict(block_table=kc.block_table, page_size=kc.page_size) if kc.paged else {}
+
+    def _latent_rows(self, ck, lines, n_ctx: int, first: int = 0) -> torch.Tensor:
+        """Rows ``[first, n_ctx)`` of the given cache lines of a latent cache tensor, ``[len(lines), n_ctx - first, columns]``."""
+        kc = self.kv_cache
+        if not kc.paged:
+            return ck[lines.long(), 0, first:n_ctx]
+        p0, p1 = first // kc.page_size, (n_ctx + kc.page_size - 1) // kc.page_size
+        pages = kc.block_table[lines.long(), p0:p1].long()                         # [B, pages]
+        rows = ck[pages][:, :, 0].reshape(pages.shape[0], (p1 - p0) * kc.page_size, ck.shape[-1])
+        return rows[:, first - p0 * kc.page_size: n_ctx - p0 * kc.page_size]
+
+    def _step_context_len(self, q_start, n_new, T: int) -> int:
+        """Positions that the step's rows reach at most.  A step that starts every row at position 0 needs no look at the
+        device (T, which keeps the step capturable in a CUDA graph); a step of portions reads it back once."""
+        return self._step_context(q_start, n_new, T)[1]
+
+    def _step_context(self, q_start, n_new, T: int) -> Tuple[int, int]:
+        """``(first, end)``: the smallest first position of the step's rows and the positions they reach at most."""
+        if not self._step_past_context:
+            return 0, T
+        if "context" not in self._step_kv:
+            ends = q_start + (n_new if n_new is not None else T)
+            first, end = torch.stack([q_start.min(), ends.max()]).tolist()
+            self._step_kv["context"] = (int(first), int(end))
+        return self._step_kv["context"]
+
+
+class RasodraInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, RasodraForCausalLM):
     supports_prefill_at_offset = True
 
     def __init__(self, config: RasodraConfig, inference_config: Optional[InferenceConfig] = None, device=None):
@@ -111,10 +147,6 @@ class RasodraInferenceModel(KVCacheInferenceMixin, RasodraForCausalLM):
         return y.reshape(x.shape[:-1] + (linear.weight.shape[0],))
 
     # -- mixers: h [B, T, W] in the activation dtype -> [B, T, W] ---------------------------------------------------------
-    def _paged(self) -> dict:
-        kc = self.kv_cache
-        return dict(block_table=kc.block_table, page_size=kc.page_size) if kc.paged else {}
-
     TC_PREFILL_MIN_TOKENS = 128          # shorter steps stay on the cache-reading kernels
 
     def _chunks_as_batch(self, qk, m, T: int) -> bool:
@@ -149,24 +181,6 @@ class RasodraInferenceModel(KVCacheInferenceMixin, RasodraForCausalLM):
             o = wa_ops.window_attention_prefill(q, ck, cv, q_start, m.scale, n_new=n_new, seq_ids=seq_ids, chunk=m.chunk,
                                                 **paged)
         return self._proj(mixer.o_proj, o.reshape(B, T, m.heads * m.vdim))
-
-    def _latent_rows(self, ck, lines, n_ctx: int) -> torch.Tensor:
-        """Rows ``[0, n_ctx)`` of the given cache lines of a latent cache tensor, ``[len(lines), n_ctx, rank + rot]``."""
-        kc = self.kv_cache
-        if not kc.paged:
-            return ck[lines.long(), 0, :n_ctx]
-        n_pages = (n_ctx + kc.page_size - 1) // kc.page_size
-        pages = kc.block_table[lines.long(), :n_pages].long()                      # [B, n_pages]
-        return ck[pages][:, :, 0].reshape(pages.shape[0], n_pages * kc.page_size, ck.shape[-1])[:, :n_ctx]
-
-    def _step_context_len(self, q_start, n_new, T: int) -> int:
-        """Positions that the step's rows reach at most.  A step that starts every row at position 0 needs no look at the
-        device (T, which keeps the step capturable in a CUDA graph); a step of portions reads it back once."""
-        if not self._step_past_context:
-            return T
-        if "n_ctx" not in self._step_kv:
-            self._step_kv["n_ctx"] = int((q_start + (n_new if n_new is not None else T)).max())
-        return self._step_kv["n_ctx"]
 
     def _mix_latent(self, i, mixer, h, q_start, n_new, seq_ids):
         m, cfg, dt = mixer.cfg, self.config, self.config.torch_dtype
@@ -572,6 +586,177 @@ class VufasunInferenceModel(KVCacheInferenceMixin, VufasunForCausalLM):
         if self.layer_probe is not None:
             self.layer_probe(i, x.sum(dim=1).view(B, T, W))
         return x.view(B, T, SW), (h_next.view(B, T, W) if h_next is not None else None)
+
+    def forward_speculation(self, *a, **kw):
+        raise NotImplementedError("the speculation verify graph is not wired for this family")
+
+
+class TidavikInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, TidavikForCausalLM):
+    """Tidavik over the KV cache.  The step function (padding, cache lines through ``seq_ids``, indexed logits, sampler,
+    ``generate``), the schedulers and the runners are the mixin's; this class says what the entry and a layer do:
+
+      * ``hidden`` is the fp32 stream, ``residual`` the normed copy that the sublayer about to run reads, in the activation
+        dtype: embedding + position vector + entry norm + the first layer's norm are one kernel, and so are the residual
+        add (with the sublayer's output bias) and the next norm (``ops.stream_norm``);
+      * ONE matrix product of the mixer's input gives all its projections (``layer.in_proj``, parts at ``layer.columns``);
+      * latent layers: both latents normed in one kernel that also writes the cache row, query up-projection; prompt steps
+        expand keys and values from the latent rows (only those that some window of the step reaches) with one product and
+        attend over them, token generation absorbs the key up-projection into the query and attends over the cached rows;
+        the per-head output gate is applied inside the attention kernels;
+      * the other layers: bias, whole-projection norm of q and k or unit-RMS values, and the cache write in one kernel,
+        then the windowed attention with soft cap and logarithmic bias and sigmoid weights, or soft cap and a zero-score
+        sink;
+      * bf16 prompts from position 0 with equal key and value sizes of 64 or 128 run on the tcgen05 attention kernel, q / k /
+        v read as views of the projection outputs.
+    A step may start at any position: attention reads earlier keys from the cache."""
+
+    supports_prefill_at_offset = True
+    TC_PREFILL_MIN_TOKENS = 128          # shorter steps stay on the cache-reading attention kernels
+
+    def __init__(self, config: TidavikConfig, inference_config: Optional[InferenceConfig] = None, device=None):
+        TidavikForCausalLM.__init__(self, config, device=device)
+        self._init_inference(inference_config)
+        self._position_freq: Optional[torch.Tensor] = None
+        self.layer_probe = None            # callable(i, x) after every layer (debugging / layer-by-layer checks)
+
+    def _decoder_layers(self):
+        return self.layers
+
+    def _embedding(self):
+        return self.embed_tokens
+
+    def _final_norm(self):
+        return self.norm
+
+    def init_kv_cache(self, device=None, dtype=None) -> KVCache:
+        ic, cfg = self.inference_config, self.config
+        device = device or next(self.parameters()).device
+        specs = []
+        for L in cfg.layers:
+            m = L.mixer
+            specs.append((1, m.kv_rank, m.kv_rank, "columns") if L.type == "latent_attention" else (m.kv_heads, m.dim, m.vdim))
+        self.kv_cache = KVCache(len(specs), ic.max_batch_size, 0, ic.seq_len, 0, dtype=dtype or cfg.torch_dtype,
+                                device=device, paged=ic.paged_kv, page_size=ic.page_size,
+                                num_pages=ic.num_kv_pages if ic.paged_kv else None, layer_specs=specs)
+        return self.kv_cache
+
+    def _embed_step(self, input_ids: torch.Tensor, position_ids: torch.Tensor):
+        cfg = self.config
+        if self._position_freq is None or self._position_freq.device != input_ids.device:
+            self._position_freq = sn_ops.position_frequencies(cfg.hidden_size, POSITION_BASE, device=input_ids.device)
+        first = self.layers[0].norm1 if len(self.layers) else None
+        return sn_ops.embed_norm(self.embed_tokens.weight, input_ids, position_ids.expand_as(input_ids), self._position_freq,
+                                 self.embed_norm, cfg.rms_norm_eps, first, cfg.torch_dtype)
+
+    def _add_norm(self, norm, hidden: torch.Tensor, residual: Optional[torch.Tensor]):
+        """Only the model's final norm comes through here: plain RMS norm of the fp32 stream."""
+        return sn_ops.residual_norm_(hidden.contiguous(), None, w_next=norm, eps=self.config.rms_norm_eps,
+                                     out_dtype=self.config.torch_dtype)[1], None
+
+    def _tc_prefill(self, x: torch.Tensor, m, T: int) -> bool:
+        return (T >= self.TC_PREFILL_MIN_TOKENS and not self._step_past_context
+                and wa_ops.tc_prefill_applies(x, m.dim, m.vdim, x.stride(-2)))
+
+    # -- mixers: big [B, T, n_out] = the fused projection of the normed input -> [N, W] before the output bias -------------
+    def _mix_latent(self, i, layer, big, q_start, n_new, seq_ids):
+        mixer, m, cfg, dt = layer.mixer, layer.mixer.cfg, self.config, self.config.torch_dtype
+        B, T, _ = big.shape
+        N, H, D, Dv, R = B * T, m.heads, m.dim, m.vdim, m.kv_rank
+        ck, cv = self.kv_cache.layer(i)
+        paged = self._paged()
+        at = layer.columns
+        gate = big[..., at["g"][0]: at["g"][0] + H]
+        from_zero = T > 1 and not self._step_past_context
+        cq, c = la_ops.latent_norms(big, at["dq"][0], at["dkv"][0], m.q_rank, R, ck, mixer.q_norm, mixer.kv_norm, q_start,
+                                    cfg.rms_norm_eps, n_new=n_new, seq_ids=seq_ids, rows=from_zero, **paged)
+        q = gemm_nt(cq, mixer.uq_proj.weight)
+        if T == 1:
+            q_abs = torch.empty(N, H, R, dtype=dt, device=big.device)
+            torch.bmm(q.view(N, H, D).transpose(0, 1), mixer.uk(), out=q_abs.transpose(0, 1))
+            o_lat = wa_ops.window_attention_decode(q_abs, ck, cv, q_start, m.scale, m.window, seq_ids=seq_ids,
+                                                   gate=gate[:, 0], **paged)
+            o = torch.empty(N, H, Dv, dtype=dt, device=big.device)
+            torch.bmm(o_lat.transpose(0, 1), mixer.uv().transpose(1, 2), out=o.transpose(0, 1))
+            return gemm_nt(o.view(N, H * Dv), mixer.o_proj.weight)
+        if from_zero:
+            first, rows = 0, c.view(B, T, R)
+        else:
+            lo, end = self._step_context(q_start, n_new, T)
+            first = max(0, lo - m.window + 1) if m.window else 0
+            lines = seq_ids if seq_ids is not None else torch.arange(B, device=big.device)
+            rows = self._latent_rows(ck, lines, end, first).contiguous()
+        n_ctx = rows.shape[1]
+        kv = gemm_nt(rows.reshape(B * n_ctx, R), mixer.ukv_proj.weight).view(B, n_ctx, H * (D + Dv))
+        keys, vals = kv[..., : H * D].unflatten(-1, (H, D)), kv[..., H * D:].unflatten(-1, (H, Dv))
+        q4 = q.view(B, T, H, D)
+        if self._tc_prefill(kv, m, T):
+            o = wa_ops.window_attention_tc(q4.permute(0, 2, 1, 3), keys.permute(0, 2, 1, 3), vals.permute(0, 2, 1, 3),
+                                           m.scale, m.window, gate=gate).permute(0, 2, 1, 3)
+        else:                               # positions count from the first expanded row
+            o = wa_ops.window_attention_prefill(q4, keys.permute(0, 2, 1, 3), vals.permute(0, 2, 1, 3),
+                                                q_start - first if first else q_start, m.scale, m.window, n_new=n_new,
+                                                gate=gate)
+        return gemm_nt(o.reshape(N, H * Dv), mixer.o_proj.weight)
+
+    def _mix_scored(self, i, layer, big, q_start, n_new, seq_ids):
+        mixer, m, cfg = layer.mixer, layer.mixer.cfg, self.config
+        B, T, _ = big.shape
+        H, G, D, Dv = m.heads, m.kv_heads, m.dim, m.vdim
+        ck, cv = self.kv_cache.layer(i)
+        paged = self._paged()
+        qkv = big[..., : m.columns]
+        tc = T > 1 and self._tc_prefill(qkv, m, T)
+        q = wa_ops.qk_norm_cache_write(qkv, ck, cv, q_start, H, G, D, Dv, cfg.rms_norm_eps, n_new=n_new, seq_ids=seq_ids,
+                                       normalize=m.sigmoid, whole_norm=m.sigmoid, q_weight=mixer.q_norm,
+                                       k_weight=mixer.k_norm, bias=mixer.qkv_bias, value_norm=not m.sigmoid, writeback=tc,
+                                       **paged)
+        kw = mixer.score_args()
+        if T == 1:
+            o = wa_ops.window_attention_decode(q[:, 0], ck, cv, q_start, m.scale, m.window, seq_ids=seq_ids, **kw, **paged)
+        elif tc:
+            k = qkv[..., H * D: (H + G) * D].unflatten(-1, (G, D)).permute(0, 2, 1, 3)
+            v = qkv[..., (H + G) * D:].unflatten(-1, (G, Dv)).permute(0, 2, 1, 3)
+            o = wa_ops.window_attention_tc(q.permute(0, 2, 1, 3), k, v, m.scale, m.window, **kw).permute(0, 2, 1, 3)
+        else:
+            o = wa_ops.window_attention_prefill(q, ck, cv, q_start, m.scale, m.window, n_new=n_new, seq_ids=seq_ids, **kw,
+                                                **paged)
+        return gemm_nt(o.reshape(B * T, H * Dv), mixer.o_proj.weight)
+
+    _MIX = {"latent_attention": _mix_latent, "attention": _mix_scored, "attention_2": _mix_scored}
+
+    def _feed_forward(self, mlp, h2: torch.Tensor) -> torch.Tensor:
+        N, w = h2.shape[0], mlp.gate_up_proj.weight
+        if backend.gemm_backend() == "tcgen05" and decode_fused.qualifies(h2):
+            act = decode_fused.gate_up_swiglu(h2, None, 0.0, w)
+        elif (backend.gemm_backend() == "tcgen05" and N <= decode_fused.BATCHED_SWIGLU_MAX_ROWS
+              and decode_fused.qualifies_batched(h2)):
+            act = decode_fused.gate_up_swiglu_batched(h2, w)
+        else:
+            act = moe_ops.glu_bias(gemm_nt(h2, w), 0, mlp.ff_pad, mlp.ff_pad)
+        return gemm_nt(act, mlp.down_proj.weight)
+
+    # -- one layer --------------------------------------------------------------------------------------------------
+    def _layer(self, i: int, layer, hidden, residual, positions, seq_ids, lengths, prefill):
+        cfg, dt, eps = self.config, self.config.torch_dtype, self.config.rms_norm_eps
+        B, T, W = hidden.shape
+        N = B * T
+        x = (hidden if hidden.is_contiguous() else hidden.contiguous()).view(N, W)
+        h = residual.reshape(N, W)
+        if "q_start" not in self._step_kv:      # one int32 copy of the rows' first positions per step, not per kernel
+            self._step_kv["q_start"] = positions[:, 0].to(torch.int32).contiguous()
+        q_start = self._step_kv["q_start"]
+        n_new = self._step_new_tokens if prefill else None
+        big = gemm_nt(h, layer.in_proj.weight).view(B, T, -1)
+        y = self._MIX[layer.type](self, i, layer, big, q_start, n_new, seq_ids)
+        nxt = self.layers[i + 1].norm1 if i + 1 < len(self.layers) else None
+        if layer.mlp is None:
+            x, h = sn_ops.residual_norm_(x, y, layer.mixer.o_bias, nxt, eps, dt)
+        else:
+            x, h = sn_ops.residual_norm_(x, y, layer.mixer.o_bias, layer.norm2, eps, dt)
+            x, h = sn_ops.residual_norm_(x, self._feed_forward(layer.mlp, h), None, nxt, eps, dt)
+        if self.layer_probe is not None:
+            self.layer_probe(i, x.view(B, T, W))
+        return x.view(B, T, W), (h.view(B, T, W) if h is not None else None)
 
     def forward_speculation(self, *a, **kw):
         raise NotImplementedError("the speculation verify graph is not wired for this family")

@@ -316,9 +316,8 @@ class KVCacheInferenceMixin:
         self._step_new_tokens = ((last_token_index + 1).to(torch.int32) if (prefill and last_token_index is not None)
                                  else None)
         default_lines = seq_ids is None
-        hidden = self._embed(input_ids)
+        hidden, residual = self._embed_step(input_ids, position_ids)
         lengths = (position_ids[:, -1] + 1).to(torch.int32)
-        residual = None
         # token generation without continuous batching: row b IS cache line b -- never gather cache lines by seq_ids
         # (an index_select of a [B, Hkv, S, D] cache per layer and token costs more than the attention itself)
         identity = default_lines or not self.inference_config.is_continuous_batching
@@ -377,6 +376,10 @@ class KVCacheInferenceMixin:
                 last_token_index: Optional[torch.Tensor] = None):
         """Calling the inference model runs one graph: context encoding (T > 1) or token generation (T == 1)."""
         return self.forward_infer(input_ids, position_ids, seq_ids, last_token_index)
+
+    def _embed_step(self, input_ids: torch.Tensor, position_ids: torch.Tensor):
+        """``(hidden, residual)`` ahead of the first layer; families whose entry needs the positions override this."""
+        return self._embed(input_ids), None
 
     def _embed(self, input_ids: torch.Tensor) -> torch.Tensor:
         emb = self._embedding()

@@ -142,6 +142,24 @@ def _vufasun_cls():
     return VufasunInferenceModel
 
 
+def _tidavik_config(d, dtype):
+    from ..models.tidavik import TidavikConfig
+
+    return TidavikConfig.from_dict(d, torch_dtype=dtype)
+
+
+def _tidavik_convert(sd, cfg):
+    from ..models.tidavik import convert_tidavik_state_dict
+
+    return convert_tidavik_state_dict(sd, cfg)
+
+
+def _tidavik_cls():
+    from .hybrid import TidavikInferenceModel
+
+    return TidavikInferenceModel
+
+
 register_family(ModelFamily("llama", lambda c: _arch(c).startswith("llama"), _llama_config, _llama_cls, _llama_convert))
 register_family(ModelFamily("gekazen", lambda c: _arch(c) == "gekazen", _gekazen_config, _gekazen_cls, _gekazen_convert,
                             kernel_group="window_moe_serving"))
@@ -151,6 +169,8 @@ register_family(ModelFamily("gogalix", lambda c: _arch(c) == "gogalix", _gogalix
                             kernel_group="delta_serving"))
 register_family(ModelFamily("vufasun", lambda c: _arch(c) == "vufasun", _vufasun_config, _vufasun_cls, _vufasun_convert,
                             kernel_group="retention_serving"))
+register_family(ModelFamily("tidavik", lambda c: _arch(c) == "tidavik", _tidavik_config, _tidavik_cls, _tidavik_convert,
+                            kernel_group="scored_serving"))
 
 
 def read_config(model_dir: str) -> Dict[str, Any]:

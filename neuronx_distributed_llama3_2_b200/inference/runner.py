@@ -374,6 +374,16 @@ class GogalixRunner(InferenceRunner):
         super().__init__(*a, **kw)
 
 
+class TidavikRunner(InferenceRunner):
+    """Runner of the Tidavik family (``models/tidavik.py``): same buckets, graphs and generate loop."""
+
+    def __init__(self, *a, **kw):
+        from .hybrid import TidavikInferenceModel
+
+        kw.setdefault("model_cls", TidavikInferenceModel)
+        super().__init__(*a, **kw)
+
+
 class VufasunRunner(InferenceRunner):
     """Runner of the Vufasun family (``models/vufasun.py``): same buckets, graphs and generate loop."""
 

@@ -13,3 +13,5 @@ from .gogalix import (GogalixConfig, GogalixForCausalLM, convert_gogalix_state_d
                       tiny_gogalix)
 from .vufasun import (VufasunConfig, VufasunForCausalLM, convert_vufasun_state_dict, export_vufasun_state_dict,  # noqa: F401
                       tiny_vufasun)
+from .tidavik import (TidavikConfig, TidavikForCausalLM, convert_tidavik_state_dict, export_tidavik_state_dict,  # noqa: F401
+                      tiny_tidavik)

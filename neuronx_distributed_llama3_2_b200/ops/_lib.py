@@ -68,8 +68,16 @@ GROUPS["retention_serving"] = ["window_attention.cu", "moe_sparse.cu", "mlstm.cu
                                "runtime.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "fused_gemm_ar.cu", "tma_host.cu",
                                "flash_attn_tc.cu", "attn_tc_host.cu"]
 
+# the scored-attention family (latent attention behind low-rank queries, soft-capped and sigmoid attention in sliding
+# windows, dense gated feed-forward on a pre-norm fp32 stream): attention over the cache, latent rows, the stream's norms,
+# the gated activation, the GEMM kernels behind the linear layers with their fused token-generation form, and the tcgen05
+# flash attention of prompts
+GROUPS["scored_serving"] = ["window_attention.cu", "latent_attention.cu", "stream_norm.cu", "moe_sparse.cu", "runtime.cu",
+                            "gemm_tcgen05.cu", "gemm_smallm.cu", "decode_fused.cu", "fused_gemm_ar.cu", "tma_host.cu",
+                            "flash_attn_tc.cu", "attn_tc_host.cu"]
+
 # sources whose fp32 state is carried over thousands of steps: no approximate exp / tanh / division
-PRECISE_SOURCES = {"mlstm.cu", "delta_rule.cu", "retention.cu", "hyper_connection.cu"}
+PRECISE_SOURCES = {"mlstm.cu", "delta_rule.cu", "retention.cu", "hyper_connection.cu", "stream_norm.cu"}
 
 _lib: Optional[ctypes.CDLL] = None
 _group_libs = {}

@@ -6,6 +6,10 @@
     score(i, j)   = scale * <q_i, k_j> - slope_h * (i - j)
     p(i, j)       = exp(score(i, j)) / (sum over visible j' of exp(score(i, j')) [+ exp(sink_h)])
 
+``log_bias = (r1, r2)``: ``score -= r1_h * ln(1 + r2_h * (i - j))``; ``softcap``: ``score = cap * tanh(score / cap)`` ahead
+of the distance biases; ``sigmoid_bias``: the weights are ``sigmoid(score + b_h)``, not normalised over the keys, instead of
+the softmax; ``gate``: the output of head ``h`` is multiplied by ``sigmoid`` of that head's pre-activation.
+
 ``sinks``: a learned per-head logit that is attached to no position and only takes probability mass.  The value rows may be
 a column range of the key rows (``cache_v`` a view of ``cache_k``): the cache of a compressed key/value projection.
 
@@ -78,8 +82,12 @@ def qk_norm_cache_write(qkv: torch.Tensor, cache_k: Optional[torch.Tensor], cach
                         page_size: int = 0, writeback: bool = False, q_weight: Optional[torch.Tensor] = None,
                         k_weight: Optional[torch.Tensor] = None, rope: Optional[tuple] = None,
                         value_from_key: bool = False, value_heads: Optional[int] = None, rope_layout: str = "pairs",
-                        whole_norm: bool = False) -> torch.Tensor:
-    """``q_weight / k_weight [dim]``: weight of the per-head norm (after the division).  ``rope = (cos, sin)`` tables
+                        whole_norm: bool = False, bias: Optional[torch.Tensor] = None,
+                        value_norm: bool = False) -> torch.Tensor:
+    """``bias`` (one fp32 number per column of ``qkv``): added to the projection ahead of everything else.  ``value_norm``:
+    every value head is divided by its root mean square over ``vdim`` (no weight) before it is cached.
+
+    ``q_weight / k_weight [dim]``: weight of the per-head norm (after the division).  ``rope = (cos, sin)`` tables
     ``[positions, rot/2]`` (``ops.rope.build_interleaved_rope_cache``): queries and keys turn pairwise on their first
     ``rot`` dimensions, after the norm; pair ``i`` is the dimensions ``(2i, 2i + 1)`` (``rope_layout="pairs"``) or
     ``(i, i + rot/2)`` (``"halves"``).  ``value_from_key``: the projection has no value columns, the cached value is
@@ -91,7 +99,8 @@ def qk_norm_cache_write(qkv: torch.Tensor, cache_k: Optional[torch.Tensor], cach
     key and value heads of the real rows (``t < n_new[b]``) are written at position ``q_start[b] + t`` of cache line
     ``seq_ids[b]``.  ``normalize``: queries and keys are divided by their root mean square over ``dim`` (fp32, ``eps``
     inside the root) before they are written.  ``writeback``: the normalised keys of the real rows also replace the
-    raw ones inside ``qkv`` (for a kernel that reads q / k / v as strided views of the projection output).
+    raw ones inside ``qkv`` (for a kernel that reads q / k / v as strided views of the projection output), and so do the
+    values where ``bias`` or ``value_norm`` changes them.
     ``value_heads``: the row holds that many value heads instead of ``kv_heads`` (value head ``g`` then serves the key
     heads ``g, g + value_heads, ...``: several attention maps over the same values).  ``qkv`` may be a column range of
     a wider projection output (rows ``stride(1)`` apart)."""
@@ -118,7 +127,8 @@ def qk_norm_cache_write(qkv: torch.Tensor, cache_k: Optional[torch.Tensor], cach
         cos, sin = rope if rope is not None else (None, None)
         # scratch of the whole-projection statistics (1 / rms of all query heads, of all key heads, per row)
         stat = torch.empty(B * T, 2, dtype=torch.float32, device=qkv.device) if (whole_norm and normalize) else None
-        rc = L.nxd_qk_prep_cache_write(_c.c_int(_code(qkv.dtype)), _lib.ptr(qkv), _c.c_longlong(ld), _lib.ptr(q),
+        bias_c = bias.float().contiguous() if bias is not None else None
+        rc = L.nxd_qkv_prep_cache_write(_c.c_int(_code(qkv.dtype)), _lib.ptr(qkv), _c.c_longlong(ld), _lib.ptr(q),
                                        _lib.ptr(ck), _lib.ptr(cv), *cargs, _lib.ptr(qs), _lib.ptr(nn_), _lib.ptr(sid),
                                        _c.c_int(B), _c.c_int(T), _c.c_int(heads), _c.c_int(kv_heads), _c.c_int(dim),
                                        _c.c_int(vdim), _c.c_int(int(has_kv)), _c.c_int(int(normalize)), _c.c_float(eps),
@@ -126,8 +136,8 @@ def qk_norm_cache_write(qkv: torch.Tensor, cache_k: Optional[torch.Tensor], cach
                                        _lib.ptr(cos), _lib.ptr(sin), _c.c_int(2 * cos.shape[1] if cos is not None else 0),
                                        _c.c_int(int(value_from_key)), _c.c_int(gv),
                                        _c.c_int(int(rope_layout == "halves")), _c.c_int(int(whole_norm)),
-                                       _lib.ptr(stat), _lib.stream_ptr())
-        _lib.check(rc, "nxd_qk_prep_cache_write", L)
+                                       _lib.ptr(stat), _lib.ptr(bias_c), _c.c_int(int(value_norm)), _lib.stream_ptr())
+        _lib.check(rc, "nxd_qkv_prep_cache_write", L)
         return q
 
     pos_bt = q_start.long().reshape(B, 1) + torch.arange(T, device=qkv.device).reshape(1, T)
@@ -144,19 +154,27 @@ def qk_norm_cache_write(qkv: torch.Tensor, cache_k: Optional[torch.Tensor], cach
             from .rope import rope_halves_ref, rope_interleaved_ref
 
             xf = (rope_halves_ref if rope_layout == "halves" else rope_interleaved_ref)(xf, pos_bt, rope[0], rope[1])
-        return xf.to(x.dtype)
+        return xf.to(qkv.dtype)
 
-    q = unit(qkv[..., : heads * dim].reshape(B, T, heads, dim), q_weight)
+    raw = qkv
+    if bias is not None:
+        raw = raw.float() + bias.float()
+    q = unit(raw[..., : heads * dim].reshape(B, T, heads, dim), q_weight)
     if has_kv:
-        k_raw = qkv[..., heads * dim: (heads + kv_heads) * dim].reshape(B, T, kv_heads, dim)
+        k_raw = raw[..., heads * dim: (heads + kv_heads) * dim].reshape(B, T, kv_heads, dim)
         k = unit(k_raw, k_weight)
-        v = k_raw if value_from_key else qkv[..., (heads + kv_heads) * dim:].reshape(B, T, gv, vdim)
+        v = k_raw if value_from_key else raw[..., (heads + kv_heads) * dim:].reshape(B, T, gv, vdim)
+        if value_norm:
+            v = v.float() / torch.sqrt(v.float().pow(2).mean(-1, keepdim=True) + eps)
+        k, v = k.to(cache_k.dtype), v.to(cache_v.dtype)
         for b in range(B):
             n = T if n_new is None else int(n_new[b])
             line = b if seq_ids is None else int(seq_ids[b])
             p0 = int(q_start[b])
             if writeback:
                 qkv[b, :n, heads * dim: (heads + kv_heads) * dim] = k[b, :n].reshape(n, kv_heads * dim)
+                if bias is not None or value_norm:
+                    qkv[b, :n, (heads + kv_heads) * dim:] = v[b, :n].reshape(n, gv * vdim)
             for t in range(n):
                 pos = p0 + t
                 if block_table is not None:
@@ -171,7 +189,9 @@ def qk_norm_cache_write(qkv: torch.Tensor, cache_k: Optional[torch.Tensor], cach
 
 def window_attention_ref(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_pos: torch.Tensor, scale: float,
                          window: Optional[int], keep_first: int, slopes: Optional[torch.Tensor],
-                         chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
+                         softcap: Optional[float] = None, log_bias: Optional[tuple] = None,
+                         sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One sequence in fp32: ``q [Tq, H, D]`` at positions ``q_pos [Tq]`` over keys ``k [G, Tk, D]`` / ``v [Gv, Tk, Dv]``
     at positions ``0 .. Tk - 1``; with fewer value heads than key heads, key head ``g`` reads value head ``g % Gv``."""
     H, G = q.shape[1], k.shape[0]
@@ -188,16 +208,39 @@ def window_attention_ref(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_po
     if chunk:
         vis = vis & (torch.div(q_pos.reshape(-1, 1), chunk, rounding_mode="floor")
                      == torch.div(j.reshape(1, -1), chunk, rounding_mode="floor"))
+    if softcap:
+        s = softcap * torch.tanh(s / softcap)
     if slopes is not None:
         s = s - slopes.float().reshape(H, 1, 1) * dist.float()
+    if log_bias is not None:
+        r1, r2 = (t.float().reshape(H, 1, 1) for t in log_bias)
+        s = s - r1 * torch.log(1.0 + r2 * dist.clamp(min=0).float())
     s = s.masked_fill(~vis, float("-inf"))
+    g = torch.sigmoid(gate.float()).unsqueeze(-1) if gate is not None else 1.0          # [Tq, H, 1]
+    if sigmoid_bias is not None:
+        assert sinks is None
+        p = torch.sigmoid(s + sigmoid_bias.float().reshape(H, 1, 1))                      # masked scores: weight 0
+        return torch.einsum("hqk,hkd->qhd", p, vf) * g
     if sinks is not None:
         s = torch.cat([s, sinks.float().reshape(H, 1, 1).expand(H, s.shape[1], 1)], dim=-1)
     p = torch.softmax(s, dim=-1)
     if sinks is not None:
         p = p[..., :-1]
     p = torch.nan_to_num(p, nan=0.0)                                      # a row that sees nothing
-    return torch.einsum("hqk,hkd->qhd", p, vf)
+    return torch.einsum("hqk,hkd->qhd", p, vf) * g
+
+
+def _mod_args(softcap, log_bias, sigmoid_bias, gate, x):
+    """The score / output modifications of an attention call as C arguments (and the tensors to keep alive)."""
+    r1, r2 = (t.float().contiguous() for t in log_bias) if log_bias is not None else (None, None)
+    pb = sigmoid_bias.float().contiguous() if sigmoid_bias is not None else None
+    if gate is not None:
+        assert gate.dtype == x.dtype and gate.stride(-1) == 1
+        assert gate.dim() == 2 or gate.shape[0] == 1 or gate.stride(0) == gate.shape[1] * gate.stride(1)
+    ld = gate.stride(-2) if gate is not None else 0
+    return (_c.c_float(float(softcap) if softcap else 0.0), _lib.ptr(r1), _lib.ptr(r2), _lib.ptr(pb), _lib.ptr(gate),
+            _c.c_longlong(ld)), (r1, r2, pb)
+
 
 
 def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tensor, q_start: torch.Tensor,
@@ -205,8 +248,12 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
                              slopes: Optional[torch.Tensor] = None, n_new: Optional[torch.Tensor] = None,
                              seq_ids: Optional[torch.Tensor] = None, block_table: Optional[torch.Tensor] = None,
                              page_size: int = 0, impl: str = "auto", chunk: Optional[int] = None,
-                             sinks: Optional[torch.Tensor] = None, value_heads: Optional[int] = None) -> torch.Tensor:
-    """``impl``: ``auto`` | ``generic`` (fp32-math tile kernel, any sizes) | ``mma`` (bf16 tensor-core kernel, an error
+                             sinks: Optional[torch.Tensor] = None, value_heads: Optional[int] = None,
+                             softcap: Optional[float] = None, log_bias: Optional[tuple] = None,
+                             sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``gate [B, T, H]``: output gate pre-activations (may be a column range of a projection output).
+
+    ``impl``: ``auto`` | ``generic`` (fp32-math tile kernel, any sizes) | ``mma`` (bf16 tensor-core kernel, an error
     where it does not apply) -- for tests and measurements.
 
     ``q [B, T, H, D]``: new tokens of every row at positions ``q_start[b] + t`` (their keys / values already in the
@@ -221,14 +268,15 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
         cargs, bt = _cache_args(cache_k, cache_v, block_table, page_size, rows=True)
         sk = sinks.float().contiguous() if sinks is not None else None
         L = _lib.lib(GROUP)
-        rc = L.nxd_masked_attn_prefill(_c.c_int(_code(q.dtype)), _lib.ptr(q), _lib.ptr(cache_k), _lib.ptr(cache_v),
+        margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q)
+        rc = L.nxd_scored_attn_prefill(_c.c_int(_code(q.dtype)), _lib.ptr(q), _lib.ptr(cache_k), _lib.ptr(cache_v),
                                        *cargs, _lib.ptr(out), _lib.ptr(qs), _lib.ptr(nn_), _lib.ptr(sid),
                                        _lib.ptr(slopes), _lib.ptr(sk), _c.c_int(B), _c.c_int(T), _c.c_int(H), _c.c_int(G),
                                        _c.c_int(D), _c.c_int(Dv), _c.c_float(scale), _c.c_int(w), _c.c_int(keep_first),
                                        _c.c_int(int(chunk) if chunk else 0),
                                        _c.c_int({"auto": 0, "generic": 1, "mma": 2}[impl]),
-                                       _c.c_int(int(value_heads) if value_heads else 0), _lib.stream_ptr())
-        _lib.check(rc, "nxd_masked_attn_prefill", L)
+                                       _c.c_int(int(value_heads) if value_heads else 0), *margs, _lib.stream_ptr())
+        _lib.check(rc, "nxd_scored_attn_prefill", L)
         return out
     out = torch.zeros(B, T, H, Dv, dtype=q.dtype, device=q.device)
     for b in range(B):
@@ -240,7 +288,8 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
         kk = _cache_rows(cache_k, line, p0 + n, block_table, page_size)
         vv = _cache_rows(cache_v, line, p0 + n, block_table, page_size)
         pos = torch.arange(p0, p0 + n, device=q.device)
-        out[b, :n] = window_attention_ref(q[b, :n], kk, vv, pos, scale, w, keep_first, slopes, chunk, sinks).to(q.dtype)
+        out[b, :n] = window_attention_ref(q[b, :n], kk, vv, pos, scale, w, keep_first, slopes, chunk, sinks,
+                                          softcap, log_bias, sigmoid_bias, gate[b, :n] if gate is not None else None).to(q.dtype)
     return out
 
 
@@ -249,9 +298,11 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
                             slopes: Optional[torch.Tensor] = None, seq_ids: Optional[torch.Tensor] = None,
                             block_table: Optional[torch.Tensor] = None, page_size: int = 0,
                             impl: str = "auto", chunk: Optional[int] = None,
-                            sinks: Optional[torch.Tensor] = None, value_heads: Optional[int] = None) -> torch.Tensor:
+                            sinks: Optional[torch.Tensor] = None, value_heads: Optional[int] = None,
+                            softcap: Optional[float] = None, log_bias: Optional[tuple] = None,
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One new token per row: ``q [B, H, D]`` at ``positions[b]`` -> ``[B, H, Dv]``; only the kept first rows and the
-    window's rows of the cache line are read."""
+    window's rows of the cache line are read.  ``gate [B, H]``: output gate pre-activations."""
     B, H, D = q.shape
     G, Dv = cache_k.shape[1], cache_v.shape[3]
     w = int(window) if window else 0
@@ -261,23 +312,25 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
         pos, sid = _i32(positions), _i32(seq_ids)
         cargs, bt = _cache_args(cache_k, cache_v, block_table, page_size, rows=True)
         sk = sinks.float().contiguous() if sinks is not None else None
-        if (impl == "auto" and q.dtype == torch.bfloat16 and G == 1 and not w and not chunk and slopes is None
+        plain = not softcap and log_bias is None and sigmoid_bias is None
+        if (impl == "auto" and q.dtype == torch.bfloat16 and G == 1 and not keep_first and not chunk and slopes is None and plain
                 and cache_v.data_ptr() == cache_k.data_ptr() and cache_v.stride(2) == cache_k.stride(2)
                 and cache_v.stride(0) == cache_k.stride(0)):
             # latent rows (one key/value head, values = the first columns of the key rows): the kernel that streams the
             # rows once per 16 query heads, with the context split over CTAs when the batch alone does not fill the GPU
             from . import latent_attention as la
 
-            if la.latent_decode(q, cache_k, Dv, out, pos, sid, sk, scale, bt, page_size):
+            if la.latent_decode(q, cache_k, Dv, out, pos, sid, sk, scale, bt, page_size, w, gate):
                 return out
         L = _lib.lib(GROUP)
-        rc = L.nxd_masked_attn_decode(_c.c_int(_code(q.dtype)), _lib.ptr(q), _lib.ptr(cache_k), _lib.ptr(cache_v), *cargs,
+        margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q)
+        rc = L.nxd_scored_attn_decode(_c.c_int(_code(q.dtype)), _lib.ptr(q), _lib.ptr(cache_k), _lib.ptr(cache_v), *cargs,
                                       _lib.ptr(out), _lib.ptr(pos), _lib.ptr(sid), _lib.ptr(slopes), _lib.ptr(sk),
                                       _c.c_int(B), _c.c_int(H), _c.c_int(G), _c.c_int(D), _c.c_int(Dv), _c.c_float(scale),
                                       _c.c_int(w), _c.c_int(keep_first), _c.c_int(int(chunk) if chunk else 0),
                                       _c.c_int({"auto": 0, "generic": 1, "mma": 2}[impl]),
-                                      _c.c_int(int(value_heads) if value_heads else 0), _lib.stream_ptr())
-        _lib.check(rc, "nxd_masked_attn_decode", L)
+                                      _c.c_int(int(value_heads) if value_heads else 0), *margs, _lib.stream_ptr())
+        _lib.check(rc, "nxd_scored_attn_decode", L)
         return out
     out = torch.empty(B, H, Dv, dtype=q.dtype, device=q.device)
     for b in range(B):
@@ -286,7 +339,8 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
         kk = _cache_rows(cache_k, line, p + 1, block_table, page_size)
         vv = _cache_rows(cache_v, line, p + 1, block_table, page_size)
         out[b] = window_attention_ref(q[b:b + 1], kk, vv, torch.tensor([p], device=q.device), scale, w, keep_first,
-                                      slopes, chunk, sinks)[0].to(q.dtype)
+                                      slopes, chunk, sinks, softcap, log_bias, sigmoid_bias,
+                                      gate[b:b + 1] if gate is not None else None)[0].to(q.dtype)
     return out
 
 
@@ -324,11 +378,14 @@ def tc_prefill_applies(q: torch.Tensor, dim: int, vdim: int, n_out: int) -> bool
 
 
 def window_attention_tc(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float, window: Optional[int] = None,
-                        keep_first: int = 0, slopes: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        keep_first: int = 0, slopes: Optional[torch.Tensor] = None,
+                        sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
+                        log_bias: Optional[tuple] = None, sigmoid_bias: Optional[torch.Tensor] = None,
+                        gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Prefill from position 0 on the tcgen05 flash-attention kernel (``csrc/flash_attn_tc.cu``, windowed
     instantiation): ``q [B, H, T, D]``, ``k / v [B, G, T, D]`` as (strided) views with unit stride on ``D`` ->
     ``[B, H, T, D]`` stored as ``[B, T, H, D]``.  All rows are taken as ``T`` tokens long (right padding only ever
-    sits behind the real tokens of a causal row)."""
+    sits behind the real tokens of a causal row).  ``gate [B, T, H]``: output gate pre-activations."""
     from .flash_attn import _fix, _strides
 
     q, k, v = _fix(q), _fix(k), _fix(v)
@@ -336,9 +393,11 @@ def window_attention_tc(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale
     G = k.shape[1]
     o = torch.empty(B, T, H, D, dtype=q.dtype, device=q.device).permute(0, 2, 1, 3)
     L = _lib.lib()
-    rc = L.nxd_flash_attn_fwd_tc_window(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), _lib.ptr(o), _strides(q, k, v, o),
+    margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q)
+    sk = sinks.float().contiguous() if sinks is not None else None
+    rc = L.nxd_flash_attn_fwd_tc_scored(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), _lib.ptr(o), _strides(q, k, v, o),
                                         _c.c_int(B), _c.c_int(H), _c.c_int(G), _c.c_int(T), _c.c_int(T), _c.c_int(D),
                                         _c.c_float(scale), _c.c_int(int(window) if window else 0), _c.c_int(keep_first),
-                                        _lib.ptr(slopes), _lib.stream_ptr())
-    _lib.check(rc, "nxd_flash_attn_fwd_tc_window")
+                                        _lib.ptr(slopes), _lib.ptr(sk), *margs, _lib.stream_ptr())
+    _lib.check(rc, "nxd_flash_attn_fwd_tc_scored", L)
     return o
