@@ -127,8 +127,8 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     }
     if (warp == 1) ptx::tmem_alloc<1>(tmem_ptr_smem, L::kTmemCols);
     float* dtab = reinterpret_cast<float*>(sP);          // bias table (SCORE): the P staging area is free, P lives in TMEM
-    constexpr float kL2e = score::kLog2e;
-    const float r1 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r1[hq] * kL2e : 0.f;
+    constexpr float kL2e = score::kLog2e;                // r1 ln(.) in log2 units is r1 log2(.)
+    const float r1 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r1[hq] : 0.f;
     const float r2 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r2[hq] : 0.f;
     if (SCORE > 0 && p.bias_entries > 0) {
         const float sl = p.slopes != nullptr ? p.slopes[hq] * kL2e : 0.f;

@@ -408,7 +408,7 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
     for (int i = 0; i < DV / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
     uint32_t qf[D / 16][4];
     const bool biased = MODE > 0 && (mod.r1 != nullptr || slopes != nullptr);
-    const float r1 = (MODE > 0 && mod.r1 != nullptr) ? mod.r1[h] * LOG2E : 0.f;
+    const float r1 = (MODE > 0 && mod.r1 != nullptr) ? mod.r1[h] : 0.f;
     const float r2 = (MODE > 0 && mod.r1 != nullptr) ? mod.r2[h] : 0.f;
     const float pb2 = MODE == 2 ? mod.pb[h] * LOG2E : 0.f;
     const float cap_in = (MODE > 0 && mod.cap > 0.f) ? scale / mod.cap : 0.f, cap_out = mod.cap * LOG2E;
@@ -827,8 +827,8 @@ window_attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict
     const float cap_in = (MODE > 0 && mod.cap > 0.f) ? scale / mod.cap : 0.f, cap_out = mod.cap * LOG2E;
     float ra0 = 0.f, ra1 = 0.f, rb0 = 0.f, rb1 = 0.f, pb0 = 0.f, pb1 = 0.f;      // logarithmic bias, sigmoid offset per row
     if (MODE > 0 && mod.r1 != nullptr) {
-        if (ok0) ra0 = mod.r1[h0 + r_lo] * LOG2E, rb0 = mod.r2[h0 + r_lo];
-        if (ok1) ra1 = mod.r1[h0 + r_lo + 8] * LOG2E, rb1 = mod.r2[h0 + r_lo + 8];
+        if (ok0) ra0 = mod.r1[h0 + r_lo], rb0 = mod.r2[h0 + r_lo];
+        if (ok1) ra1 = mod.r1[h0 + r_lo + 8], rb1 = mod.r2[h0 + r_lo + 8];
     }
     if (MODE == 2) {
         if (ok0) pb0 = mod.pb[h0 + r_lo] * LOG2E;

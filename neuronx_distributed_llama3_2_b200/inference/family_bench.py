@@ -767,3 +767,184 @@ def run_retention(steps: int = 10, warmup: int = 3, device=None, sizes=None) -> 
         out["kernels"][s["name"]] = retention_kernel_cases(s, steps, warmup, dev)
     out["gpu_launches"] = _lib.kernel_launches() - before
     return out
+
+
+# ---- Tidavik next to Rasodra (attention over the cache and latent attention with a dense feed-forward) ------------------------
+def tidavik_config(s: dict):
+    from ..models.tidavik import TidavikConfig
+
+    # gate, up and down of (width x f) against Rasodra's two matrices of (width x ff): f = 2/3 ff keeps the parameters equal
+    ff = {"kind": "dense", "ff": (2 * s["ff"] // 3 + 127) // 128 * 128}
+    mask = {"size": s["chunk"]}
+    att = {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+           "softcap": 30.0, "mask": mask}
+    lat = {"heads": s["heads"], "dim": s["lat_dim"], "vdim": s["lat_vdim"], "q_rank": 2 * s["rank"], "kv_rank": s["rank"],
+           "scale": s["lat_dim"] ** -0.5, "mask": mask}
+    return TidavikConfig.from_dict({
+        "architecture": "Tidavik", "vocab": VOCAB, "width": s["width"], "norm": {"eps": 1e-6},
+        "layers": [{"type": "attention", "mixer": att, "mlp": ff}, {"type": "attention_2", "mixer": att, "mlp": ff},
+                   {"type": "latent_attention", "mixer": lat, "mlp": ff},
+                   {"type": "latent_attention", "mixer": lat, "mlp": ff}]}, torch_dtype=torch.bfloat16)
+
+
+def rasodra_attention_config(s: dict):
+    """Rasodra without its recurrent layer: chunked attention twice, latent attention twice."""
+    from ..models.rasodra import RasodraConfig
+
+    d = rasodra_config(s).to_dict()
+    att, _, lat, _ = d["layers"]
+    d["layers"] = [att, att, lat, lat]
+    return RasodraConfig.from_dict(d, torch_dtype=torch.bfloat16)
+
+
+def scored_serve_case(s: dict, steps: int, warmup: int, dev) -> dict:
+    from .hybrid import RasodraInferenceModel, TidavikInferenceModel
+
+    timer = _Timer(dev)
+    out = {"size": dict(s)}
+    ic = dict(batch_size=s["decode_batch"], max_batch_size=s["decode_batch"], max_context_length=s["prompt"],
+              seq_len=s["prompt"] + 64, is_continuous_batching=True, use_cuda_graphs=False)
+    for name, make in (("tidavik", lambda: TidavikInferenceModel(tidavik_config(s), InferenceConfig(**ic), device=dev)),
+                       ("rasodra", lambda: RasodraInferenceModel(rasodra_attention_config(s), InferenceConfig(**ic), device=dev))):
+        torch.manual_seed(0)
+        model = make()
+        model.init_kv_cache(device=dev)
+        out[name] = _serve(model, s, timer, steps, warmup, dev)
+        out[name]["parameters"] = sum(p.numel() for p in model.parameters())
+        del model
+        torch.cuda.empty_cache()
+    out["tidavik_over_rasodra"] = {k: out["tidavik"][k] / out["rasodra"][k]
+                                   for k in ("prefill_tokens_per_s", "decode_tokens_per_s")}
+    return out
+
+
+def scored_kernel_cases(s: dict, steps: int, warmup: int, dev) -> List[dict]:
+    """Tidavik's own kernels on the shapes of ``s``, alone, with roofline fractions, each next to the like kernel of the
+    Rasodra / Gekazen families (windowed attention without score modifications, latent decode, projection epilogue,
+    residual and norm, activation)."""
+    from ..ops import latent_attention as la
+    from ..ops import rope as rope_ops
+    from ..ops import stream_norm as sn
+
+    pk = peaks()
+    timer = _Timer(dev)
+    bf = torch.bfloat16
+    B, T, H, G, D, W, Bd = s["prefill_batch"], s["prompt"], s["heads"], s["kv_heads"], s["dim"], s["width"], s["decode_batch"]
+    win, S, N = s["chunk"], T + 64, B * T
+    rows = []
+
+    def row(kernel, like, fn, flops=None, nbytes=None):
+        ms = timer(fn, steps, warmup)
+        r = {"kernel": kernel, "like": like, "ms": ms, "peak": pk["source"]}
+        if flops is not None:
+            r["tflops"] = flops / ms / 1e9
+            r["of_peak"] = r["tflops"] / pk["bf16_tflops"]
+        if nbytes is not None:
+            r["gbs"] = nbytes / ms / 1e6
+            r["of_peak"] = r["gbs"] / pk["hbm_gbs"]
+        rows.append(r)
+
+    zero = torch.zeros(B, dtype=torch.int32, device=dev)
+    pairs = sum(min(i + 1, win) for i in range(T))
+    r1, r2, pb = torch.full((H,), 0.5, device=dev), torch.full((H,), 0.2, device=dev), torch.full((H,), -5.0, device=dev)
+    one = torch.zeros(H, device=dev)
+    kinds = [("soft cap + logarithmic bias + sigmoid weights", dict(softcap=30.0, log_bias=(r1, r2), sigmoid_bias=pb)),
+             ("soft cap + one in the denominator", dict(softcap=30.0, sinks=one)),
+             ("plain softmax (the like kernel)", {})]
+    # prompts on the tcgen05 kernel (views of the projection output), and over the cache
+    qkv = torch.randn(B, T, (H + 2 * G) * D, device=dev, dtype=bf)
+    view = lambda a, n: qkv[..., a * D: (a + n) * D].unflatten(-1, (n, D)).permute(0, 2, 1, 3)               # noqa: E731
+    q4, k4, v4 = view(0, H), view(H, G), view(H + G, G)
+    for name, kw in kinds:
+        row(f"windowed prefill, tcgen05: {name}", "prefill attention",
+            lambda: wa.window_attention_tc(q4, k4, v4, D ** -0.5, win, **kw), flops=4.0 * D * pairs * H * B)
+    q = torch.randn(B, T, H, D, device=dev, dtype=bf)
+    ck = torch.randn(max(B, Bd), G, S, D, device=dev, dtype=bf)
+    cv = torch.randn(max(B, Bd), G, S, D, device=dev, dtype=bf)
+    for name, kw in kinds:
+        row(f"windowed prefill over the cache, mma.sync: {name}", "prefill attention",
+            lambda: wa.window_attention_prefill(q, ck, cv, zero, D ** -0.5, win, **kw), flops=4.0 * D * pairs * H * B)
+    qd = torch.randn(Bd, H, D, device=dev, dtype=bf)
+    posd = torch.full((Bd,), T, dtype=torch.int32, device=dev)
+    for name, kw in kinds:
+        row(f"windowed decode: {name}", "decode attention",
+            lambda: wa.window_attention_decode(qd, ck, cv, posd, D ** -0.5, win, **kw), nbytes=2.0 * win * G * 2 * D * Bd)
+    ckw, cvw = torch.zeros(B, G, S, D, device=dev, dtype=bf), torch.zeros(B, G, S, D, device=dev, dtype=bf)
+    bias = torch.randn((H + 2 * G) * D, device=dev)
+    qw, kw_ = torch.ones(H * D, device=dev), torch.ones(G * D, device=dev)
+    ep = 2.0 * N * (2 * H * D + 4 * G * D)
+    row("bias + whole-projection q / k norm + cache write", "projection epilogue",
+        lambda: wa.qk_norm_cache_write(qkv, ckw, cvw, zero, H, G, D, D, 1e-6, q_weight=qw, k_weight=kw_, whole_norm=True,
+                                       bias=bias), nbytes=ep)
+    row("bias + unit-RMS values + cache write", "projection epilogue",
+        lambda: wa.qk_norm_cache_write(qkv, ckw, cvw, zero, H, G, D, D, 1e-6, normalize=False, bias=bias, value_norm=True),
+        nbytes=ep)
+    row("per-head unit q / k norm + cache write (the like kernel)", "projection epilogue",
+        lambda: wa.qk_norm_cache_write(qkv, ckw, cvw, zero, H, G, D, D, 1e-6), nbytes=ep)
+    del qkv, q, ck, cv, ckw, cvw
+    # latent layers
+    Dl, Dv, R, Rot, Q = s["lat_dim"], s["lat_vdim"], s["rank"], s["lat_rot"], 2 * s["rank"]
+    ql = torch.randn(B, T, H, Dl, device=dev, dtype=bf)
+    kv = torch.randn(B, T, H * (Dl + Dv), device=dev, dtype=bf)
+    gate = torch.randn(B, T, H, device=dev, dtype=bf)
+    kx, vx = kv[..., : H * Dl].unflatten(-1, (H, Dl)).permute(0, 2, 1, 3), kv[..., H * Dl:].unflatten(-1, (H, Dv)).permute(0, 2, 1, 3)
+    fl = 2.0 * (Dl + Dv) * pairs * H * B
+    row("latent prefill, expanded heads, tcgen05, output gate inside", "prefill attention",
+        lambda: wa.window_attention_tc(ql.permute(0, 2, 1, 3), kx, vx, 0.07, win, gate=gate), flops=fl)
+    row("latent prefill, expanded heads, mma.sync (portions), output gate inside", "prefill attention",
+        lambda: wa.window_attention_prefill(ql, kx, vx, zero, 0.07, win, gate=gate), flops=fl)
+    qr = torch.randn(B, T, H, Dl + Rot, device=dev, dtype=bf)
+    kr = torch.randn(B, T, H, Dl + Rot, device=dev, dtype=bf).permute(0, 2, 1, 3)
+    row("latent prefill of the closest family, window added (the like kernel)", "prefill attention",
+        lambda: wa.window_attention_prefill(qr, kr, vx, zero, 0.07, win, sinks=one), flops=2.0 * (Dl + Rot + Dv) * pairs * H * B)
+    del qr, kr, kv, ql
+    cl = torch.randn(Bd, 1, S, R, device=dev, dtype=bf)
+    qa, gd = torch.randn(Bd, H, R, device=dev, dtype=bf), torch.randn(Bd, H, device=dev, dtype=bf)
+    row("latent decode in the window (absorbed queries, output gate)", "decode attention",
+        lambda: wa.window_attention_decode(qa, cl, cl, posd, 0.07, win, gate=gd), nbytes=2.0 * win * R * Bd)
+    cr = torch.randn(Bd, 1, S, R + Rot, device=dev, dtype=bf)
+    qb = torch.randn(Bd, H, R + Rot, device=dev, dtype=bf)
+    posw = torch.full((Bd,), win - 1, dtype=torch.int32, device=dev)
+    row("latent decode of the closest family over as many rows (the like kernel)", "decode attention",
+        lambda: wa.window_attention_decode(qb, cr, cr[..., :R], posw, 0.07, sinks=one), nbytes=2.0 * win * (R + Rot) * Bd)
+    proj = torch.randn(B, T, Q + R + (H + 7) // 8 * 8, device=dev, dtype=bf)
+    wq, wc = torch.ones(Q, device=dev), torch.ones(R, device=dev)
+    row("both latent norms + cache row", "projection epilogue",
+        lambda: la.latent_norms(proj, 0, Q, Q, R, cl, wq, wc, zero, 1e-6, rows=True), nbytes=2.0 * N * (2 * Q + 3 * R))
+    pr = torch.randn(B, T, H * (Dl + Rot) + R + Rot, device=dev, dtype=bf)
+    tables = rope_ops.build_interleaved_rope_cache(S, Rot, 1e6, device=dev)
+    row("latent norm + rotations + cache row (the like kernel)", "projection epilogue",
+        lambda: la.latent_prep(pr, 0, H * (Dl + Rot), None, cr, wc, tables, zero, H, Dl, Rot, R, 1e-6),
+        nbytes=2.0 * N * (2 * H * (Dl + Rot) + 2 * (R + Rot)))
+    del cl, cr, proj, pr
+    # the stream
+    x32, y = torch.randn(N, W, device=dev), torch.randn(N, W, device=dev, dtype=bf)
+    w1, w2, b1 = torch.ones(W, device=dev), torch.ones(W, device=dev), torch.zeros(W, device=dev)
+    row("residual add with output bias + next norm", "norm", lambda: sn.residual_norm_(x32, y, b1, w1, 1e-6, bf),
+        nbytes=float(N * W * (4 + 4 + 2 + 2)))
+    row("post-norm + residual + next norm (the like kernel)", "norm", lambda: norm_ops.norm_chain_(x32, y, w1, w2, 1e-6, bf),
+        nbytes=float(N * W * (4 + 4 + 2 + 2)))
+    table = torch.randn(VOCAB, W, device=dev, dtype=bf)
+    ids = torch.randint(0, VOCAB, (B, T), device=dev)
+    pos = torch.arange(T, device=dev).expand(B, T).contiguous()
+    freq = sn.position_frequencies(W, device=dev)
+    row("embedding + position vector + entry norm + first norm", "norm",
+        lambda: sn.embed_norm(table, ids, pos, freq, w1, 1e-6, w2, bf), nbytes=float(N * W * (2 + 4 + 2)))
+    F = (2 * s["ff"] // 3 + 127) // 128 * 128
+    src = torch.randn(N, 2 * F, device=dev, dtype=bf)
+    row("silu(gate) * up from the fused projection", "activation", lambda: moe_sparse.glu_bias(src, 0, F, F), nbytes=2.0 * N * 3 * F)
+    row("SwiGLU of the Llama decoder (the like kernel)", "activation", lambda: act_ops.swiglu(src), nbytes=2.0 * N * 3 * F)
+    return rows
+
+
+def run_scored(steps: int = 10, warmup: int = 3, device=None, sizes=None) -> dict:
+    dev = device or torch.device("cuda", torch.cuda.current_device())
+    before = _lib.kernel_launches()
+    out = {"metric": "Tidavik vs Rasodra (attention layers), serving throughput at equal layer sizes", "dtype": "bf16",
+           "data": "synthetic token ids, random-init weights", "steps": steps, "warmup": max(warmup, 3),
+           "l2": "192 MB written between timed runs", "peaks": peaks(), "cases": [], "kernels": {}}
+    for s in (sizes or HYBRID_SIZES):
+        out["cases"].append(scored_serve_case(s, steps, warmup, dev))
+        out["kernels"][s["name"]] = scored_kernel_cases(s, steps, warmup, dev)
+    out["gpu_launches"] = _lib.kernel_launches() - before
+    return out
