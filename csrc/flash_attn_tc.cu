@@ -128,12 +128,16 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
     if (warp == 1) ptx::tmem_alloc<1>(tmem_ptr_smem, L::kTmemCols);
     float* dtab = reinterpret_cast<float*>(sP);          // bias table (SCORE): the P staging area is free, P lives in TMEM
     constexpr float kL2e = score::kLog2e;                // r1 ln(.) in log2 units is r1 log2(.)
+    constexpr float kSign = SCORE == 2 ? -1.f : 1.f;     // sigmoid weights are computed from the negative score
     const float r1 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r1[hq] : 0.f;
     const float r2 = (SCORE > 0 && p.mod.r1 != nullptr) ? p.mod.r2[hq] : 0.f;
+    const float bias_slope = (SCORE > 0 && p.slopes != nullptr) ? p.slopes[hq] * kL2e : 0.f;
+    const float bias_const = SCORE == 2 ? -p.mod.pb[hq] * kL2e : 0.f;
+    // what a score at that distance gains, with the sign of kSign (and the sigmoid's offset)
+    auto bias_at = [&](float dist) { return fmaf(-kSign, r1 * __log2f(fmaf(r2, dist, 1.f)) + bias_slope * dist, bias_const); };
     if (SCORE > 0 && p.bias_entries > 0) {
-        const float sl = p.slopes != nullptr ? p.slopes[hq] * kL2e : 0.f;
         const int n = min(p.bias_entries, m0 + kBM + offset);
-        for (int i = threadIdx.x; i < n; i += kThreadsTc) dtab[i] = r1 * __log2f(fmaf(r2, (float)i, 1.f)) + sl * (float)i;
+        for (int i = threadIdx.x; i < n; i += kThreadsTc) dtab[i] = bias_at((float)i);
     }
     ptx::tcgen05_fence_before();
     __syncthreads();
@@ -230,8 +234,12 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
         float m_run = -INFINITY, l_run = 0.f;
         const float sc = WIN ? 1.f : p.scale_log2;                   // WIN: scores are converted to log2 units up front
         const float cap_in = (SCORE > 0 && p.mod.cap > 0.f) ? p.scale_log2 / (kL2e * p.mod.cap) : 0.f;
-        const float cap_out = p.mod.cap * kL2e;
-        const float pb2 = SCORE == 2 ? p.mod.pb[hq] * kL2e : 0.f;
+        const float cap_out = kSign * p.mod.cap * kL2e;
+        // capped score = s P(s^2): the tanh series with the scales inside (no cap: P is the constant scale)
+        const float ci2 = cap_in * cap_in, s_limit = cap_in > 0.f ? score::kSeriesLimit / cap_in : INFINITY;
+        const float q0 = kSign * p.scale_log2, q1 = -q0 * ci2 / 3.f, q2 = q0 * ci2 * ci2 * (2.f / 15.f);
+        const float q3 = -q0 * ci2 * ci2 * ci2 * (17.f / 315.f), q4 = q0 * ci2 * ci2 * ci2 * ci2 * (62.f / 2835.f);
+        const uint64_t k0 = f2_pack(q0, q0), k1 = f2_pack(q1, q1), k2 = f2_pack(q2, q2), k3 = f2_pack(q3, q3), k4 = f2_pack(q4, q4);
         const float slope2 = (WIN && p.slopes != nullptr) ? p.slopes[hq] * 1.4426950408889634f : 0.f;
         // one tile of the online softmax; MASK is instantiated only for tiles on the causal diagonal / past Sk
         auto tile_softmax = [&](auto mask_tag, int j) {
@@ -244,43 +252,51 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
             ptx::mbar_arrive(s_empty);
             const int n0 = tile(j) * kBN;
             if (SCORE > 0) {
-                if (cap_in > 0.f) {
-                    float am0 = 0.f, am1 = 0.f;
-#pragma unroll
-                    for (int c = 0; c < kBN; c += 2) {
-                        am0 = fmaxf(am0, fabsf(__uint_as_float(sr[c])));
-                        am1 = fmaxf(am1, fabsf(__uint_as_float(sr[c + 1])));
-                    }
-                    if (__any_sync(0xffffffffu, fmaxf(am0, am1) * cap_in >= score::kSeriesLimit)) {
-#pragma unroll
-                        for (int c = 0; c < kBN; ++c)
-                            sr[c] = __float_as_uint(cap_out * score::tanh_exp(__uint_as_float(sr[c]) * cap_in));
-                    } else {
-#pragma unroll
-                        for (int c = 0; c < kBN; ++c)
-                            sr[c] = __float_as_uint(cap_out * score::tanh_series(__uint_as_float(sr[c]) * cap_in));
-                    }
-                } else {
-#pragma unroll
-                    for (int c = 0; c < kBN; ++c) sr[c] = __float_as_uint(__uint_as_float(sr[c]) * p.scale_log2);
-                }
+                // sr <- score in log2 units (SCORE 2: its negative), two columns per packed instruction: the capped score is
+                // s * P(s^2) with the cap's scales inside P, the bias joins in the last multiply-add
                 const int d0 = grow + offset - n0;                          // distance of column 0
-                if (p.bias_entries > 0) {
-                    if (MASK) {
+                float am0 = 0.f, am1 = 0.f;
 #pragma unroll
-                        for (int c = 0; c < kBN; ++c)
-                            sr[c] = __float_as_uint(__uint_as_float(sr[c]) - dtab[min(max(d0 - c, 0), p.bias_entries - 1)]);
+                for (int c = 0; c < kBN; c += 2) {
+                    am0 = fmaxf(am0, fabsf(__uint_as_float(sr[c])));
+                    am1 = fmaxf(am1, fabsf(__uint_as_float(sr[c + 1])));
+                }
+                const bool series = !__any_sync(0xffffffffu, fmaxf(am0, am1) >= s_limit);
+                auto cap_and_bias = [&](auto bias) {                        // bias(c): what columns c, c + 1 gain
+                    if (series) {
+#pragma unroll
+                        for (int c = 0; c < kBN; c += 2) {
+                            const uint64_t s2 = f2_pack(__uint_as_float(sr[c]), __uint_as_float(sr[c + 1]));
+                            const uint64_t z = f2_mul(s2, s2);
+                            uint64_t h = f2_fma(z, k4, k3);
+                            h = f2_fma(z, h, k2);
+                            h = f2_fma(z, h, k1);
+                            h = f2_fma(z, h, k0);
+                            h = f2_fma(s2, h, bias(c));
+                            sr[c] = (uint32_t)h;
+                            sr[c + 1] = (uint32_t)(h >> 32);
+                        }
                     } else {
-                        const float* tb = dtab + d0;
 #pragma unroll
-                        for (int c = 0; c < kBN; ++c) sr[c] = __float_as_uint(__uint_as_float(sr[c]) - tb[-c]);
+                        for (int c = 0; c < kBN; c += 2) {
+                            const uint64_t t = bias(c);
+                            sr[c] = __float_as_uint(fmaf(cap_out, score::tanh_exp(__uint_as_float(sr[c]) * cap_in), f2_lo(t)));
+                            sr[c + 1] = __float_as_uint(fmaf(cap_out, score::tanh_exp(__uint_as_float(sr[c + 1]) * cap_in), f2_hi(t)));
+                        }
                     }
+                };
+                if (p.bias_entries > 0) {
+                    const float* tb = dtab + d0;
+                    if (MASK)
+                        cap_and_bias([&](int c) { return f2_pack(dtab[min(max(d0 - c, 0), p.bias_entries - 1)],
+                                                                 dtab[min(max(d0 - c - 1, 0), p.bias_entries - 1)]); });
+                    else
+                        cap_and_bias([&](int c) { return f2_pack(tb[-c], tb[-c - 1]); });
                 } else if (p.bias_entries < 0) {
-#pragma unroll
-                    for (int c = 0; c < kBN; ++c) {
-                        const float dist = (float)max(d0 - c, 0);
-                        sr[c] = __float_as_uint(__uint_as_float(sr[c]) - r1 * __log2f(fmaf(r2, dist, 1.f)) - slope2 * dist);
-                    }
+                    cap_and_bias([&](int c) { return f2_pack(bias_at((float)max(d0 - c, 0)), bias_at((float)max(d0 - c - 1, 0))); });
+                } else {
+                    const uint64_t t = f2_pack(bias_const, bias_const);
+                    cap_and_bias([&](int) { return t; });
                 }
             } else if (WIN) {
                 // log2 units: s * scale - slope * (query position - key position)
@@ -298,20 +314,20 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
                 const int kept = WIN ? p.keep_first - n0 : 0;
 #pragma unroll
                 for (int c = 0; c < kBN; ++c)
-                    if (c >= first_bad || (WIN && c < first_good && c >= kept)) sr[c] = 0xff800000u;   // -inf
+                    if (c >= first_bad || (WIN && c < first_good && c >= kept)) sr[c] = SCORE == 2 ? 0x7f800000u : 0xff800000u;   // -inf
             }
             uint32_t pk[kBN / 2];
             if constexpr (SCORE == 2) {
-                // sigmoid(x) = 1 / (1 + 2^-x2); one reciprocal serves two weights (the clamp keeps the product finite)
+                // sigmoid(x) = 1 / (1 + 2^-x2), sr = -x2; one reciprocal serves two weights (the clamp keeps the product finite)
 #pragma unroll
                 for (int c = 0; c < kBN; c += 2) {
-                    const float x0 = __uint_as_float(sr[c]) + pb2, x1 = __uint_as_float(sr[c + 1]) + pb2;
-                    const float a = 1.f + ex2_approx(fminf(-x0, 60.f)), bq = 1.f + ex2_approx(fminf(-x1, 60.f));
-                    const float r = __fdividef(1.f, a * bq);
+                    const float y0 = __uint_as_float(sr[c]), y1 = __uint_as_float(sr[c + 1]);
+                    const float a = 1.f + ex2_approx(fminf(y0, 60.f)), bq = 1.f + ex2_approx(fminf(y1, 60.f));
+                    const float r = rcp_approx(a * bq);
                     float p0 = r * bq, p1 = r * a;
                     if (MASK) {
-                        if (x0 == -INFINITY) p0 = 0.f;
-                        if (x1 == -INFINITY) p1 = 0.f;
+                        if (y0 == INFINITY) p0 = 0.f;
+                        if (y1 == INFINITY) p1 = 0.f;
                     }
                     pk[c >> 1] = pack_bf16x2(p0, p1);
                 }
