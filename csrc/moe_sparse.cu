@@ -7,8 +7,10 @@
 //                 renormalise: the `top` largest LOGITS are taken and the weights are the softmax over the chosen
 //                 logits only (times out_scale)
 //                 sigmoid scores (mode 2): s = sigmoid(z) per expert instead of the softmax, otherwise as the first form
+//                 normalised scores (mode 3): the first form with the chosen s divided by their sum (+ 1e-20)
 //   activation    g = min(gate, limit), u = clamp(up, -limit, limit);  a = g * sigmoid(alpha * g) * (u + up_shift)
 //                 (limit = +inf, alpha = 1, up_shift = 0: plain silu(gate) * up)
+//                 experts without a gate: a = max(up, 0)^2
 //   expert index >= E means an identity expert: its output is the token's input itself
 // Expert weights are stored [E, in, out] (the layout of the grouped expert layers), gate | up fused on the out dim.
 #include "common.cuh"
@@ -125,10 +127,16 @@ moe_router_kernel(const T* __restrict__ h, const float* __restrict__ wr, const f
         if (bi >= R) bi = 0;      // every score NaN: keep the index in range
         if (lane == 0) {
             idx[n * top + k] = bi;
-            wts[n * top + k] = renorm ? ps[bi] : ps[bi] * out_scale;
+            wts[n * top + k] = (renorm || mode == 3) ? ps[bi] : ps[bi] * out_scale;
             cs[bi] = -INFINITY;
         }
         __syncwarp();
+    }
+    if (mode == 3 && lane == 0) {
+        float sum = 1e-20f;
+        for (int k = 0; k < top; ++k) sum += wts[n * top + k];
+        const float inv = out_scale / sum;
+        for (int k = 0; k < top; ++k) wts[n * top + k] *= inv;
     }
     if (renorm && lane == 0) {   // softmax over the chosen logits only; the first pick is the largest
         const float mx = wts[n * top];
@@ -205,6 +213,56 @@ moe_gate_up_act_kernel(const T* __restrict__ h, const T* __restrict__ wgu, const
                 u += red[((long long)w * COLS + threadIdx.x) * 2 + 1];
             }
             stf(act + p * F + f, glu_act(g, u, limit, alpha, up_shift));
+        }
+    }
+}
+
+// the same for experts without a gate: act = max(h @ wu, 0)^2, wu [E, W, F]
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(GV_WARPS * 32)
+moe_up_relu2_kernel(const T* __restrict__ h, const T* __restrict__ wu, const int* __restrict__ idx, T* __restrict__ act,
+                    int pairs_per_token, int W, int F, int E) {
+    extern __shared__ float smem[];
+    constexpr int PER = VEC ? 2 : 1, COLS = 32 * PER;
+    float* hs = smem;                                  // [W]
+    float* red = smem + W;                             // [GV_WARPS][COLS]
+    const long long p = blockIdx.x;
+    const int e = idx != nullptr ? idx[p] : 0;
+    if (e < 0 || e >= E) return;                       // identity expert: no intermediate
+    const long long t = p / pairs_per_token;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    for (int c = threadIdx.x; c < W; c += GV_WARPS * 32) hs[c] = ldf(h + t * W + c);
+    __syncthreads();
+    const int f0 = blockIdx.y * COLS + lane * PER;
+    const int per = (W + GV_WARPS - 1) / GV_WARPS;
+    const int k_lo = warp * per, k_hi = min(W, k_lo + per);
+    float u0 = 0.f, u1 = 0.f;
+    if (f0 < F) {
+        const T* base = wu + (long long)e * W * F + f0;
+#pragma unroll 8
+        for (int k = k_lo; k < k_hi; ++k) {
+            const float hv = hs[k];
+            if (VEC) {
+                float a, b;
+                ld2(base + (long long)k * F, a, b);
+                u0 = fmaf(hv, a, u0);
+                u1 = fmaf(hv, b, u1);
+            } else {
+                u0 = fmaf(hv, ldf(base + (long long)k * F), u0);
+            }
+        }
+    }
+    red[warp * COLS + lane * PER] = u0;
+    if (VEC) red[warp * COLS + lane * PER + 1] = u1;
+    __syncthreads();
+    if (threadIdx.x < COLS) {
+        const int f = blockIdx.y * COLS + threadIdx.x;
+        if (f < F) {
+            float u = 0.f;
+#pragma unroll
+            for (int w = 0; w < GV_WARPS; ++w) u += red[w * COLS + threadIdx.x];
+            u = fmaxf(u, 0.f);
+            stf(act + p * F + f, u * u);
         }
     }
 }
@@ -366,7 +424,7 @@ __global__ void moe_gather_combine_kernel(const T* __restrict__ ys, const int* _
 
 // dtype: 0 bf16, 1 fp32 (activations and expert weights).  R = router outputs (experts + identity experts).
 // zbias [R] fp32 or NULL: added to the logits; mode 0: softmax scores; 1: choice on the logits, weights = softmax over the
-// chosen ones; 2: sigmoid scores.
+// chosen ones; 2: sigmoid scores; 3: softmax scores, the chosen ones divided by their sum.
 NXD_API int nxd_moe_router(int dtype, const void* h, const float* wr, const float* corr, const float* wsg, int* idx,
                            float* wts, float* sgate, long long N, int W, int R, int top, float out_scale,
                            const float* zbias, int mode, void* stream) {
@@ -415,6 +473,34 @@ NXD_API int nxd_moe_gate_up_act(int dtype, const void* h, const void* wgu, const
         if (vec) NXD_GU(float, true); else NXD_GU(float, false);
     }
 #undef NXD_GU
+    NXD_LAUNCH_CHECK();
+    return 0;
+}
+
+// act[p, :] = max(h[p / pairs_per_token] @ wu[idx[p]], 0)^2; wu [E, W, F]; idx as in nxd_moe_gate_up_act.
+NXD_API int nxd_moe_up_relu2(int dtype, const void* h, const void* wu, const int* idx, void* act, long long P,
+                             int pairs_per_token, int W, int F, int E, void* stream) {
+    if (P == 0) return 0;
+    NXD_REQUIRE(P < (1ll << 31), "up: %lld pairs", P);
+    const bool vec = (F % 2) == 0;
+    const int cols = vec ? 64 : 32;
+    const size_t smem = (size_t)(W + GV_WARPS * cols) * sizeof(float);
+    NXD_REQUIRE(smem <= 200 * 1024, "up: input width %d", W);
+    dim3 grid((unsigned)P, (F + cols - 1) / cols);
+    cudaStream_t st = (cudaStream_t)stream;
+#define NXD_UP(T, V)                                                                                                  \
+    do {                                                                                                              \
+        auto kern = moe_up_relu2_kernel<T, V>;                                                                        \
+        if (smem > 48 * 1024)                                                                                         \
+            NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));       \
+        kern<<<grid, GV_WARPS * 32, smem, st>>>((const T*)h, (const T*)wu, idx, (T*)act, pairs_per_token, W, F, E);   \
+    } while (0)
+    if (dtype == 0) {
+        if (vec) NXD_UP(bf16, true); else NXD_UP(bf16, false);
+    } else {
+        if (vec) NXD_UP(float, true); else NXD_UP(float, false);
+    }
+#undef NXD_UP
     NXD_LAUNCH_CHECK();
     return 0;
 }

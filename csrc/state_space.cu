@@ -1,0 +1,1059 @@
+// State-space mixers: recurrences whose state lives in fp32 device memory, one per cache line, decayed by step sizes that
+// the tokens themselves choose.
+//
+//   selective scan (one decay per channel and state)                              S [channels, N] per line
+//       S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n;    y_c = sum_n S[c, n] C_n + D_c x_c;    out = y silu(z)
+//   state-space heads (one decay per head; B and C shared by the heads of a group) S [heads, N, P] per line
+//       S <- exp(-exp(A_log) dt) S + dt B x^T;                  y = S^T C + D x
+//
+// dt = softplus(pre-activation + bias).  x (and B, C of the second kind) come out of a short causal convolution per channel
+// with a bias and silu.  A row that starts at position 0 starts from zeros, any other row continues from its line's state;
+// padding tokens (t >= n_new[b]) change nothing and come out as zeros.
+//
+// Kernels:
+//   conv_silu          convolution + silu of a column range of a projection; also moves the line's convolution state (the
+//                      last taps - 1 raw inputs) when one thread sees the whole step, else conv_state does it afterwards
+//   selective_scan     states of a channel split over R lanes of NS registers, tokens in double-buffered blocks of 16 through
+//                      shared memory (cp.async); the R partial sums of R consecutive tokens are summed by one transposing
+//                      butterfly; gate, skip term and store once per block.  Prompts and single tokens
+//   ssd_step           one token: a thread owns four neighbouring columns of a head's state, the rows are spread over the
+//                      CTA; the state is read and written once
+//   ssd_scan           token by token, a column's rows split over R lanes (fp32 prompts, short steps, unusual sizes)
+//   ssd_chunk          bf16 prompts in chunks of 64 tokens on mma.sync, one CTA walks the chunks of 64 (or 32) columns of a
+//                      head with the fp32 state in accumulator registers.  Operands that are products of fp32 numbers (decayed
+//                      scores, scaled inputs, the state) go in as the sum of two bf16 numbers, so that their relative error
+//                      is 2^-17, not 2^-9
+//   gate_norm          y act(z) [* constant], or divided by the root mean square over equal groups of columns and weighted
+// This file is compiled without fast-math: the state lives for thousands of steps.
+#include "common.cuh"
+#include "mma_sync.cuh"
+
+namespace {
+
+__device__ __forceinline__ float ldf(const float* p) { return *p; }
+__device__ __forceinline__ float ldf(const bf16* p) { return __bfloat162float(*p); }
+__device__ __forceinline__ void stf(float* p, float v) { *p = v; }
+__device__ __forceinline__ void stf(bf16* p, float v) { *p = __float2bfloat16_rn(v); }
+__device__ __forceinline__ float silu_f(float z) { return z / (1.f + expf(-z)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return 1.f / (1.f + expf(-z)); }
+__device__ __forceinline__ float softplus_f(float z) { return z > 20.f ? z : log1pf(expf(z)); }
+// 2^x; arguments here are never positive, results below 2^-126 become zero
+__device__ __forceinline__ float exp2_ftz(float x) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+    return r;
+}
+constexpr float LOG2E = 1.4426950408889634f;
+
+template <int VEC>
+__device__ __forceinline__ void ldv(const float* p, float* v) {
+    if (VEC == 4) {
+        const float4 t = *reinterpret_cast<const float4*>(p);
+        v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w;
+    } else {
+        v[0] = *p;
+    }
+}
+template <int VEC>
+__device__ __forceinline__ void ldv(const bf16* p, float* v) {
+    if (VEC == 4) {
+        const uint2 raw = *reinterpret_cast<const uint2*>(p);
+        const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&raw.x));
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&raw.y));
+        v[0] = a.x, v[1] = a.y, v[2] = b.x, v[3] = b.y;
+    } else {
+        v[0] = __bfloat162float(*p);
+    }
+}
+template <int VEC>
+__device__ __forceinline__ void stv(float* p, const float* v) {
+    if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    else *p = v[0];
+}
+template <int VEC>
+__device__ __forceinline__ void stv(bf16* p, const float* v) {
+    if (VEC == 4) {
+        uint2 raw;
+        *reinterpret_cast<bf162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
+        *reinterpret_cast<bf162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
+        *reinterpret_cast<uint2*>(p) = raw;
+    } else {
+        *p = __float2bfloat16_rn(v[0]);
+    }
+}
+
+// ---- short convolution ----------------------------------------------------------------------------------------------------
+// VEC raw inputs (channels c ..) at step index s, which may lie before the step: then they come from the line's state (slot
+// K + s holds position p0 + s), zeros before the start of the sequence
+template <typename T, int VEC>
+__device__ __forceinline__ void conv_input(const T* __restrict__ row0, long long ld, const float* __restrict__ st, int s, int p0,
+                                           int K, int C, int c, float* v) {
+    if (s >= 0) {
+        ldv<VEC>(row0 + (long long)s * ld + c, v);
+    } else if (p0 + s < 0) {
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) v[i] = 0.f;
+    } else {
+        ldv<VEC>(st + (long long)(K + s) * C + c, v);
+    }
+}
+
+// slot s of the line's state <- raw input of position (p0 + n) - K + s.  Slots are written upwards and read from at or above
+// the slot being written (n >= 1), so one thread can do it in place.
+template <typename T, int VEC>
+__device__ __forceinline__ void move_conv_state(const T* __restrict__ row0, long long ld, float* __restrict__ st, int n, int p0,
+                                                int K, int C, int c) {
+    for (int s = 0; s < K; ++s) {
+        float v[VEC];
+        conv_input<T, VEC>(row0, ld, st, n - K + s, p0, K, C, c, v);
+        stv<VEC>(st + (long long)s * C + c, v);
+    }
+}
+
+// TAPS: compile-time number of taps (inputs slide through registers), or 0 (inputs are read again per tap)
+template <typename T, typename TO, int VEC, int TAPS>
+__global__ void __launch_bounds__(128)
+conv_silu_kernel(const T* __restrict__ proj, long long ld, const float* __restrict__ conv_w, const float* __restrict__ bias,
+                 float* __restrict__ conv_state, TO* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
+                 const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int C, int taps, int TT, int move) {
+    const int c = (blockIdx.x * 128 + threadIdx.x) * VEC;
+    if (c >= C) return;
+    const int b = blockIdx.z, t0 = blockIdx.y * TT, t1 = min(t0 + TT, Tn);
+    const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+    const int p0 = q_start[b];
+    const int K = (TAPS > 0 ? TAPS : taps) - 1;
+    float* st = conv_state + (long long)line * K * C;
+    const T* row0 = proj + (long long)b * Tn * ld;
+    TO* orow = out + (long long)b * Tn * ld_out + c;
+    float bv[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) bv[i] = bias != nullptr ? bias[c + i] : 0.f;
+    const int te = min(t1, n);
+    if (TAPS > 0) {
+        constexpr int NT = TAPS > 0 ? TAPS : 1;
+        float w[NT][VEC], win[NT][VEC];
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) w[j][i] = conv_w[(long long)(c + i) * NT + j];
+        if (t0 < te) {
+#pragma unroll
+            for (int j = 0; j + 1 < NT; ++j) conv_input<T, VEC>(row0, ld, st, t0 - (NT - 1) + j, p0, K, C, c, win[j + 1]);
+        }
+#pragma unroll 4
+        for (int t = t0; t < te; ++t) {
+            float acc[VEC];
+#pragma unroll
+            for (int j = 0; j + 1 < NT; ++j)
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) win[j][i] = win[j + 1][i];
+            ldv<VEC>(row0 + (long long)t * ld + c, win[NT - 1]);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) {
+                acc[i] = bv[i];
+#pragma unroll
+                for (int j = 0; j < NT; ++j) acc[i] = fmaf(w[j][i], win[j][i], acc[i]);
+                acc[i] = silu_f(acc[i]);
+            }
+            stv<VEC>(orow + (long long)t * ld_out, acc);
+        }
+    } else {
+        for (int t = t0; t < te; ++t) {
+            float acc[VEC], v[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) acc[i] = bv[i];
+            for (int j = 0; j <= K; ++j) {
+                conv_input<T, VEC>(row0, ld, st, t - K + j, p0, K, C, c, v);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) acc[i] = fmaf(conv_w[(long long)(c + i) * (K + 1) + j], v[i], acc[i]);
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) acc[i] = silu_f(acc[i]);
+            stv<VEC>(orow + (long long)t * ld_out, acc);
+        }
+    }
+    float zero[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) zero[i] = 0.f;
+    for (int t = max(t0, n); t < t1; ++t) stv<VEC>(orow + (long long)t * ld_out, zero);
+    if (move && n > 0) move_conv_state<T, VEC>(row0, ld, st, n, p0, K, C, c);
+}
+
+template <typename T>
+__global__ void conv_state_kernel(const T* __restrict__ proj, long long ld, float* __restrict__ conv_state,
+                                  const int* __restrict__ q_start, const int* __restrict__ n_new,
+                                  const int* __restrict__ seq_ids, int Tn, int C, int taps) {
+    const int c = blockIdx.x * blockDim.x + threadIdx.x, b = blockIdx.y;
+    if (c >= C) return;
+    const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
+    if (n <= 0) return;
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+    move_conv_state<T, 1>(proj + (long long)b * Tn * ld, ld, conv_state + (long long)line * (taps - 1) * C, n, q_start[b],
+                          taps - 1, C, c);
+}
+
+// ---- selective scan --------------------------------------------------------------------------------------------------------
+// v[j] of lane r (r = its place among R neighbouring lanes) -> the sum over the R lanes of v[r], R - 1 shuffles in all
+template <int R>
+__device__ __forceinline__ float transpose_sum(float (&v)[R], int r) {
+#pragma unroll
+    for (int o = 1; o < R; o <<= 1) {
+        const bool up = (r & o) != 0;
+#pragma unroll
+        for (int j = 0; j < R; j += 2 * o) {
+            const float keep = up ? v[j + o] : v[j], give = up ? v[j] : v[j + o];
+            v[j] = keep + __shfl_xor_sync(0xffffffffu, give, o);
+        }
+    }
+    return v[0];
+}
+
+constexpr int SS_THREADS = 128, SS_TS = 16;
+
+template <typename T, int NS, int R>
+__global__ void __launch_bounds__(SS_THREADS)
+selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __restrict__ dt, long long ld_dt,
+                      const float* __restrict__ dt_bias, const float* __restrict__ bc, long long ld_bc, int b_off, int c_off,
+                      const T* __restrict__ z, long long ld_z, const float* __restrict__ a_log, const float* __restrict__ dskip,
+                      float* __restrict__ S, T* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
+                      const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int C, int N, int async) {
+    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS > R ? SS_TS : R;
+    struct Buf {
+        float B[TS][NP], Cm[TS][NP], dt[TS][CH];
+        T x[TS][CH], z[TS][CH];
+    };
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    Buf* bufs = reinterpret_cast<Buf*>(smem_raw);
+    float(*us)[CH] = reinterpret_cast<float(*)[CH]>(smem_raw + 2 * sizeof(Buf));           // dt * x
+    float(*ys)[CH] = us + TS;                                                                // sum_n S C
+    const int tid = threadIdx.x, r = tid % R, cl = tid / R;
+    const int c0 = blockIdx.x * CH, c = c0 + cl, b = blockIdx.y;
+    const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
+    const long long row0 = (long long)b * Tn;
+    const int nch = min(CH, C - c0);
+    for (int idx = tid; idx < (Tn - max(n, 0)) * nch; idx += SS_THREADS)                     // padding rows
+        stf(out + (row0 + max(n, 0) + idx / nch) * ld_out + c0 + idx % nch, 0.f);
+    if (n <= 0) return;
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+    float* Sc = S + ((long long)line * C + c) * N;
+    const bool fresh = q_start[b] == 0;
+    float s[NS], a2[NS];
+#pragma unroll
+    for (int j = 0; j < NS; ++j) {
+        const int i = r * NS + j;
+        const bool ok = c < C && i < N;
+        s[j] = (ok && !fresh) ? Sc[i] : 0.f;
+        a2[j] = ok ? -expf(a_log[(long long)c * N + i]) * LOG2E : 0.f;
+    }
+    // columns N .. NP - 1 of B and C are zeros in both buffers and stay so
+    if (N < NP)
+        for (int idx = tid; idx < 2 * TS * (NP - N); idx += SS_THREADS) {
+            const int k = idx / (TS * (NP - N)), q = idx % (TS * (NP - N));
+            bufs[k].B[q / (NP - N)][N + q % (NP - N)] = 0.f;
+            bufs[k].Cm[q / (NP - N)][N + q % (NP - N)] = 0.f;
+        }
+    constexpr int XV = 16 / sizeof(T);                       // elements of T per 16 bytes
+    constexpr int CX = CH / XV > 0 ? CH / XV : 1;            // such pieces per token (narrower CTAs never copy that way)
+    auto fetch = [&](int t0, int k) {
+        Buf& d = bufs[k];
+        const int cnt = min(TS, n - t0);
+        if (async) {
+            for (int idx = tid; idx < cnt * (N / 4); idx += SS_THREADS) {
+                const int tt = idx / (N / 4), i = (idx % (N / 4)) * 4;
+                const float* src = bc + (row0 + t0 + tt) * ld_bc + i;
+                mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.B[tt][i]), src + b_off, true);
+                mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.Cm[tt][i]), src + c_off, true);
+            }
+            for (int idx = tid; idx < cnt * (CH / 4); idx += SS_THREADS) {
+                const int tt = idx / (CH / 4), i = (idx % (CH / 4)) * 4;
+                const bool ok = i < nch;
+                mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.dt[tt][i]), dt + (row0 + t0 + tt) * ld_dt + c0 + (ok ? i : 0), ok);
+            }
+            for (int idx = tid; idx < cnt * CX; idx += SS_THREADS) {
+                const int tt = idx / CX, i = (idx % CX) * XV;
+                const bool ok = i < nch;
+                const long long at = row0 + t0 + tt;
+                mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.x[tt][i]), x + at * ld_x + c0 + (ok ? i : 0), ok);
+                mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.z[tt][i]), z + at * ld_z + c0 + (ok ? i : 0), ok);
+            }
+        } else {
+            for (int idx = tid; idx < cnt * N; idx += SS_THREADS) {
+                const int tt = idx / N, i = idx % N;
+                const float* src = bc + (row0 + t0 + tt) * ld_bc + i;
+                d.B[tt][i] = src[b_off];
+                d.Cm[tt][i] = src[c_off];
+            }
+            for (int idx = tid; idx < cnt * CH; idx += SS_THREADS) {
+                const int tt = idx / CH, i = idx % CH;
+                const bool ok = i < nch;
+                const long long at = row0 + t0 + tt;
+                d.dt[tt][i] = ok ? dt[at * ld_dt + c0 + i] : 0.f;
+                stf(&d.x[tt][i], ok ? ldf(x + at * ld_x + c0 + i) : 0.f);
+                stf(&d.z[tt][i], ok ? ldf(z + at * ld_z + c0 + i) : 0.f);
+            }
+        }
+        mma::cp_async_commit();
+    };
+    fetch(0, 0);
+    int k = 0;
+    for (int t0 = 0; t0 < n; t0 += TS, k ^= 1) {
+        const int cnt = min(TS, n - t0);
+        if (t0 + TS < n) {
+            fetch(t0 + TS, k ^ 1);
+            mma::cp_async_wait<1>();
+        } else {
+            mma::cp_async_wait<0>();
+        }
+        __syncthreads();
+        Buf& d = bufs[k];
+        for (int idx = tid; idx < TS * CH; idx += SS_THREADS) {          // step sizes; tokens past the end: no step
+            const int tt = idx / CH, i = idx % CH;
+            float v = 0.f, u = 0.f;
+            if (tt < cnt && i < nch) {
+                v = softplus_f(d.dt[tt][i] + (dt_bias != nullptr ? dt_bias[c0 + i] : 0.f));
+                u = v * ldf(&d.x[tt][i]);
+            }
+            d.dt[tt][i] = v;
+            us[tt][i] = u;
+        }
+        if (cnt < TS)                                                    // rows that no copy has filled
+            for (int idx = tid; idx < (TS - cnt) * N; idx += SS_THREADS) {
+                d.B[cnt + idx / N][idx % N] = 0.f;
+                d.Cm[cnt + idx / N][idx % N] = 0.f;
+            }
+        __syncthreads();
+        for (int g0 = 0; g0 < cnt; g0 += R) {
+            float y[R];
+#pragma unroll
+            for (int q = 0; q < R; ++q) {
+                const float dv = d.dt[g0 + q][cl], u = us[g0 + q][cl];
+                float acc[2] = {0.f, 0.f};
+#pragma unroll
+                for (int j = 0; j < NS; j += 4) {
+                    const float4 bv = *reinterpret_cast<const float4*>(&d.B[g0 + q][r * NS + j]);
+                    const float4 cv = *reinterpret_cast<const float4*>(&d.Cm[g0 + q][r * NS + j]);
+                    s[j] = fmaf(exp2_ftz(dv * a2[j]), s[j], u * bv.x);
+                    s[j + 1] = fmaf(exp2_ftz(dv * a2[j + 1]), s[j + 1], u * bv.y);
+                    s[j + 2] = fmaf(exp2_ftz(dv * a2[j + 2]), s[j + 2], u * bv.z);
+                    s[j + 3] = fmaf(exp2_ftz(dv * a2[j + 3]), s[j + 3], u * bv.w);
+                    acc[0] = fmaf(s[j], cv.x, acc[0]);
+                    acc[1] = fmaf(s[j + 1], cv.y, acc[1]);
+                    acc[0] = fmaf(s[j + 2], cv.z, acc[0]);
+                    acc[1] = fmaf(s[j + 3], cv.w, acc[1]);
+                }
+                y[q] = acc[0] + acc[1];
+            }
+            ys[g0 + r][cl] = transpose_sum<R>(y, r);
+        }
+        __syncthreads();
+        for (int idx = tid; idx < cnt * CH; idx += SS_THREADS) {
+            const int tt = idx / CH, i = idx % CH;
+            if (i < nch) {
+                const float xv = ldf(&d.x[tt][i]);
+                stf(out + (row0 + t0 + tt) * ld_out + c0 + i, (ys[tt][i] + dskip[c0 + i] * xv) * silu_f(ldf(&d.z[tt][i])));
+            }
+        }
+        __syncthreads();                                                 // everyone is done with this buffer, us and ys
+    }
+    if (c < C) {
+#pragma unroll
+        for (int j = 0; j < NS; ++j) {
+            const int i = r * NS + j;
+            if (i < N) Sc[i] = s[j];
+        }
+    }
+}
+
+template <typename T, int NS, int R>
+int launch_selective(const void* x, long long ld_x, const float* dt, long long ld_dt, const float* dt_bias, const float* bc,
+                     long long ld_bc, int b_off, int c_off, const void* z, long long ld_z, const float* a_log,
+                     const float* dskip, float* S, void* out, long long ld_out, const int* q_start, const int* n_new,
+                     const int* seq_ids, int B, int Tn, int C, int N, cudaStream_t st) {
+    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS > R ? SS_TS : R;
+    constexpr size_t smem = 2 * (size_t)TS * (2 * NP * 4 + CH * 4 + 2 * CH * sizeof(T)) + 2 * (size_t)TS * CH * 4;
+    auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+    constexpr int XV = 16 / sizeof(T);
+    const int async = CH % XV == 0 && C % XV == 0 && ld_x % XV == 0 && ld_z % XV == 0 && ld_dt % 4 == 0 && ld_bc % 4 == 0 &&
+                      b_off % 4 == 0 && c_off % 4 == 0 && N % 4 == 0 && al(x) && al(z) && al(dt) && al(bc);
+    auto kern = selective_scan_kernel<T, NS, R>;
+    if (smem > 48 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    dim3 grid((C + CH - 1) / CH, B);
+    kern<<<grid, SS_THREADS, smem, st>>>((const T*)x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, (const T*)z, ld_z, a_log,
+                                         dskip, S, (T*)out, ld_out, q_start, n_new, seq_ids, Tn, C, N, async);
+    NXD_LAUNCH_CHECK();
+    return 0;
+}
+
+// ---- state-space heads: one token ------------------------------------------------------------------------------------------
+// blockIdx.x: slice of 32 columns, y: head, z: row.  A thread owns VEC neighbouring columns and every ROWS-th state row.
+template <typename T, typename TY, int VEC>
+__global__ void __launch_bounds__(128)
+ssd_step_kernel(const T* __restrict__ xbc, long long ld, int x_off, int b_off, int c_off, const float* __restrict__ dt,
+                long long ld_dt, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                const float* __restrict__ dskip, float* __restrict__ S, TY* __restrict__ y, const int* __restrict__ q_start,
+                const int* __restrict__ seq_ids, int H, int G, int N, int P) {
+    constexpr int LC = 32 / VEC, ROWS = 128 / LC;              // lanes per row, rows in flight
+    extern __shared__ float smem[];
+    float* Bs = smem;                                          // [N]
+    float* Cs = Bs + N;                                        // [N]
+    __shared__ float red[ROWS][32];
+    const int tid = threadIdx.x, lc = tid % LC, rg = tid / LC;
+    const int p0 = blockIdx.x * 32 + lc * VEC, h = blockIdx.y, b = blockIdx.z, g = h / (H / G);
+    const T* row = xbc + (long long)b * ld;
+    for (int i = tid; i < N; i += 128) {
+        Bs[i] = ldf(row + b_off + g * N + i);
+        Cs[i] = ldf(row + c_off + g * N + i);
+    }
+    const float step = softplus_f(dt[(long long)b * ld_dt + h] + (dt_bias != nullptr ? dt_bias[h] : 0.f));
+    const float decay = expf(-expf(a_log[h]) * step);
+    const bool fresh = q_start[b] == 0, ok = p0 < P;
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+    float xv[VEC], u[VEC], acc[VEC];
+#pragma unroll
+    for (int i = 0; i < VEC; ++i) {
+        xv[i] = ok ? ldf(row + x_off + (long long)h * P + p0 + i) : 0.f;
+        u[i] = step * xv[i];
+        acc[i] = 0.f;
+    }
+    __syncthreads();
+    float* Sg = S + ((long long)line * H + h) * N * P + p0;
+    if (ok) {
+#pragma unroll 4
+        for (int i = rg; i < N; i += ROWS) {
+            float v[VEC];
+            if (fresh) {
+#pragma unroll
+                for (int q = 0; q < VEC; ++q) v[q] = 0.f;
+            } else {
+                ldv<VEC>(Sg + (long long)i * P, v);
+            }
+            const float bv = Bs[i], cv = Cs[i];
+#pragma unroll
+            for (int q = 0; q < VEC; ++q) {
+                v[q] = fmaf(decay, v[q], u[q] * bv);
+                acc[q] = fmaf(v[q], cv, acc[q]);
+            }
+            stv<VEC>(Sg + (long long)i * P, v);
+        }
+    }
+#pragma unroll
+    for (int q = 0; q < VEC; ++q) red[rg][lc * VEC + q] = acc[q];
+    __syncthreads();
+    if (tid < 32) {
+        const int p = blockIdx.x * 32 + tid;
+        if (p < P) {
+            float o = 0.f;
+#pragma unroll
+            for (int q = 0; q < ROWS; ++q) o += red[q][tid];
+            const float xp = ldf(row + x_off + (long long)h * P + p);
+            stf(y + ((long long)b * H + h) * P + p, fmaf(dskip[h], xp, o));
+        }
+    }
+}
+
+// ---- state-space heads: token by token -------------------------------------------------------------------------------------
+// A thread keeps NPT rows of one state column in registers; the R lanes that share a column sit cpw = 32 / R lanes apart.
+// Slices are padded to NPT + 4 floats in shared memory, so that the R 16-byte reads of a warp fall into different banks.
+template <typename T, typename TY, int NPT>
+__global__ void __launch_bounds__(128)
+ssd_scan_kernel(const T* __restrict__ xbc, long long ld, int x_off, int b_off, int c_off, const float* __restrict__ dt,
+                long long ld_dt, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                const float* __restrict__ dskip, float* __restrict__ S, TY* __restrict__ y, const int* __restrict__ q_start,
+                const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int H, int G, int N, int P, int R) {
+    constexpr int PITCH = NPT + 4, TS = 16;
+    extern __shared__ __align__(16) float smem[];
+    const int DS = R * PITCH, CT = 128 / R, cpw = 32 / R, NP = R * NPT;
+    float* Bs = smem;                        // [TS][DS]
+    float* Cs = Bs + TS * DS;                // [TS][DS]
+    float* xs = Cs + TS * DS;                // [TS][CT]
+    __shared__ float sd[TS], sg[TS];         // step, decay
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, r = lane / cpw, cl = warp * cpw + lane % cpw;
+    const int col0 = blockIdx.x * CT, col = col0 + cl, h = blockIdx.y, b = blockIdx.z, g = h / (H / G);
+    const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
+    const long long row0 = (long long)b * Tn;
+    if (r == 0 && col < P)
+        for (int t = max(n, 0); t < Tn; ++t) stf(y + ((row0 + t) * H + h) * P + col, 0.f);
+    if (n <= 0) return;
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+    float* Sg = S + ((long long)line * H + h) * N * P + col;
+    const bool fresh = q_start[b] == 0;
+    float s[NPT];
+#pragma unroll
+    for (int j = 0; j < NPT; ++j) {
+        const int i = r * NPT + j;
+        s[j] = (!fresh && i < N && col < P) ? Sg[(long long)i * P] : 0.f;
+    }
+    const float a = expf(a_log[h]), dsk = dskip[h];
+    for (int t0 = 0; t0 < n; t0 += TS) {
+        const int cnt = min(TS, n - t0);
+        __syncthreads();
+        for (int idx = tid; idx < cnt * NP; idx += 128) {
+            const int tt = idx / NP, i = idx - tt * NP;
+            const T* row = xbc + (row0 + t0 + tt) * ld;
+            const int at = tt * DS + (i / NPT) * PITCH + (i % NPT);
+            Bs[at] = i < N ? ldf(row + b_off + g * N + i) : 0.f;
+            Cs[at] = i < N ? ldf(row + c_off + g * N + i) : 0.f;
+        }
+        for (int idx = tid; idx < cnt * CT; idx += 128) {
+            const int tt = idx / CT, i = idx - tt * CT;
+            xs[idx] = col0 + i < P ? ldf(xbc + (row0 + t0 + tt) * ld + x_off + (long long)h * P + col0 + i) : 0.f;
+        }
+        if (tid < cnt) {
+            const float step = softplus_f(dt[(row0 + t0 + tid) * ld_dt + h] + (dt_bias != nullptr ? dt_bias[h] : 0.f));
+            sd[tid] = step;
+            sg[tid] = expf(-a * step);
+        }
+        __syncthreads();
+        for (int tt = 0; tt < cnt; ++tt) {
+            const float xv = xs[tt * CT + cl], u = sd[tt] * xv, dec = sg[tt];
+            const float4* b4 = reinterpret_cast<const float4*>(Bs + tt * DS + r * PITCH);
+            const float4* c4 = reinterpret_cast<const float4*>(Cs + tt * DS + r * PITCH);
+            float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+            for (int v = 0; v < NPT / 4; ++v) {
+                const float4 bv = b4[v], cv = c4[v];
+                s[4 * v] = fmaf(dec, s[4 * v], u * bv.x), s[4 * v + 1] = fmaf(dec, s[4 * v + 1], u * bv.y);
+                s[4 * v + 2] = fmaf(dec, s[4 * v + 2], u * bv.z), s[4 * v + 3] = fmaf(dec, s[4 * v + 3], u * bv.w);
+                acc[0] = fmaf(s[4 * v], cv.x, acc[0]), acc[1] = fmaf(s[4 * v + 1], cv.y, acc[1]);
+                acc[2] = fmaf(s[4 * v + 2], cv.z, acc[2]), acc[3] = fmaf(s[4 * v + 3], cv.w, acc[3]);
+            }
+            float o = (acc[0] + acc[1]) + (acc[2] + acc[3]);
+            for (int off = cpw; off < 32; off <<= 1) o += __shfl_xor_sync(0xffffffffu, o, off);
+            if (r == 0 && col < P) stf(y + ((row0 + t0 + tt) * H + h) * P + col, fmaf(dsk, xv, o));
+        }
+    }
+    if (col < P) {
+#pragma unroll
+        for (int j = 0; j < NPT; ++j) {
+            const int i = r * NPT + j;
+            if (i < N) Sg[(long long)i * P] = s[j];
+        }
+    }
+}
+
+// ---- state-space heads: chunks of 64 tokens on the tensor cores --------------------------------------------------------------
+// One CTA: PT = 16 * WARPS columns of one head of one row, all chunks in order.  With cum_t the running sum of the chunk's log
+// decays,
+//     y_t = exp(cum_t) S_0^T C_t + sum_{s <= t} (C_t . B_s) exp(cum_t - cum_s) dt_s x_s  (+ D x_t)
+//     S_L = exp(cum_L) S_0 + sum_s exp(cum_L - cum_s) dt_s B_s x_s^T
+// Every exponent is a sum of log decays and never positive.  A warp owns 16 columns: their state (transposed, [16, NPAD]) sits in
+// accumulator registers, whose layout is the B operand of S_0^T C and the accumulator of the update at once.  The score
+// tile is computed once per CTA (a warp: 64 / WARPS rows) and passed through shared memory.
+constexpr int CL = 64;                       // tokens per chunk
+
+__device__ __forceinline__ void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+    const bf162 h = __floats2bfloat162_rn(a, b);
+    const float2 f = __bfloat1622float2(h);
+    const bf162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
+    hi = *reinterpret_cast<const uint32_t*>(&h);
+    lo = *reinterpret_cast<const uint32_t*>(&l);
+}
+__device__ __forceinline__ float2 unpack2(uint32_t v) { return __bfloat1622float2(*reinterpret_cast<const bf162*>(&v)); }
+
+template <int NT, int WARPS>
+struct ChunkSmem {
+    static constexpr int NPAD = 16 * NT, LDN = NPAD + 8, PT = 16 * WARPS, LDP = PT + 8, LDS = CL + 8;
+    bf16 C[2][CL][LDN], B[2][CL][LDN], X[2][CL][LDP];
+    bf16 Ph[CL][LDS], Pl[CL][LDS];
+    float dt[CL], cum[CL];
+};
+
+template <typename TY, int NT, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
+ssd_chunk_kernel(const bf16* __restrict__ xbc, long long ld, int x_off, int b_off, int c_off, const float* __restrict__ dt,
+                 long long ld_dt, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
+                 const float* __restrict__ dskip, float* __restrict__ S, TY* __restrict__ y, const int* __restrict__ q_start,
+                 const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int H, int G, int N, int P) {
+    using Sm = ChunkSmem<NT, WARPS>;
+    constexpr int THREADS = WARPS * 32, MT = 4 / WARPS;          // 16-row tiles of the score tile per warp
+    extern __shared__ __align__(16) unsigned char smem_raw[];
+    Sm& sm = *reinterpret_cast<Sm*>(smem_raw);
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, qr = lane >> 2, qc = (lane & 3) * 2;
+    const int p_cta = blockIdx.x * Sm::PT, h = blockIdx.y, b = blockIdx.z, g = h / (H / G);
+    const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
+    const long long row0 = (long long)b * Tn;
+    const int pw = p_cta + warp * 16;                            // first column of this warp
+    {
+        const int np = min(Sm::PT, P - p_cta), from = max(n, 0);
+        for (int idx = tid; idx < (Tn - from) * np; idx += THREADS)
+            stf(y + ((row0 + from + idx / np) * H + h) * P + p_cta + idx % np, 0.f);
+    }
+    if (n <= 0) return;
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+    float* Sg = S + ((long long)line * H + h) * N * P;
+    const bool fresh = q_start[b] == 0;
+    const float a = expf(a_log[h]), dsk = dskip[h], dtb = dt_bias != nullptr ? dt_bias[h] : 0.f;
+
+    // state, transposed: tile j holds columns (of N) 8 j .. 8 j + 7; [0], [1]: row pw + qr, [2], [3]: row pw + qr + 8
+    float s[2 * NT][4];
+#pragma unroll
+    for (int j = 0; j < 2 * NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int i = j * 8 + qc + (e & 1), p = pw + qr + (e >> 1) * 8;
+            s[j][e] = (!fresh && i < N && p < P) ? Sg[(long long)i * P + p] : 0.f;
+        }
+
+    auto fetch = [&](int t0, int k) {
+        constexpr int CN = Sm::NPAD / 8, CP = Sm::PT / 8;
+        for (int idx = tid; idx < CL * CN; idx += THREADS) {
+            const int t = idx / CN, i = (idx % CN) * 8;
+            const bool ok = t0 + t < n && i < N;
+            const bf16* src = xbc + (row0 + (ok ? t0 + t : 0)) * ld + (long long)g * N + (ok ? i : 0);
+            mma::cp_async16((uint32_t)__cvta_generic_to_shared(&sm.C[k][t][i]), src + c_off, ok);
+            mma::cp_async16((uint32_t)__cvta_generic_to_shared(&sm.B[k][t][i]), src + b_off, ok);
+        }
+        for (int idx = tid; idx < CL * CP; idx += THREADS) {
+            const int t = idx / CP, i = (idx % CP) * 8;
+            const bool ok = t0 + t < n && p_cta + i < P;
+            const bf16* src = xbc + (row0 + (ok ? t0 + t : 0)) * ld + x_off + (long long)h * P + (ok ? p_cta + i : 0);
+            mma::cp_async16((uint32_t)__cvta_generic_to_shared(&sm.X[k][t][i]), src, ok);
+        }
+        mma::cp_async_commit();
+    };
+    // raw step sizes of the next chunk, two tokens per lane of warp 0
+    float raw0 = 0.f, raw1 = 0.f;
+    auto fetch_dt = [&](int t0) {
+        if (warp == 0) {
+            raw0 = t0 + 2 * lane < n ? dt[(row0 + t0 + 2 * lane) * ld_dt + h] : 0.f;
+            raw1 = t0 + 2 * lane + 1 < n ? dt[(row0 + t0 + 2 * lane + 1) * ld_dt + h] : 0.f;
+        }
+    };
+    fetch_dt(0);
+    fetch(0, 0);
+    int k = 0;
+    for (int t0 = 0; t0 < n; t0 += CL, k ^= 1) {
+        if (warp == 0) {
+            const float d0 = t0 + 2 * lane < n ? softplus_f(raw0 + dtb) : 0.f;
+            const float d1 = t0 + 2 * lane + 1 < n ? softplus_f(raw1 + dtb) : 0.f;
+            const float l0 = -a * d0, l1 = -a * d1;
+            float run = l0 + l1;                                  // inclusive sum over the lanes' pairs
+#pragma unroll
+            for (int o = 1; o < 32; o <<= 1) {
+                const float up = __shfl_up_sync(0xffffffffu, run, o);
+                if (lane >= o) run += up;
+            }
+            sm.dt[2 * lane] = d0, sm.dt[2 * lane + 1] = d1;
+            sm.cum[2 * lane] = run - l1, sm.cum[2 * lane + 1] = run;
+        }
+        if (t0 + CL < n) {
+            fetch(t0 + CL, k ^ 1);
+            fetch_dt(t0 + CL);
+            mma::cp_async_wait<1>();
+        } else {
+            mma::cp_async_wait<0>();
+        }
+        __syncthreads();
+        const uint32_t c_addr = (uint32_t)__cvta_generic_to_shared(&sm.C[k][0][0]);
+        const uint32_t b_addr = (uint32_t)__cvta_generic_to_shared(&sm.B[k][0][0]);
+        const uint32_t x_addr = (uint32_t)__cvta_generic_to_shared(&sm.X[k][0][0]);
+        const uint32_t ph_addr = (uint32_t)__cvta_generic_to_shared(&sm.Ph[0][0]);
+        const uint32_t pl_addr = (uint32_t)__cvta_generic_to_shared(&sm.Pl[0][0]);
+
+        // decayed scores of this warp's rows, columns up to the diagonal
+#pragma unroll
+        for (int mi = 0; mi < MT; ++mi) {
+            const int m = warp + mi * WARPS;                      // 16-row tile
+            float acc[8][4];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[j][0] = acc[j][1] = acc[j][2] = acc[j][3] = 0.f;
+#pragma unroll
+            for (int kk = 0; kk < NT; ++kk) {
+                uint32_t af[4];
+                mma::ldsm_x4(af, c_addr + ((m * 16 + (lane & 15)) * Sm::LDN + kk * 16 + (lane >> 4) * 8) * 2);
+#pragma unroll
+                for (int np = 0; np < 4; ++np) {
+                    if (np <= m) {
+                        uint32_t bf[4];
+                        mma::ldsm_x4(bf, b_addr + ((np * 16 + (lane & 7) + (lane >> 4) * 8) * Sm::LDN + kk * 16 +
+                                                   ((lane >> 3) & 1) * 8) * 2);
+                        mma::mma16816(acc[2 * np], af, bf[0], bf[1]);
+                        mma::mma16816(acc[2 * np + 1], af, bf[2], bf[3]);
+                    }
+                }
+            }
+            const int ta = m * 16 + qr, tb = ta + 8;
+            const float ca = sm.cum[ta], cb = sm.cum[tb];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                if (j <= 2 * m + 1) {
+                    const int c0 = j * 8 + qc;
+                    const float k0 = sm.cum[c0], k1 = sm.cum[c0 + 1], d0 = sm.dt[c0], d1 = sm.dt[c0 + 1];
+                    const float v0 = c0 <= ta ? acc[j][0] * (expf(ca - k0) * d0) : 0.f;
+                    const float v1 = c0 + 1 <= ta ? acc[j][1] * (expf(ca - k1) * d1) : 0.f;
+                    const float v2 = c0 <= tb ? acc[j][2] * (expf(cb - k0) * d0) : 0.f;
+                    const float v3 = c0 + 1 <= tb ? acc[j][3] * (expf(cb - k1) * d1) : 0.f;
+                    uint32_t hi, lo;
+                    split2(v0, v1, hi, lo);
+                    *reinterpret_cast<uint32_t*>(&sm.Ph[ta][c0]) = hi;
+                    *reinterpret_cast<uint32_t*>(&sm.Pl[ta][c0]) = lo;
+                    split2(v2, v3, hi, lo);
+                    *reinterpret_cast<uint32_t*>(&sm.Ph[tb][c0]) = hi;
+                    *reinterpret_cast<uint32_t*>(&sm.Pl[tb][c0]) = lo;
+                }
+            }
+        }
+        // what the state at the chunk's start gives
+        float o[4][2][4];
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int j = 0; j < 2; ++j) o[m][j][0] = o[m][j][1] = o[m][j][2] = o[m][j][3] = 0.f;
+        const bool first = t0 == 0 && fresh;
+        if (!first) {
+#pragma unroll
+            for (int kk = 0; kk < NT; ++kk) {
+                uint32_t h0, h1, h2, h3, l0, l1, l2, l3;
+                split2(s[2 * kk][0], s[2 * kk][1], h0, l0);
+                split2(s[2 * kk + 1][0], s[2 * kk + 1][1], h1, l1);
+                split2(s[2 * kk][2], s[2 * kk][3], h2, l2);
+                split2(s[2 * kk + 1][2], s[2 * kk + 1][3], h3, l3);
+#pragma unroll
+                for (int m = 0; m < 4; ++m) {
+                    uint32_t af[4];
+                    mma::ldsm_x4(af, c_addr + ((m * 16 + (lane & 15)) * Sm::LDN + kk * 16 + (lane >> 4) * 8) * 2);
+                    mma::mma16816(o[m][0], af, h0, h1);
+                    mma::mma16816(o[m][1], af, h2, h3);
+                    mma::mma16816(o[m][0], af, l0, l1);
+                    mma::mma16816(o[m][1], af, l2, l3);
+                }
+            }
+#pragma unroll
+            for (int m = 0; m < 4; ++m) {
+                const float ea = expf(sm.cum[m * 16 + qr]), eb = expf(sm.cum[m * 16 + qr + 8]);
+#pragma unroll
+                for (int j = 0; j < 2; ++j) o[m][j][0] *= ea, o[m][j][1] *= ea, o[m][j][2] *= eb, o[m][j][3] *= eb;
+            }
+        }
+        __syncthreads();                                          // the score tile is complete
+        // the chunk's own tokens, and the update of the state: x as B operand / its scaled transpose as A operand
+        const float cum_l = sm.cum[CL - 1];
+        const float dl = expf(cum_l);
+#pragma unroll
+        for (int j = 0; j < 2 * NT; ++j) s[j][0] *= dl, s[j][1] *= dl, s[j][2] *= dl, s[j][3] *= dl;
+#pragma unroll
+        for (int ks = 0; ks < 4; ++ks) {
+            uint32_t xf[4];                                       // k = token, two 8-column blocks
+            mma::ldsm_x4_t(xf, x_addr + ((ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * Sm::LDP + warp * 16 + (lane >> 4) * 8) * 2);
+#pragma unroll
+            for (int m = 0; m < 4; ++m) {
+                if (m >= ks) {
+                    uint32_t af[4];
+                    const uint32_t off = ((m * 16 + (lane & 15)) * Sm::LDS + ks * 16 + (lane >> 4) * 8) * 2;
+                    mma::ldsm_x4(af, ph_addr + off);
+                    mma::mma16816(o[m][0], af, xf[0], xf[1]);
+                    mma::mma16816(o[m][1], af, xf[2], xf[3]);
+                    mma::ldsm_x4(af, pl_addr + off);
+                    mma::mma16816(o[m][0], af, xf[0], xf[1]);
+                    mma::mma16816(o[m][1], af, xf[2], xf[3]);
+                }
+            }
+            // rows = columns of x, k = token: {rows 0-7, 8-15} x {tokens 0-7, 8-15}
+            uint32_t xt[4], ah[4], al[4];
+            mma::ldsm_x4_t(xt, x_addr + ((ks * 16 + (lane & 7) + (lane >> 4) * 8) * Sm::LDP + warp * 16 + ((lane >> 3) & 1) * 8) * 2);
+            const int s0 = ks * 16 + qc;
+            const float w0 = expf(cum_l - sm.cum[s0]) * sm.dt[s0], w1 = expf(cum_l - sm.cum[s0 + 1]) * sm.dt[s0 + 1];
+            const float w2 = expf(cum_l - sm.cum[s0 + 8]) * sm.dt[s0 + 8], w3 = expf(cum_l - sm.cum[s0 + 9]) * sm.dt[s0 + 9];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const float2 v = unpack2(xt[i]);
+                split2(v.x * (i < 2 ? w0 : w2), v.y * (i < 2 ? w1 : w3), ah[i], al[i]);
+            }
+#pragma unroll
+            for (int j = 0; j < NT; ++j) {
+                uint32_t bf[4];
+                mma::ldsm_x4_t(bf, b_addr + ((ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * Sm::LDN + j * 16 + (lane >> 4) * 8) * 2);
+                mma::mma16816(s[2 * j], ah, bf[0], bf[1]);
+                mma::mma16816(s[2 * j + 1], ah, bf[2], bf[3]);
+                mma::mma16816(s[2 * j], al, bf[0], bf[1]);
+                mma::mma16816(s[2 * j + 1], al, bf[2], bf[3]);
+            }
+        }
+        // store, with the skip term
+#pragma unroll
+        for (int m = 0; m < 4; ++m)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+                const int t = m * 16 + qr + e * 8;
+                if (t0 + t < n) {
+#pragma unroll
+                    for (int j = 0; j < 2; ++j) {
+                        const int p = pw + j * 8 + qc;
+                        if (p < P) {                              // P is even here
+                            const float2 xv = unpack2(*reinterpret_cast<const uint32_t*>(&sm.X[k][t][warp * 16 + j * 8 + qc]));
+                            float v[2] = {fmaf(dsk, xv.x, o[m][j][2 * e]), fmaf(dsk, xv.y, o[m][j][2 * e + 1])};
+                            TY* dst = y + ((row0 + t0 + t) * H + h) * P + p;
+                            if (sizeof(TY) == 4) *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
+                            else *reinterpret_cast<uint32_t*>(dst) = mma::pack2(v[0], v[1]);
+                        }
+                    }
+                }
+            }
+        __syncthreads();                                          // buffer k, the score tile and the sums are free again
+    }
+#pragma unroll
+    for (int j = 0; j < 2 * NT; ++j)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+            const int i = j * 8 + qc + (e & 1), p = pw + qr + (e >> 1) * 8;
+            if (i < N && p < P) Sg[(long long)i * P + p] = s[j][e];
+        }
+}
+
+// ---- gate and grouped norm -------------------------------------------------------------------------------------------------
+// One CTA per (row, group of gs columns): v = y act(z);  out = v / sqrt(mean(v^2) + eps) * w  (w over all columns).
+template <typename TY, typename T, int VEC>
+__global__ void gate_norm_kernel(const TY* __restrict__ y, long long ld_y, const T* __restrict__ z, long long ld_z,
+                                 const float* __restrict__ w, T* __restrict__ out, long long ld_out, int gs, float eps, int act) {
+    constexpr int RV = 4;                    // column groups per thread that stay in registers
+    __shared__ float red[32];
+    const long long row = blockIdx.x;
+    const int c0 = blockIdx.y * gs;
+    const TY* yr = y + row * ld_y + c0;
+    const T* zr = z + row * ld_z + c0;
+    T* orow = out + row * ld_out + c0;
+    float v[RV][VEC], ss = 0.f;
+    auto gated = [&](int c, float* t) {
+        float g[VEC];
+        ldv<VEC>(yr + c, t);
+        ldv<VEC>(zr + c, g);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) t[i] *= act == 1 ? silu_f(g[i]) : sigmoid_f(g[i]);
+    };
+#pragma unroll
+    for (int k = 0; k < RV; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * VEC;
+        if (c < gs) {
+            gated(c, v[k]);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) ss = fmaf(v[k][i], v[k][i], ss);
+        }
+    }
+    for (int c = (threadIdx.x + RV * blockDim.x) * VEC; c < gs; c += blockDim.x * VEC) {
+        float t[VEC];
+        gated(c, t);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss = fmaf(t[i], t[i], ss);
+    }
+    const float r = 1.f / sqrtf(block_sum(ss, red) / (float)gs + eps);
+    auto store = [&](int c, float* t) {
+        float g[VEC];
+        ldv<VEC>(w + c0 + c, g);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) g[i] *= t[i] * r;
+        stv<VEC>(orow + c, g);
+    };
+#pragma unroll
+    for (int k = 0; k < RV; ++k) {
+        const int c = (threadIdx.x + k * blockDim.x) * VEC;
+        if (c < gs) store(c, v[k]);
+    }
+    for (int c = (threadIdx.x + RV * blockDim.x) * VEC; c < gs; c += blockDim.x * VEC) {
+        float t[VEC];
+        gated(c, t);
+        store(c, t);
+    }
+}
+
+// out = y act(z) mul, no norm
+template <typename TY, typename T, int VEC>
+__global__ void gate_mul_kernel(const TY* __restrict__ y, long long ld_y, const T* __restrict__ z, long long ld_z,
+                                T* __restrict__ out, long long ld_out, int n, float mul, int act) {
+    const long long row = blockIdx.x;
+    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; c < n; c += gridDim.y * blockDim.x * VEC) {
+        float t[VEC], g[VEC];
+        ldv<VEC>(y + row * ld_y + c, t);
+        ldv<VEC>(z + row * ld_z + c, g);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) t[i] *= (act == 1 ? silu_f(g[i]) : sigmoid_f(g[i])) * mul;
+        stv<VEC>(out + row * ld_out + c, t);
+    }
+}
+
+template <typename TY, typename T>
+int launch_gate(const void* y, long long ld_y, const void* z, long long ld_z, const float* w, void* out, long long ld_out,
+                long long rows, int n, int groups, float eps, float mul, int act, bool vec, cudaStream_t st) {
+    const int gs = groups > 0 ? n / groups : n;
+    if (groups > 0) {
+        const int per = vec ? 4 : 1;
+        int threads = 32;
+        while (threads < 256 && threads * per * 2 < gs) threads <<= 1;
+        dim3 grid((unsigned)rows, groups);
+        if (vec) gate_norm_kernel<TY, T, 4><<<grid, threads, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, w, (T*)out, ld_out, gs, eps, act);
+        else gate_norm_kernel<TY, T, 1><<<grid, threads, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, w, (T*)out, ld_out, gs, eps, act);
+    } else {
+        dim3 grid((unsigned)rows, (n + 1023) / 1024);
+        if (vec) gate_mul_kernel<TY, T, 4><<<grid, 256, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, (T*)out, ld_out, n, mul, act);
+        else gate_mul_kernel<TY, T, 1><<<grid, 256, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, (T*)out, ld_out, n, mul, act);
+    }
+    NXD_LAUNCH_CHECK();
+    return 0;
+}
+
+}  // namespace
+
+// dtypes: 0 bf16, 1 fp32.  proj [B * Tn, ld] points at the first of the C channels; conv_w fp32 [C, taps] (last column = the
+// current token), bias fp32 [C] or NULL; conv_state fp32 [lines, taps - 1, C], moved to the end of the step (zeros before
+// the start of the sequence; rows without real tokens keep theirs).  out [B * Tn, ld_out]: silu(convolution), zeros in padding
+// rows.  q_start [B], n_new [B] or NULL, seq_ids [B] or NULL as in the attention entry points.
+NXD_API int nxd_conv_silu(int dtype, int out_dtype, const void* proj, long long ld, const float* conv_w, const float* bias,
+                          float* conv_state, void* out, long long ld_out, const int* q_start, const int* n_new,
+                          const int* seq_ids, int B, int Tn, int C, int taps, void* stream) {
+    if ((long long)B * Tn * C == 0) return 0;
+    NXD_REQUIRE(taps >= 1, "short convolution with %d taps", taps);
+    NXD_REQUIRE(B < 65536, "short convolution: %d rows", B);
+    cudaStream_t st = (cudaStream_t)stream;
+    auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+    const bool vec = C % 4 == 0 && ld % 4 == 0 && ld_out % 4 == 0 && al(proj) && al(out) && al(conv_state);
+    // few tokens: one thread walks the whole step and moves the state itself
+    const int TT = Tn <= 64 ? Tn : 32, move = Tn <= 64 ? 1 : 0;
+    dim3 grid((C + 128 * (vec ? 4 : 1) - 1) / (128 * (vec ? 4 : 1)), (Tn + TT - 1) / TT, B);
+    NXD_REQUIRE(grid.y < 65536, "short convolution: %d tokens", Tn);
+#define NXD_CONV(T, TO, V, K)                                                                                            \
+    conv_silu_kernel<T, TO, V, K><<<grid, 128, 0, st>>>((const T*)proj, ld, conv_w, bias, conv_state, (TO*)out, ld_out,    \
+                                                        q_start, n_new, seq_ids, Tn, C, taps, TT, move)
+#define NXD_CONV_T(T, TO)                                                                                                \
+    do {                                                                                                                 \
+        if (taps == 4) { if (vec) NXD_CONV(T, TO, 4, 4); else NXD_CONV(T, TO, 1, 4); }                                    \
+        else { if (vec) NXD_CONV(T, TO, 4, 0); else NXD_CONV(T, TO, 1, 0); }                                              \
+    } while (0)
+    if (dtype == 0 && out_dtype == 0) NXD_CONV_T(bf16, bf16);
+    else if (dtype == 0) NXD_CONV_T(bf16, float);
+    else { NXD_REQUIRE(out_dtype == 1, "short convolution: fp32 input, 16-bit output"); NXD_CONV_T(float, float); }
+#undef NXD_CONV_T
+#undef NXD_CONV
+    NXD_LAUNCH_CHECK();
+    if (!move && taps > 1) {
+        dim3 g2((C + 127) / 128, B);
+        if (dtype == 0) conv_state_kernel<bf16><<<g2, 128, 0, st>>>((const bf16*)proj, ld, conv_state, q_start, n_new, seq_ids, Tn, C, taps);
+        else conv_state_kernel<float><<<g2, 128, 0, st>>>((const float*)proj, ld, conv_state, q_start, n_new, seq_ids, Tn, C, taps);
+        NXD_LAUNCH_CHECK();
+    }
+    return 0;
+}
+
+// x, z, out [B * Tn, ...] (dtype), dt fp32 pre-activations [B * Tn, ld_dt] (softplus(dt + dt_bias) is taken here), bc fp32
+// [B * Tn, ld_bc]: B at column b_off, C at c_off (N each); a_log fp32 [C, N], dskip fp32 [C]; S fp32 [lines, C, N] in place.
+NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const float* dt, long long ld_dt, const float* dt_bias,
+                               const float* bc, long long ld_bc, int b_off, int c_off, const void* z, long long ld_z,
+                               const float* a_log, const float* dskip, float* S, void* out, long long ld_out,
+                               const int* q_start, const int* n_new, const int* seq_ids, int B, int Tn, int C, int N,
+                               void* stream) {
+    if ((long long)B * Tn * C == 0) return 0;
+    NXD_REQUIRE(N >= 1 && N <= 512, "selective scan: %d states per channel", N);
+    NXD_REQUIRE(B < 65536, "selective scan: %d rows", B);
+    cudaStream_t st = (cudaStream_t)stream;
+#define NXD_SEL(T, NS_, R_)                                                                                              \
+    return launch_selective<T, NS_, R_>(x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, z, ld_z, a_log, dskip, S, out, \
+                                        ld_out, q_start, n_new, seq_ids, B, Tn, C, N, st)
+#define NXD_SEL_T(T)                                                                                                     \
+    do {                                                                                                                 \
+        if (N <= 4) NXD_SEL(T, 4, 1);                                                                                    \
+        if (N <= 8) NXD_SEL(T, 4, 2);                                                                                    \
+        if (N <= 16) NXD_SEL(T, 4, 4);                                                                                   \
+        if (N <= 32) NXD_SEL(T, 8, 4);                                                                                   \
+        if (N <= 64) NXD_SEL(T, 8, 8);                                                                                   \
+        if (N <= 128) NXD_SEL(T, 16, 8);                                                                                 \
+        if (N <= 256) NXD_SEL(T, 16, 16);                                                                                \
+        NXD_SEL(T, 16, 32);                                                                                              \
+    } while (0)
+    if (dtype == 0) NXD_SEL_T(bf16);
+    NXD_SEL_T(float);
+#undef NXD_SEL_T
+#undef NXD_SEL
+}
+
+// xbc [B * Tn, ld] (dtype): x [H, P] at column x_off, B and C [G, N] at b_off and c_off (after the convolution); dt fp32
+// pre-activations [B * Tn, ld_dt], one per head; dt_bias (or NULL), a_log, dskip fp32 [H]; S fp32 [lines, H, N, P] in place;
+// y [B * Tn, H, P] (y_dtype).  impl: 0 choose, 1 token by token, 2 chunks on the tensor cores (an error where they do not apply).
+NXD_API int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long long ld, int x_off, int b_off, int c_off,
+                                  const float* dt, long long ld_dt, const float* dt_bias, const float* a_log,
+                                  const float* dskip, float* S, void* y, const int* q_start, const int* n_new,
+                                  const int* seq_ids, int B, int Tn, int H, int G, int N, int P, int impl, void* stream) {
+    if ((long long)B * Tn * H * P == 0) return 0;
+    NXD_REQUIRE(G > 0 && H % G == 0, "state-space heads: %d heads over %d groups", H, G);
+    NXD_REQUIRE(N >= 1 && N <= 1024, "state-space heads: state size %d", N);
+    NXD_REQUIRE(B < 65536 && H < 65536, "state-space heads: %d rows of %d heads", B, H);
+    NXD_REQUIRE(y_dtype == 1 || y_dtype == dtype, "state-space heads: output type");
+    cudaStream_t st = (cudaStream_t)stream;
+    auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+    if (Tn == 1 && n_new == nullptr && impl == 0) {
+        const bool vec = P % 4 == 0 && al(S);
+        dim3 grid((P + 31) / 32, H, B);
+        const size_t smem = (size_t)2 * N * sizeof(float);
+#define NXD_STEP(T, TY, V)                                                                                               \
+    ssd_step_kernel<T, TY, V><<<grid, 128, smem, st>>>((const T*)xbc, ld, x_off, b_off, c_off, dt, ld_dt, dt_bias, a_log, \
+                                                       dskip, S, (TY*)y, q_start, seq_ids, H, G, N, P)
+        if (dtype == 1) { if (vec) NXD_STEP(float, float, 4); else NXD_STEP(float, float, 1); }
+        else if (y_dtype == 1) { if (vec) NXD_STEP(bf16, float, 4); else NXD_STEP(bf16, float, 1); }
+        else { if (vec) NXD_STEP(bf16, bf16, 4); else NXD_STEP(bf16, bf16, 1); }
+#undef NXD_STEP
+        NXD_LAUNCH_CHECK();
+        return 0;
+    }
+    const bool chunks = dtype == 0 && N <= 128 && N % 8 == 0 && P % 8 == 0 && ld % 8 == 0 && x_off % 8 == 0 && b_off % 8 == 0 &&
+                        c_off % 8 == 0 && al(xbc) && al(y);
+    NXD_REQUIRE(impl != 2 || chunks, "state-space heads: the chunk form does not apply (state %d, head size %d)", N, P);
+    if (impl == 2 || (impl == 0 && chunks && Tn >= CL)) {
+#define NXD_CHUNK(TY, NT_, W_)                                                                                           \
+    do {                                                                                                                 \
+        auto kern = ssd_chunk_kernel<TY, NT_, W_>;                                                                       \
+        const size_t smem = sizeof(ChunkSmem<NT_, W_>);                                                                  \
+        if (smem > 48 * 1024)                                                                                            \
+            NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));          \
+        dim3 grid((P + 16 * W_ - 1) / (16 * W_), H, B);                                                                  \
+        kern<<<grid, W_ * 32, smem, st>>>((const bf16*)xbc, ld, x_off, b_off, c_off, dt, ld_dt, dt_bias, a_log, dskip, S, \
+                                          (TY*)y, q_start, n_new, seq_ids, Tn, H, G, N, P);                               \
+    } while (0)
+#define NXD_CHUNK_N(TY, W_)                                                                                              \
+    do { if (N <= 32) NXD_CHUNK(TY, 2, W_); else if (N <= 64) NXD_CHUNK(TY, 4, W_); else NXD_CHUNK(TY, 8, W_); } while (0)
+        // heads of at most 32 columns, and grids that would leave half the GPU idle, take the narrow slices
+        const bool narrow = P <= 32 || (long long)B * H * ((P + 63) / 64) * 2 <= nxd_num_sms();
+        if (y_dtype == 1) { if (narrow) NXD_CHUNK_N(float, 2); else NXD_CHUNK_N(float, 4); }
+        else { if (narrow) NXD_CHUNK_N(bf16, 2); else NXD_CHUNK_N(bf16, 4); }
+#undef NXD_CHUNK_N
+#undef NXD_CHUNK
+        NXD_LAUNCH_CHECK();
+        return 0;
+    }
+    const int npt = N <= 32 ? 8 : (N <= 64 ? 16 : 32);
+    int R = 1;
+    while (R * npt < N) R <<= 1;
+    const int CT = 128 / R;
+    const size_t smem = (size_t)16 * (2 * R * (npt + 4) + CT) * sizeof(float);
+    dim3 grid((P + CT - 1) / CT, H, B);
+#define NXD_SCAN(T, TY, N_)                                                                                              \
+    do {                                                                                                                 \
+        auto kern = ssd_scan_kernel<T, TY, N_>;                                                                          \
+        if (smem > 48 * 1024)                                                                                            \
+            NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));          \
+        kern<<<grid, 128, smem, st>>>((const T*)xbc, ld, x_off, b_off, c_off, dt, ld_dt, dt_bias, a_log, dskip, S, (TY*)y, \
+                                      q_start, n_new, seq_ids, Tn, H, G, N, P, R);                                        \
+    } while (0)
+#define NXD_SCAN_T(T, TY) do { if (npt == 8) NXD_SCAN(T, TY, 8); else if (npt == 16) NXD_SCAN(T, TY, 16); else NXD_SCAN(T, TY, 32); } while (0)
+    if (dtype == 1) NXD_SCAN_T(float, float);
+    else if (y_dtype == 1) NXD_SCAN_T(bf16, float);
+    else NXD_SCAN_T(bf16, bf16);
+#undef NXD_SCAN_T
+#undef NXD_SCAN
+    NXD_LAUNCH_CHECK();
+    return 0;
+}
+
+// y [rows, ld_y] (y_dtype: 0 bf16, 1 fp32), z and out [rows, ...] (dtype): act 0 sigmoid, 1 silu.  groups > 0: v = y act(z),
+// every one of the groups of n / groups columns divided by sqrt(mean(v^2) + eps), times w fp32 [n].  groups == 0: y act(z) mul.
+NXD_API int nxd_gate_norm(int y_dtype, int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w,
+                          void* out, long long ld_out, long long rows, int n, int groups, float eps, float mul, int act,
+                          void* stream) {
+    if (rows * n == 0) return 0;
+    NXD_REQUIRE(rows < (1ll << 31), "gate: %lld rows", rows);
+    NXD_REQUIRE(groups == 0 || (n % groups == 0 && groups < 65536), "gate: %d columns in %d groups", n, groups);
+    auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
+    const int gs = groups > 0 ? n / groups : n;
+    const bool vec = gs % 4 == 0 && ld_y % 4 == 0 && ld_z % 4 == 0 && ld_out % 4 == 0 && al(y) && al(z) && al(out) && al(w);
+    cudaStream_t st = (cudaStream_t)stream;
+    if (dtype == 1) { NXD_REQUIRE(y_dtype == 1, "gate: 16-bit input, fp32 gate"); return launch_gate<float, float>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, mul, act, vec, st); }
+    if (y_dtype == 1) return launch_gate<float, bf16>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, mul, act, vec, st);
+    return launch_gate<bf16, bf16>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, mul, act, vec, st);
+}

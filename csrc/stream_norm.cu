@@ -3,6 +3,8 @@
 //   embed_norm      x = e / sqrt(mean(e^2) + eps) * w_embed,  e = table[token] (+ position vector);  h = norm(x) * w_next
 //                   position vector: entry 2 i = sin(p f_i), entry 2 i + 1 = cos(p f_i), f_i = base^(-2 i / W)
 //   residual_norm   x <- x + y (+ bias);   h = cast(x / sqrt(mean(x^2) + eps) * w_next)
+//   stream_update   x <- [x] + scale * (y + bias) + mul * table[token] + shift, any of the terms, and the same norm: the entry of a
+//                   model (no x yet), a sublayer with a layer scale, the start of a pass of a looped range of layers
 //
 // One CTA per token; the row stays in registers between the passes (up to RV groups of VEC columns per thread; wider rows are
 // read again), statistics in fp32.  Angles are reduced in double precision, so positions of any size keep the accuracy of
@@ -50,17 +52,71 @@ __device__ __forceinline__ void stv(bf16* p, const float* v) {
 
 constexpr int RV = 4;            // column groups per thread that stay in registers
 
-template <typename TY, typename TH, int VEC, int NT>
+// the further terms of a stream update
+struct StreamTerms {
+    const float* scale;          // [W], times (y + bias)
+    const float* shift;          // [W]
+    const void* table;           // [vocab, W], bf16 or fp32, times mul
+    const long long* ids;        // [rows]
+    float mul;
+    int vocab, table_fp32, init; // init: x holds nothing yet
+};
+
+template <typename TY, typename TH, int VEC, int NT, bool TERMS>
 __global__ void __launch_bounds__(NT)
 residual_norm_kernel(float* __restrict__ x, const TY* __restrict__ y, const float* __restrict__ bias,
-                     const float* __restrict__ w, TH* __restrict__ h, int W, float eps) {
+                     const float* __restrict__ w, TH* __restrict__ h, int W, float eps, const StreamTerms ex) {
     __shared__ float red[32];
     const long long row = blockIdx.x;
     float* xr = x + row * W;
     const TY* yr = y != nullptr ? y + row * W : nullptr;
     float v[RV][VEC];
     float ss = 0.f;
+    long long trow = 0;
+    if (TERMS && ex.table != nullptr) trow = min(max(ex.ids[row], 0ll), (long long)ex.vocab - 1) * W;
+    auto load_terms = [&](int c, float* t) {
+        float a[VEC], b[VEC];
+        if (ex.init) {
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) t[i] = 0.f;
+        } else {
+            ldv<VEC>(xr + c, t);
+        }
+        if (yr != nullptr) {
+            ldv<VEC>(yr + c, a);
+            if (bias != nullptr) {
+                ldv<VEC>(bias + c, b);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) a[i] += b[i];
+            }
+            if (ex.scale != nullptr) {
+                ldv<VEC>(ex.scale + c, b);
+#pragma unroll
+                for (int i = 0; i < VEC; ++i) a[i] *= b[i];
+            }
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) t[i] += a[i];
+        }
+        if (ex.table != nullptr) {
+            if (ex.table_fp32) ldv<VEC>((const float*)ex.table + trow + c, a);
+            else ldv<VEC>((const bf16*)ex.table + trow + c, a);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) t[i] = fmaf(a[i], ex.mul, t[i]);
+        }
+        if (ex.shift != nullptr) {
+            ldv<VEC>(ex.shift + c, a);
+#pragma unroll
+            for (int i = 0; i < VEC; ++i) t[i] += a[i];
+        }
+        stv<VEC>(xr + c, t);
+#pragma unroll
+        for (int i = 0; i < VEC; ++i) ss = fmaf(t[i], t[i], ss);
+    };
     auto load = [&](int c, float* t) {
+        if (TERMS) {
+            load_terms(c, t);
+            return;
+        }
         ldv<VEC>(xr + c, t);
         if (yr != nullptr) {
             float a[VEC];
@@ -159,11 +215,11 @@ embed_norm_kernel(const TE* __restrict__ table, const long long* __restrict__ id
     }
 }
 
-template <typename TY, typename TH>
+template <typename TY, typename TH, bool TERMS>
 int launch_residual(float* x, const void* y, const float* bias, const float* w, void* h, long long rows, int W, float eps,
-                    bool vec, cudaStream_t st) {
+                    bool vec, const StreamTerms& ex, cudaStream_t st) {
 #define NXD_RN(V, NT)                                                                                                    \
-    residual_norm_kernel<TY, TH, V, NT><<<(unsigned)rows, NT, 0, st>>>(x, (const TY*)y, bias, w, (TH*)h, W, eps)
+    residual_norm_kernel<TY, TH, V, NT, TERMS><<<(unsigned)rows, NT, 0, st>>>(x, (const TY*)y, bias, w, (TH*)h, W, eps, ex)
     if (vec && W <= 1024) NXD_RN(4, 64);
     else if (vec && W <= 2048) NXD_RN(4, 128);
     else if (vec) NXD_RN(4, 256);
@@ -184,11 +240,35 @@ NXD_API int nxd_residual_norm(int y_dtype, int h_dtype, float* x, const void* y,
     cudaStream_t st = (cudaStream_t)stream;
     auto al = [](const void* p) { return p == nullptr || ((uintptr_t)p % 16) == 0; };
     const bool vec = W % 4 == 0 && al(x) && al(y) && al(bias) && al(w) && al(h);
+    const StreamTerms ex = {};
     switch ((y_dtype << 1) | h_dtype) {
-        case 0: return launch_residual<bf16, bf16>(x, y, bias, w, h, rows, W, eps, vec, st);
-        case 1: return launch_residual<bf16, float>(x, y, bias, w, h, rows, W, eps, vec, st);
-        case 2: return launch_residual<float, bf16>(x, y, bias, w, h, rows, W, eps, vec, st);
-        default: return launch_residual<float, float>(x, y, bias, w, h, rows, W, eps, vec, st);
+        case 0: return launch_residual<bf16, bf16, false>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+        case 1: return launch_residual<bf16, float, false>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+        case 2: return launch_residual<float, bf16, false>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+        default: return launch_residual<float, float, false>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+    }
+}
+
+// As nxd_residual_norm with further terms: x <- (init ? 0 : x) + scale * (y + bias) + mul * table[ids] + shift.  scale and shift
+// [W] fp32 or NULL; table [vocab, W] (t_dtype) with ids [rows] int64, or NULL.
+NXD_API int nxd_stream_update(int y_dtype, int h_dtype, int t_dtype, float* x, const void* y, const float* bias,
+                              const float* scale, const void* table, const long long* ids, float mul, int vocab,
+                              const float* shift, int init, const float* w, void* h, long long rows, int W, float eps,
+                              void* stream) {
+    if (rows == 0) return 0;
+    NXD_REQUIRE(rows < (1ll << 31), "stream update: %lld rows", rows);
+    NXD_REQUIRE(table == nullptr || (ids != nullptr && vocab > 0), "stream update: a table without ids");
+    cudaStream_t st = (cudaStream_t)stream;
+    auto al = [](const void* p) { return p == nullptr || ((uintptr_t)p % 16) == 0; };
+    const bool vec = W % 4 == 0 && al(x) && al(y) && al(bias) && al(w) && al(h) && al(scale) && al(shift) && al(table);
+    StreamTerms ex;
+    ex.scale = scale, ex.shift = shift, ex.table = table, ex.ids = ids, ex.mul = mul, ex.vocab = vocab, ex.table_fp32 = t_dtype;
+    ex.init = init;
+    switch ((y_dtype << 1) | h_dtype) {
+        case 0: return launch_residual<bf16, bf16, true>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+        case 1: return launch_residual<bf16, float, true>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+        case 2: return launch_residual<float, bf16, true>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
+        default: return launch_residual<float, float, true>(x, y, bias, w, h, rows, W, eps, vec, ex, st);
     }
 }
 

@@ -436,7 +436,7 @@ int nxd_glu_bias(int dtype, const void* src, long long ld, int gate_off, int up_
                  int act_kind, void* stream);
 /* router: s = softmax(wr h + zbias); the `top` largest (s + corr) are chosen, weight = s * out_scale; sgate =
  * sigmoid(<wsg, h>).  mode 1: the `top` largest logits are chosen, weight = softmax over the chosen logits; mode 2:
- * s = sigmoid of every logit instead of the softmax */
+ * s = sigmoid of every logit instead of the softmax; mode 3: as mode 0, the chosen s divided by their sum (+ 1e-20) */
 int nxd_moe_router(int dtype, const void* h, const float* wr, const float* corr, const float* wsg, int* idx, float* wts,
                    float* sgate, long long N, int W, int R, int top, float out_scale, const float* zbias, int mode,
                    void* stream);
@@ -445,6 +445,9 @@ int nxd_moe_router(int dtype, const void* h, const float* wr, const float* corr,
 int nxd_moe_gate_up_act(int dtype, const void* h, const void* wgu, const int* idx, void* act, long long P,
                         int pairs_per_token, int W, int F, int E, float limit, float alpha, float up_shift,
                         const float* in_scale, void* stream);
+/* experts without a gate: act[p, :] = max(h[p / pairs_per_token] @ wu[idx[p]], 0)^2, wu [E, W, F] */
+int nxd_moe_up_relu2(int dtype, const void* h, const void* wu, const int* idx, void* act, long long P, int pairs_per_token,
+                     int W, int F, int E, void* stream);
 int nxd_moe_down_combine(int dtype, const void* act, const void* wd, const int* idx, const float* wts, const void* h,
                          const void* act_s, const void* wds, const float* sgate, float* y, long long N, int top, int W,
                          int F, int Fs, int E, void* stream);
@@ -481,6 +484,34 @@ int nxd_residual_norm(int y_dtype, int h_dtype, float* x, const void* y, const f
 int nxd_embed_norm(int e_dtype, int h_dtype, const void* table, const long long* ids, const long long* pos,
                    const double* freq, const float* w_embed, const float* w_next, float* x, void* h, long long rows, int W,
                    int vocab, float eps, void* stream);
+/* the same stream with further terms: x <- (init ? 0 : x) + scale * (y + bias) + mul * table[ids] + shift, then the norm */
+int nxd_stream_update(int y_dtype, int h_dtype, int t_dtype, float* x, const void* y, const float* bias,
+                      const float* scale, const void* table, const long long* ids, float mul, int vocab,
+                      const float* shift, int init, const float* w, void* h, long long rows, int W, float eps, void* stream);
+
+/* State-space mixers (csrc/state_space.cu) on fp32 states of cache lines; rows, lines and padding as in the attention entry
+ * points, zero state where q_start[b] == 0.  dtypes: 0 bf16, 1 fp32.
+ * Short causal convolution per channel + bias + silu; moves conv_state [lines, taps - 1, C] to the end of the step. */
+int nxd_conv_silu(int dtype, int out_dtype, const void* proj, long long ld, const float* conv_w, const float* bias,
+                  float* conv_state, void* out, long long ld_out, const int* q_start, const int* n_new, const int* seq_ids,
+                  int B, int Tn, int C, int taps, void* stream);
+/* S[c, n] <- exp(dt_c A[c, n]) S[c, n] + dt_c x_c B_n, y_c = sum_n S[c, n] C_n + D_c x_c, out = y silu(z);
+ * dt = softplus(dt + dt_bias), A = -exp(a_log); S [lines, C, N] */
+int nxd_selective_scan(int dtype, const void* x, long long ld_x, const float* dt, long long ld_dt, const float* dt_bias,
+                       const float* bc, long long ld_bc, int b_off, int c_off, const void* z, long long ld_z,
+                       const float* a_log, const float* dskip, float* S, void* out, long long ld_out, const int* q_start,
+                       const int* n_new, const int* seq_ids, int B, int Tn, int C, int N, void* stream);
+/* S <- exp(-exp(a_log_h) dt) S + dt B x^T, y = S^T C + D_h x per head, B and C shared by the H / G heads of a group;
+ * S [lines, H, N, P].  impl: 0 choose, 1 token by token, 2 chunks of 64 tokens on the tensor cores (bf16) */
+int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long long ld, int x_off, int b_off, int c_off,
+                          const float* dt, long long ld_dt, const float* dt_bias, const float* a_log, const float* dskip,
+                          float* S, void* y, const int* q_start, const int* n_new, const int* seq_ids, int B, int Tn, int H,
+                          int G, int N, int P, int impl, void* stream);
+/* v = y act(z) (act 0 sigmoid, 1 silu); groups > 0: every group of n / groups columns divided by its root mean square, times w;
+ * groups == 0: v * mul */
+int nxd_gate_norm(int y_dtype, int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w,
+                  void* out, long long ld_out, long long rows, int n, int groups, float eps, float mul, int act,
+                  void* stream);
 
 #ifdef __cplusplus
 }

@@ -1,5 +1,5 @@
 """Hybrid families (recurrent mixers next to attention over the cache) over the framework's step function: Rasodra and,
-further down, Gogalix, Vufasun and Tidavik (windowed attention of several kinds, no recurrence).
+further down, Gogalix, Vufasun, Tidavik (windowed attention of several kinds, no recurrence) and Mumazen (state spaces).
 
 Rasodra over the framework's step function: chunked attention, latent attention and the recurrent matrix memory on
 one KV cache / state manager.
@@ -29,6 +29,7 @@ from typing import Dict, Optional, Tuple
 import torch
 
 from ..models.gogalix import UNIT_NORM_EPS, GogalixConfig, GogalixForCausalLM
+from ..models.mumazen import GLU_SLOPE, MumazenConfig, MumazenForCausalLM, out_proj_columns, x_proj_columns
 from ..models.rasodra import RasodraConfig, RasodraForCausalLM
 from ..models.tidavik import POSITION_BASE, TidavikConfig, TidavikForCausalLM
 from ..models.vufasun import VufasunConfig, VufasunForCausalLM
@@ -43,6 +44,7 @@ from ..ops import moe_sparse as moe_ops
 from ..ops import norm as norm_ops
 from ..ops import retention as ret_ops
 from ..ops import rope as rope_ops
+from ..ops import state_space as ss_ops
 from ..ops import stream_norm as sn_ops
 from ..ops import window_attention as wa_ops
 from ..ops.linear import gemm_nt
@@ -756,6 +758,202 @@ class TidavikInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, TidavikForCau
             x, h = sn_ops.residual_norm_(x, self._feed_forward(layer.mlp, h), None, nxt, eps, dt)
         if self.layer_probe is not None:
             self.layer_probe(i, x.view(B, T, W))
+        return x.view(B, T, W), (h.view(B, T, W) if h is not None else None)
+
+    def forward_speculation(self, *a, **kw):
+        raise NotImplementedError("the speculation verify graph is not wired for this family")
+
+
+class MumazenInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, MumazenForCausalLM):
+    """Mumazen over the KV cache / state manager.  The step function (padding, cache lines through ``seq_ids``, indexed logits,
+    sampler, ``generate``), the schedulers and the runners are the mixin's; this class says what the entry and a layer do:
+
+      * ``hidden`` is the fp32 stream, ``residual`` the normed copy that the sublayer about to run reads, in the activation
+        dtype.  Every change of the stream is one kernel with the norm that follows it (``ops.stream_norm.stream_update_``): the
+        scaled embedding; a sublayer's result (with its output bias) times layer scale and ``residual_mult``; ahead of a
+        pass of the looped range also the embedding once more (gathered from the table again) and the pass's vector;
+      * ONE matrix product of the mixer's input gives all its projections (``layer.in_proj``, parts at ``layer.columns``); the
+        products that become step sizes stay fp32 (``dt_proj``);
+      * ``parallel``: rotation + cache write, capped softmax attention over the cache, the output gate; convolution,
+        state-space heads on the line's fp32 state, gate + grouped norm; both branches write their half of one buffer, which one
+        output projection reads (the branch scales sit in the gate's and the norm's fp32 epilogues);
+      * ``mamba1``: convolution, the fp32 product for step sizes, B and C, the low-rank step sizes' second half, selective scan
+        with the gate inside, output projection;
+      * a looped layer appears once per pass in the run list: same modules, cache / state of the run's own index.
+    A step may start at any position: attention reads earlier keys from the cache, convolutions and recurrences continue from
+    the line's state."""
+
+    supports_prefill_at_offset = True
+    TC_PREFILL_MIN_TOKENS = 128          # shorter steps stay on the cache-reading attention kernels
+
+    def __init__(self, config: MumazenConfig, inference_config: Optional[InferenceConfig] = None, device=None):
+        MumazenForCausalLM.__init__(self, config, device=device)
+        self._init_inference(inference_config)
+        self._sequence = self.layer_sequence()
+        self._pass_of = config.pass_starts()
+        self._rope_cache: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
+        self.layer_probe = None            # callable(i, x) after every layer run (debugging / layer-by-layer checks)
+
+    def _decoder_layers(self):
+        return self._sequence
+
+    def _embedding(self):
+        return self.embed_tokens
+
+    def _final_norm(self):
+        return self.norm
+
+    def init_kv_cache(self, device=None, dtype=None) -> KVCache:
+        ic, cfg = self.inference_config, self.config
+        device = device or next(self.parameters()).device
+        specs, states = [], {}
+        for run, li in enumerate(cfg.layer_runs()):           # one cache / state entry per layer RUN
+            L = cfg.layers[li]
+            if L.type == "parallel":
+                a, r = L.mixer.left, L.mixer.right
+                specs.append((a.kv_heads, a.dim, a.vdim))
+                states[run] = {"S": (r.heads, r.state, r.vdim), "conv": (r.conv - 1, r.channels)}
+            else:
+                m = L.mixer
+                specs.append(None)
+                states[run] = {"S": (m.inner, m.state), "conv": (m.conv - 1, m.inner)}
+        self.kv_cache = KVCache(len(specs), ic.max_batch_size, 0, ic.seq_len, 0, dtype=dtype or cfg.torch_dtype,
+                                device=device, paged=ic.paged_kv, page_size=ic.page_size,
+                                num_pages=ic.num_kv_pages if ic.paged_kv else None, layer_specs=specs, state_specs=states)
+        return self.kv_cache
+
+    def _rotary_tables(self, rot, device) -> Optional[Tuple[torch.Tensor, torch.Tensor]]:
+        if rot is None:
+            return None
+        key = (rot.dims, rot.base, rot.factor)
+        t = self._rope_cache.get(key)
+        if t is None or t[0].device != device or t[0].shape[0] < self.kv_cache.seq_len:
+            t = rope_ops.build_interleaved_rope_cache(self.kv_cache.seq_len, rot.dims, rot.base, device=device, factor=rot.factor)
+            self._rope_cache[key] = t
+        return t
+
+    # -- the stream -------------------------------------------------------------------------------------------------
+    def _pass_terms(self, run: int) -> dict:
+        """What is added to the stream ahead of layer run ``run`` (nothing unless it begins a pass of the looped range)."""
+        t = self._pass_of.get(run)
+        if t is None:
+            return {}
+        terms = {"shift": self.loop_step[t]}
+        if t > 0:
+            terms.update(self._embedding_terms)
+        return terms
+
+    def _update(self, x, run: int, **kw):
+        """A change of the stream and the norm of what layer run ``run`` reads (after the last run: nothing to norm)."""
+        nxt = self._sequence[run].norm1 if run < len(self._sequence) else None
+        return sn_ops.stream_update_(x, w_next=nxt, eps=self.config.rms_norm_eps, out_dtype=self.config.torch_dtype, **kw)
+
+    def _embed_step(self, input_ids: torch.Tensor, position_ids: torch.Tensor):
+        B, T = input_ids.shape
+        self._embedding_terms = {"table": self.embed_tokens.weight, "ids": input_ids.reshape(-1),
+                                 "mul": self.config.embedding_scale}
+        terms = dict(self._embedding_terms)
+        if 0 in self._pass_of:                               # the first pass begins with the model
+            terms["shift"] = self.loop_step[0]
+        x, h = self._update(None, 0, **terms)
+        return x.view(B, T, -1), (h.view(B, T, -1) if h is not None else None)
+
+    def _add_norm(self, norm, hidden: torch.Tensor, residual: Optional[torch.Tensor]):
+        """Only the model's final norm comes through here: plain RMS norm of the fp32 stream."""
+        return sn_ops.residual_norm_(hidden.contiguous(), None, w_next=norm, eps=self.config.rms_norm_eps,
+                                     out_dtype=self.config.torch_dtype)[1], None
+
+    # -- mixers: big [B, T, n_out] = the fused projection of the normed input h [N, W] -> [N, W] ---------------------------
+    def _attention_heads(self, run, m, layer, big, B, T, q_start, n_new, seq_ids):
+        ck, cv = self.kv_cache.layer(run)
+        paged = self._paged()
+        at, n = layer.columns["qkv"]
+        qkv = big[..., at: at + n]
+        tc = (T >= self.TC_PREFILL_MIN_TOKENS and not self._step_past_context
+              and wa_ops.tc_prefill_applies(qkv, m.dim, m.vdim, qkv.stride(-2)))
+        q = wa_ops.qk_norm_cache_write(qkv, ck, cv, q_start, m.heads, m.kv_heads, m.dim, m.vdim, self.config.rms_norm_eps,
+                                       n_new=n_new, seq_ids=seq_ids, normalize=False,
+                                       rope=self._rotary_tables(m.rot, big.device), rope_layout="halves", writeback=tc, **paged)
+        if T == 1:
+            return wa_ops.window_attention_decode(q[:, 0], ck, cv, q_start, m.scale, seq_ids=seq_ids, softcap=m.softcap, **paged)
+        if tc:                              # q, and k / v as views of the projection (the rotated keys were written back)
+            k = qkv[..., m.heads * m.dim: (m.heads + m.kv_heads) * m.dim].unflatten(-1, (m.kv_heads, m.dim))
+            v = qkv[..., (m.heads + m.kv_heads) * m.dim:].unflatten(-1, (m.kv_heads, m.vdim))
+            return wa_ops.window_attention_tc(q.permute(0, 2, 1, 3), k.permute(0, 2, 1, 3), v.permute(0, 2, 1, 3), m.scale,
+                                              softcap=m.softcap).permute(0, 2, 1, 3)
+        return wa_ops.window_attention_prefill(q, ck, cv, q_start, m.scale, n_new=n_new, seq_ids=seq_ids, softcap=m.softcap,
+                                               **paged)
+
+    def _mix_parallel(self, run, layer, h, big, q_start, n_new, seq_ids):
+        mixer, m, cfg = layer.mixer, layer.mixer.cfg, self.config
+        B, T, _ = big.shape
+        N, a, r, cols = B * T, m.left, m.right, layer.columns
+        right, width = out_proj_columns(m)
+        joint = torch.empty(N, width, dtype=h.dtype, device=h.device)
+        if a.width != right or r.inner != width - right:      # columns that pad a half meet zero rows of the projection
+            joint.zero_()
+        rows = big.view(N, -1)
+        part = lambda n: rows[:, cols[n][0]: cols[n][0] + cols[n][1]]                      # noqa: E731
+        o = self._attention_heads(run, a, layer, big, B, T, q_start, n_new, seq_ids)
+        ss_ops.gate_norm(o.reshape(N, a.width), part("g"), act="sigmoid", mul=m.left_scale, out=joint[:, : a.width])
+        st = self.kv_cache.state(run)
+        dt = gemm_nt(h, mixer.dt_proj, out_dtype=torch.float32).view(B, T, -1)[..., : r.heads]
+        at = cols["xbc"][0]
+        xbc = ss_ops.conv_silu(big[..., at: at + r.channels], mixer.conv_weight, mixer.conv_bias, st["conv"], q_start,
+                               n_new=n_new, seq_ids=seq_ids, out_pitch=(r.channels + 7) // 8 * 8)
+        y = ss_ops.state_space_heads(xbc, (0, r.inner, r.inner + r.groups * r.state), dt, mixer.dt_bias, mixer.a_log,
+                                     mixer.d_skip, st["S"], q_start, r.groups, n_new=n_new, seq_ids=seq_ids)
+        ss_ops.gate_norm(y.view(N, r.inner), part("z"), mixer.out_norm, r.norm_groups, cfg.rms_norm_eps,
+                         out=joint[:, right: right + r.inner])
+        return gemm_nt(joint, mixer.o_proj.weight)
+
+    def _mix_mamba1(self, run, layer, h, big, q_start, n_new, seq_ids):
+        mixer, m = layer.mixer, layer.mixer.cfg
+        B, T, _ = big.shape
+        N, cols = B * T, layer.columns
+        st = self.kv_cache.state(run)
+        part = lambda n: big[..., cols[n][0]: cols[n][0] + cols[n][1]]                     # noqa: E731
+        x = ss_ops.conv_silu(part("x"), mixer.conv_weight, mixer.conv_bias, st["conv"], q_start, n_new=n_new, seq_ids=seq_ids)
+        r, b, c, _ = x_proj_columns(m)
+        p = gemm_nt(x.view(N, m.inner), mixer.x_proj, out_dtype=torch.float32)
+        dt = gemm_nt(p[:, :r].to(h.dtype).contiguous(), mixer.dt_proj, out_dtype=torch.float32)
+        y = ss_ops.selective_scan(x, dt.view(B, T, m.inner), mixer.dt_bias, p.view(B, T, -1), b, c, part("z"), mixer.a_log,
+                                  mixer.d_skip, st["S"], q_start, n_new=n_new, seq_ids=seq_ids)
+        return gemm_nt(y.view(N, m.inner), mixer.o_proj.weight)
+
+    _MIX = {"parallel": _mix_parallel, "mamba1": _mix_mamba1}
+
+    def _feed_forward(self, layer, h2: torch.Tensor):
+        """The feed-forward's result ``[N, W]`` and its output bias."""
+        mlp = layer.mlp
+        if layer.mlp_kind == "moe":
+            return mlp(h2), None                                                           # fp32
+        gu = gemm_nt(h2, mlp.gate_up_proj.weight)
+        act = moe_ops.glu_bias(gu, 0, mlp.ff_pad, mlp.ff_pad, mlp.gate_bias, mlp.up_bias, limit=mlp.limit, alpha=GLU_SLOPE,
+                               up_shift=1.0)
+        return gemm_nt(act, mlp.down_proj.weight), mlp.down_bias
+
+    # -- one layer run ------------------------------------------------------------------------------------------------
+    def _layer(self, i: int, layer, hidden, residual, positions, seq_ids, lengths, prefill):
+        cfg = self.config
+        B, T, W = hidden.shape
+        N = B * T
+        x, h = (hidden if hidden.is_contiguous() else hidden.contiguous()).view(N, W), residual.reshape(N, W)
+        if "q_start" not in self._step_kv:      # one int32 copy of the rows' first positions per step, not per kernel
+            self._step_kv["q_start"] = positions[:, 0].to(torch.int32).contiguous()
+        q_start = self._step_kv["q_start"]
+        n_new = self._step_new_tokens if prefill else None
+        big = gemm_nt(h, layer.in_proj.weight).view(B, T, -1)
+        update = {"y": self._MIX[layer.type](self, i, layer, h, big, q_start, n_new, seq_ids), "scale": layer.ls1}
+        if layer.mlp is not None:
+            x, h = sn_ops.stream_update_(x, w_next=layer.norm2, eps=cfg.rms_norm_eps, out_dtype=cfg.torch_dtype, **update)
+            y, bias = self._feed_forward(layer, h)
+            update = {"y": y, "bias": bias, "scale": layer.ls2}
+        if self.layer_probe is not None:        # the stream as the layer leaves it, ahead of what the next pass adds
+            x, _ = sn_ops.stream_update_(x, **update)
+            self.layer_probe(i, x.view(B, T, W))
+            update = {}
+        x, h = self._update(x, i + 1, **update, **self._pass_terms(i + 1))
         return x.view(B, T, W), (h.view(B, T, W) if h is not None else None)
 
     def forward_speculation(self, *a, **kw):

@@ -160,6 +160,24 @@ def _tidavik_cls():
     return TidavikInferenceModel
 
 
+def _mumazen_config(d, dtype):
+    from ..models.mumazen import MumazenConfig
+
+    return MumazenConfig.from_dict(d, torch_dtype=dtype)
+
+
+def _mumazen_convert(sd, cfg):
+    from ..models.mumazen import convert_mumazen_state_dict
+
+    return convert_mumazen_state_dict(sd, cfg)
+
+
+def _mumazen_cls():
+    from .hybrid import MumazenInferenceModel
+
+    return MumazenInferenceModel
+
+
 register_family(ModelFamily("llama", lambda c: _arch(c).startswith("llama"), _llama_config, _llama_cls, _llama_convert))
 register_family(ModelFamily("gekazen", lambda c: _arch(c) == "gekazen", _gekazen_config, _gekazen_cls, _gekazen_convert,
                             kernel_group="window_moe_serving"))
@@ -171,6 +189,8 @@ register_family(ModelFamily("vufasun", lambda c: _arch(c) == "vufasun", _vufasun
                             kernel_group="retention_serving"))
 register_family(ModelFamily("tidavik", lambda c: _arch(c) == "tidavik", _tidavik_config, _tidavik_cls, _tidavik_convert,
                             kernel_group="scored_serving"))
+register_family(ModelFamily("mumazen", lambda c: _arch(c) == "mumazen", _mumazen_config, _mumazen_cls, _mumazen_convert,
+                            kernel_group="state_space_serving"))
 
 
 def read_config(model_dir: str) -> Dict[str, Any]:

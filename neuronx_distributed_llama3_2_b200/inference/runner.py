@@ -354,6 +354,16 @@ class GekazenRunner(InferenceRunner):
         super().__init__(*a, **kw)
 
 
+class MumazenRunner(InferenceRunner):
+    """Runner of the Mumazen family (``models/mumazen.py``): same buckets, graphs and generate loop."""
+
+    def __init__(self, *a, **kw):
+        from .hybrid import MumazenInferenceModel
+
+        kw.setdefault("model_cls", MumazenInferenceModel)
+        super().__init__(*a, **kw)
+
+
 class RasodraRunner(InferenceRunner):
     """Runner of the Rasodra family (``models/rasodra.py``): same buckets, graphs and generate loop."""
 

@@ -13,5 +13,7 @@ from .gogalix import (GogalixConfig, GogalixForCausalLM, convert_gogalix_state_d
                       tiny_gogalix)
 from .vufasun import (VufasunConfig, VufasunForCausalLM, convert_vufasun_state_dict, export_vufasun_state_dict,  # noqa: F401
                       tiny_vufasun)
+from .mumazen import (MumazenConfig, MumazenForCausalLM, convert_mumazen_state_dict, export_mumazen_state_dict,  # noqa: F401
+                      tiny_mumazen)
 from .tidavik import (TidavikConfig, TidavikForCausalLM, convert_tidavik_state_dict, export_tidavik_state_dict,  # noqa: F401
                       tiny_tidavik)

@@ -111,17 +111,19 @@ class RouterBiasedTopK(RouterBase):
     router runs in fp32 whatever the activation dtype; ``select`` is the fused device path (one kernel: projection,
     softmax, choice, optional sigmoid gate of a shared expert).  ``bias``: a bias on the logits (``logit_bias``);
     ``renormalize``: the experts with the largest logits are chosen and their weights are the softmax over the chosen
-    logits only; ``score="sigmoid"``: every expert's score is the sigmoid of its own logit instead of the softmax."""
+    logits only; ``score="sigmoid"``: every expert's score is the sigmoid of its own logit instead of the softmax;
+    ``normalize``: the chosen experts' softmax scores are divided by their sum."""
 
     def __init__(self, num_experts: int, top_k: int, hidden_size: int, num_identity_experts: int = 0,
                  affinity_scale: float = 1.0, device: torch.device = torch.device("cpu"), bias: bool = False,
-                 renormalize: bool = False, score: str = "softmax"):
+                 renormalize: bool = False, score: str = "softmax", normalize: bool = False):
         super().__init__(num_experts + num_identity_experts, top_k, hidden_size, score, torch.float32, device)
         self.score = score
         self.num_real_experts = num_experts
         self.num_identity_experts = num_identity_experts
         self.affinity_scale = affinity_scale
         self.renormalize = renormalize
+        self.normalize = normalize
         self.logit_bias = torch.nn.Parameter(torch.zeros(num_experts + num_identity_experts, dtype=torch.float32,
                                                          device=device), requires_grad=False) if bias else None
         self.correction = torch.nn.Parameter(torch.zeros(num_experts + num_identity_experts, dtype=torch.float32,
@@ -133,7 +135,7 @@ class RouterBiasedTopK(RouterBase):
 
         flat = hidden_states.reshape(-1, hidden_states.shape[-1])
         return moe_sparse.route(flat, self.linear_router.weight, self.correction, self.top_k, self.affinity_scale,
-                                shared_gate_weight, self.logit_bias, self.renormalize, self.score)
+                                shared_gate_weight, self.logit_bias, self.renormalize, self.score, self.normalize)
 
     def forward(self, hidden_states):
         flat = hidden_states.reshape(-1, hidden_states.shape[-1])
@@ -146,4 +148,7 @@ class RouterBiasedTopK(RouterBase):
             return router_logits, scores * self.affinity_scale, expert_index.detach().to(torch.long)
         scores = self.apply_activation_fn(router_logits)
         _, expert_index = torch.topk(scores + self.correction.float(), self.top_k, dim=1)
+        if self.normalize:       # affinities: the chosen scores divided by their sum, zero elsewhere
+            val = scores.gather(1, expert_index)
+            scores = torch.zeros_like(scores).scatter(1, expert_index, val / (val.sum(-1, keepdim=True) + 1e-20))
         return router_logits, scores * self.affinity_scale, expert_index.detach().to(torch.long)

@@ -4,7 +4,8 @@ identity experts and an optional gated shared expert.  ``router_bias``: the rout
 ``renormalize``: the experts with the largest logits are chosen and weighted by the softmax over the chosen logits only.
 ``score="sigmoid"``: every expert's score is the sigmoid of its own logit.  ``weight_on_input``: the routing weight
 multiplies the chosen expert's input instead of its output, ``sum_j expert_j(w_j h)``.  ``shared_gated=False``: the
-shared expert is added as it is, without a sigmoid gate of its own.
+shared expert is added as it is, without a sigmoid gate of its own.  ``normalize``: the chosen experts' softmax scores are
+divided by their sum.  ``gated=False``: the experts (and the shared one) have no gate, ``down(max(up h, 0) ** 2)``.
 
 Two execution paths over the same parameters:
   * pairs   every (token, choice) pair runs a GEMV against the chosen expert's weights, picked by the index ON THE
@@ -21,6 +22,7 @@ from typing import Optional
 
 import torch
 
+from ...ops import activation as act_ops
 from ...ops import moe_sparse
 from .experts import Experts
 from .moe_parallel_layers import LinearRouter
@@ -35,9 +37,11 @@ class SparseMoE(torch.nn.Module):
                  num_identity_experts: int = 0, affinity_scale: float = 1.0, shared_intermediate_size: int = 0,
                  shared_limit: Optional[float] = None, alpha: float = moe_sparse.GLU_ALPHA,
                  dtype: torch.dtype = torch.float32, device=None, router_bias: bool = False, renormalize: bool = False,
-                 score: str = "softmax", weight_on_input: bool = False, shared_gated: bool = True):
+                 score: str = "softmax", weight_on_input: bool = False, shared_gated: bool = True,
+                 normalize: bool = False, gated: bool = True):
         super().__init__()
-        self.weight_on_input = weight_on_input
+        assert gated or not weight_on_input
+        self.weight_on_input, self.gated = weight_on_input, gated
         dev = device if device is not None else torch.device("cpu")
         self.hidden_size, self.num_experts, self.top_k = hidden_size, num_experts, top_k
         if limit is None:            # plain silu(gate) * up: no clamp, unit slope, no shift of the linear half
@@ -47,14 +51,15 @@ class SparseMoE(torch.nn.Module):
         shift = self.up_shift
         self.limit, self.alpha = limit, alpha
         self.router = RouterBiasedTopK(num_experts, top_k, hidden_size, num_identity_experts, affinity_scale, device=dev,
-                                       bias=router_bias, renormalize=renormalize, score=score)
-        self.experts = Experts(num_experts, hidden_size, intermediate_size, True, None, dtype=dtype, device=dev,
+                                       bias=router_bias, renormalize=renormalize, score=score, normalize=normalize)
+        plain = None if gated else act_ops.relu_squared
+        self.experts = Experts(num_experts, hidden_size, intermediate_size, gated, plain, dtype=dtype, device=dev,
                                glu_fn=lambda gu: moe_sparse.clamped_glu(gu, limit, alpha, shift))
         self.shared = None
         if shared_intermediate_size > 0:
             sl = shared_limit if shared_limit is not None else limit
             self.shared_limit = sl
-            self.shared = Experts(1, hidden_size, shared_intermediate_size, True, None, dtype=dtype, device=dev,
+            self.shared = Experts(1, hidden_size, shared_intermediate_size, gated, plain, dtype=dtype, device=dev,
                                   glu_fn=lambda gu: moe_sparse.clamped_glu(gu, sl, alpha, shift))
             self.shared_gate = LinearRouter(hidden_size, 1, dtype=torch.float32, device=dev) if shared_gated else None
 
@@ -71,6 +76,12 @@ class SparseMoE(torch.nn.Module):
         sorted_path = self._use_sorted(h.shape[0]) if path is None else path == "sorted"
         if sorted_path:
             return self._forward_sorted(h, idx, wts, sg)
+        if not self.gated:
+            act = moe_sparse.up_act(h, self.experts.up_proj.weight, idx)
+            s_act = s_down = None
+            if self.shared is not None:
+                s_act, s_down = moe_sparse.up_act(h, self.shared.up_proj.weight, None), self.shared.down_proj.weight[0]
+            return moe_sparse.down_combine(act, self.experts.down_proj.weight, idx, wts, h, s_act, s_down, sg)
         w_gu, w_d = self.experts.gate_up_proj.weight, self.experts.down_proj.weight
         in_scale = None
         if self.weight_on_input:            # the weight goes into the expert; the outputs are summed as they are

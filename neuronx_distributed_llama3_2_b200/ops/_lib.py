@@ -76,8 +76,16 @@ GROUPS["scored_serving"] = ["window_attention.cu", "latent_attention.cu", "strea
                             "gemm_tcgen05.cu", "gemm_smallm.cu", "decode_fused.cu", "fused_gemm_ar.cu", "tma_host.cu",
                             "flash_attn_tc.cu", "attn_tc_host.cu"]
 
+# the state-space family (selective scan and state-space heads behind short convolutions, capped attention next to the latter,
+# clamped gated and sparse feed-forward on a pre-norm fp32 stream): attention over the cache, the stream's norms, sparse MoE
+# and its activation, the mixers' own source, the GEMM kernels behind the linear layers and the tcgen05 flash attention
+GROUPS["state_space_serving"] = ["window_attention.cu", "state_space.cu", "stream_norm.cu", "moe_sparse.cu", "mlstm.cu",
+                                 "runtime.cu", "gemm_tcgen05.cu", "gemm_smallm.cu", "fused_gemm_ar.cu", "tma_host.cu",
+                                 "flash_attn_tc.cu", "attn_tc_host.cu"]
+
 # sources whose fp32 state is carried over thousands of steps: no approximate exp / tanh / division
-PRECISE_SOURCES = {"mlstm.cu", "delta_rule.cu", "retention.cu", "hyper_connection.cu", "stream_norm.cu"}
+PRECISE_SOURCES = {"mlstm.cu", "delta_rule.cu", "retention.cu", "hyper_connection.cu", "stream_norm.cu",
+                   "state_space.cu"}
 
 _lib: Optional[ctypes.CDLL] = None
 _group_libs = {}

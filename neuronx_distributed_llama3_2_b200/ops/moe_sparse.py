@@ -5,9 +5,10 @@ follow the expert index without a host round trip; a clamped gated activation; t
     s = softmax(Wr h + b);  chosen = top-k of (s + correction);  weight = s[chosen] * scale
     renormalised form:  chosen = top-k of the logits,  weight = softmax over the chosen logits only
     sigmoid form:       s = sigmoid(Wr h + b) per expert, then as the first form
+    normalised form:    as the first form, weight = s[chosen] / (sum of the chosen s + 1e-20) * scale
     the weight multiplies the expert's output, or (``in_scale``) its input:  sum_j expert_j(w_j h)
     act(g, u) = g' * sigmoid(alpha * g') * (u' + shift),  g' = min(g, limit),  u' = clamp(u, -limit, limit)
-    (limit = inf, alpha = 1, shift = 0 is the plain silu(g) * u)
+    (limit = inf, alpha = 1, shift = 0 is the plain silu(g) * u);  experts without a gate: act(u) = max(u, 0)^2
     expert index >= E: identity expert (output = input)
 
 Expert weights use the layout of the grouped expert layers (``modules/moe``): ``gate_up [E, W, 2F]``, ``down [E, F, W]``.
@@ -88,12 +89,14 @@ def glu_bias(src: torch.Tensor, gate_offset: int, up_offset: int, width: int, ga
 
 def route(h: torch.Tensor, router_w: torch.Tensor, correction: Optional[torch.Tensor], top: int, scale: float,
           shared_gate_w: Optional[torch.Tensor] = None, logit_bias: Optional[torch.Tensor] = None,
-          renormalize: bool = False, score: str = "softmax") -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
+          renormalize: bool = False, score: str = "softmax", normalize: bool = False) -> Tuple[torch.Tensor, torch.Tensor, Optional[torch.Tensor]]:
     """``h [N, W]``, ``router_w [R, W]`` fp32 -> ``(index [N, top] int32, weight [N, top] fp32, shared gate [N] fp32)``.
     ``logit_bias [R]`` is added to the logits; ``renormalize``: the largest logits are chosen and weighted by the softmax
     over the chosen logits only (``correction`` does not apply); ``score="sigmoid"``: every expert's score is the sigmoid
-    of its own logit instead of the softmax over all of them."""
+    of its own logit instead of the softmax over all of them; ``normalize`` (softmax scores): the chosen experts' scores are
+    divided by their sum."""
     assert score in ("softmax", "sigmoid") and not (renormalize and score == "sigmoid")
+    assert not normalize or (score == "softmax" and not renormalize)
     N, W = h.shape
     R = router_w.shape[0]
     if _use_kernel(h) and router_w.dtype == torch.float32:
@@ -108,7 +111,7 @@ def route(h: torch.Tensor, router_w: torch.Tensor, correction: Optional[torch.Te
         rc = L.nxd_moe_router(_c.c_int(_code(h.dtype)), _lib.ptr(h), _lib.ptr(router_w.contiguous()), _lib.ptr(corr),
                               _lib.ptr(wsg), _lib.ptr(idx), _lib.ptr(wts), _lib.ptr(sg), _c.c_longlong(N), _c.c_int(W),
                               _c.c_int(R), _c.c_int(top), _c.c_float(scale), _lib.ptr(zb),
-                              _c.c_int(2 if score == "sigmoid" else int(renormalize)), _lib.stream_ptr())
+                              _c.c_int(3 if normalize else (2 if score == "sigmoid" else int(renormalize))), _lib.stream_ptr())
         _lib.check(rc, "nxd_moe_router", L)
         return idx, wts, sg
     hf = h.float()
@@ -123,6 +126,9 @@ def route(h: torch.Tensor, router_w: torch.Tensor, correction: Optional[torch.Te
     choice = s + correction.float() if correction is not None else s
     idx = torch.topk(choice, top, dim=-1).indices
     wts = s.gather(1, idx) * scale
+    if normalize:
+        wts = s.gather(1, idx)
+        wts = wts / (wts.sum(-1, keepdim=True) + 1e-20) * scale
     return idx.to(torch.int32), wts, sg
 
 
@@ -157,6 +163,31 @@ def gate_up_act(h: torch.Tensor, w_gate_up: torch.Tensor, idx: Optional[torch.Te
                 x = x * in_scale.reshape(-1)[rows].float().unsqueeze(1)
             gu = x @ w_gate_up[e].float()
             act[rows] = clamped_glu_ref(gu[:, :F], gu[:, F:], limit, alpha, up_shift).to(h.dtype)
+    return act
+
+
+def up_act(h: torch.Tensor, w_up: torch.Tensor, idx: Optional[torch.Tensor]) -> torch.Tensor:
+    """Experts without a gate: ``max(h @ w_up[idx], 0) ** 2`` of every (token, choice) pair; ``w_up [E, W, F]``, ``idx [N, top]``
+    (or ``None``: one dense expert) -> ``[N * top, F]``.  Rows of identity experts are undefined (nothing reads them)."""
+    N, W = h.shape
+    E, _, F = w_up.shape
+    top = idx.shape[1] if idx is not None else 1
+    if _use_kernel(h) and w_up.dtype == h.dtype:
+        h = h if h.is_contiguous() else h.contiguous()
+        act = torch.empty(N * top, F, dtype=h.dtype, device=h.device)
+        L = _lib.lib(GROUP)
+        rc = L.nxd_moe_up_relu2(_c.c_int(_code(h.dtype)), _lib.ptr(h), _lib.ptr(w_up), _lib.ptr(idx), _lib.ptr(act),
+                                _c.c_longlong(N * top), _c.c_int(top), _c.c_int(W), _c.c_int(F), _c.c_int(E),
+                                _lib.stream_ptr())
+        _lib.check(rc, "nxd_moe_up_relu2", L)
+        return act
+    act = torch.zeros(N * top, F, dtype=h.dtype, device=h.device)
+    e_of = idx.reshape(-1).long() if idx is not None else torch.zeros(N, dtype=torch.long, device=h.device)
+    tok = torch.arange(N, device=h.device).repeat_interleave(top)
+    for e in range(E):
+        rows = (e_of == e).nonzero().reshape(-1)
+        if rows.numel():
+            act[rows] = (h[tok[rows]].float() @ w_up[e].float()).clamp(min=0.0).square().to(h.dtype)
     return act
 
 

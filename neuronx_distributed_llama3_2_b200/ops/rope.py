@@ -53,15 +53,17 @@ def wavelength_scaled_frequencies(freq: torch.Tensor, factor: float, low: float,
 
 
 def build_interleaved_rope_cache(max_pos: int, dims: int, base: float, device=None,
-                                 scaling: Optional[Tuple[float, float, float, float]] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+                                 scaling: Optional[Tuple[float, float, float, float]] = None,
+                                 factor: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
     """fp32 ``cos`` / ``sin`` tables ``[max_pos, dims/2]`` of the angles ``p * base ** (-2 i / dims)``, evaluated in
     float64 (a position of a few thousand times a frequency loses digits of the angle in fp32).  ``scaling = (factor, low,
-    high, original)``: the frequencies first go through ``wavelength_scaled_frequencies``."""
+    high, original)``: the frequencies first go through ``wavelength_scaled_frequencies``; ``factor``: all of them are divided
+    by it (linear scaling)."""
     i = torch.arange(dims // 2, dtype=torch.float64)
     freq = torch.pow(torch.tensor(float(base), dtype=torch.float64), -2.0 * i / dims)
     if scaling is not None:
         freq = wavelength_scaled_frequencies(freq, *[float(x) for x in scaling])
-    ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), freq)
+    ang = torch.outer(torch.arange(max_pos, dtype=torch.float64), freq / factor)
     return ang.cos().float().contiguous().to(device), ang.sin().float().contiguous().to(device)
 
 
