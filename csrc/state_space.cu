@@ -43,7 +43,31 @@ __device__ __forceinline__ float exp2_ftz(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
     return r;
 }
+// e^y for y <= 0, rounded once where it is close to 1: a decay that hardly decays is applied thousands of times, and an error of
+// even one unit in its last place that always points the same way would add up.  1 + y (1 + y/2 + ... + y^7/40320) there.
+__device__ __forceinline__ float decay_exp(float y) {
+    if (y < -0.35f) return expf(y);
+    float p = fmaf(y, 1.f / 40320.f, 1.f / 5040.f);
+    p = fmaf(y, p, 1.f / 720.f);
+    p = fmaf(y, p, 1.f / 120.f);
+    p = fmaf(y, p, 1.f / 24.f);
+    p = fmaf(y, p, 1.f / 6.f);
+    p = fmaf(y, p, 0.5f);
+    p = fmaf(y, p, 1.f);
+    return fmaf(y, p, 1.f);
+}
 constexpr float LOG2E = 1.4426950408889634f;
+// the decay of a state in the selective scan: fp32 serving rounds it as above, 16-bit serving takes the hardware's 2^x
+template <typename T>
+struct ScanDecay {
+    static __device__ __forceinline__ float rate(float a) { return a * LOG2E; }
+    static __device__ __forceinline__ float at(float dt, float rate) { return exp2_ftz(dt * rate); }
+};
+template <>
+struct ScanDecay<float> {
+    static __device__ __forceinline__ float rate(float a) { return a; }
+    static __device__ __forceinline__ float at(float dt, float rate) { return decay_exp(dt * rate); }
+};
 
 template <int VEC>
 __device__ __forceinline__ void ldv(const float* p, float* v) {
@@ -244,7 +268,7 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
         const int i = r * NS + j;
         const bool ok = c < C && i < N;
         s[j] = (ok && !fresh) ? Sc[i] : 0.f;
-        a2[j] = ok ? -expf(a_log[(long long)c * N + i]) * LOG2E : 0.f;
+        a2[j] = ok ? ScanDecay<T>::rate(-expf(a_log[(long long)c * N + i])) : 0.f;
     }
     // columns N .. NP - 1 of B and C are zeros in both buffers and stay so
     if (N < NP)
@@ -333,10 +357,10 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
                 for (int j = 0; j < NS; j += 4) {
                     const float4 bv = *reinterpret_cast<const float4*>(&d.B[g0 + q][r * NS + j]);
                     const float4 cv = *reinterpret_cast<const float4*>(&d.Cm[g0 + q][r * NS + j]);
-                    s[j] = fmaf(exp2_ftz(dv * a2[j]), s[j], u * bv.x);
-                    s[j + 1] = fmaf(exp2_ftz(dv * a2[j + 1]), s[j + 1], u * bv.y);
-                    s[j + 2] = fmaf(exp2_ftz(dv * a2[j + 2]), s[j + 2], u * bv.z);
-                    s[j + 3] = fmaf(exp2_ftz(dv * a2[j + 3]), s[j + 3], u * bv.w);
+                    s[j] = fmaf(ScanDecay<T>::at(dv, a2[j]), s[j], u * bv.x);
+                    s[j + 1] = fmaf(ScanDecay<T>::at(dv, a2[j + 1]), s[j + 1], u * bv.y);
+                    s[j + 2] = fmaf(ScanDecay<T>::at(dv, a2[j + 2]), s[j + 2], u * bv.z);
+                    s[j + 3] = fmaf(ScanDecay<T>::at(dv, a2[j + 3]), s[j + 3], u * bv.w);
                     acc[0] = fmaf(s[j], cv.x, acc[0]);
                     acc[1] = fmaf(s[j + 1], cv.y, acc[1]);
                     acc[0] = fmaf(s[j + 2], cv.z, acc[0]);
@@ -406,7 +430,7 @@ ssd_step_kernel(const T* __restrict__ xbc, long long ld, int x_off, int b_off, i
         Cs[i] = ldf(row + c_off + g * N + i);
     }
     const float step = softplus_f(dt[(long long)b * ld_dt + h] + (dt_bias != nullptr ? dt_bias[h] : 0.f));
-    const float decay = expf(-expf(a_log[h]) * step);
+    const float decay = decay_exp(-expf(a_log[h]) * step);
     const bool fresh = q_start[b] == 0, ok = p0 < P;
     const int line = seq_ids != nullptr ? seq_ids[b] : b;
     float xv[VEC], u[VEC], acc[VEC];
@@ -502,7 +526,7 @@ ssd_scan_kernel(const T* __restrict__ xbc, long long ld, int x_off, int b_off, i
         if (tid < cnt) {
             const float step = softplus_f(dt[(row0 + t0 + tid) * ld_dt + h] + (dt_bias != nullptr ? dt_bias[h] : 0.f));
             sd[tid] = step;
-            sg[tid] = expf(-a * step);
+            sg[tid] = decay_exp(-a * step);
         }
         __syncthreads();
         for (int tt = 0; tt < cnt; ++tt) {

@@ -263,7 +263,7 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
             const int dist = p_i - j;
             const bool vis = row_ok && dist >= 0 && (window <= 0 || dist < window || j < keep_first) &&
                              (chunk <= 0 || p_i / chunk == j / chunk);
-            if (mod.cap > 0.f) d = mod.cap * score::tanh_any(d / mod.cap);
+            if (mod.cap > 0.f) d = mod.cap * score::tanh_fp32(__fdiv_rn(d, mod.cap));
             if (r1 != 0.f) d -= r1 * logf(1.f + r2 * (float)max(dist, 0));
             s[m] = vis ? d - slope * (float)dist : -INFINITY;
             tmax = fmaxf(tmax, s[m]);
@@ -693,7 +693,7 @@ window_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ cache_k
         for (int r = 0; r < DEC_R; ++r) {
             if (r < R) {
                 float s = warp_sum(d[r]);
-                if (mod.cap > 0.f) s = mod.cap * score::tanh_any(s / mod.cap);
+                if (mod.cap > 0.f) s = mod.cap * score::tanh_fp32(__fdiv_rn(s, mod.cap));
                 s -= sl[r] * dist;
                 if (mod.r1 != nullptr) s -= r1[r] * logf(1.f + r2[r] * dist);
                 const float m_new = sig ? 0.f : fmaxf(m_r[r], s);
