@@ -55,11 +55,11 @@ def parse_args():
     ap.add_argument("--no-inference", action="store_true",
                     help="skip the second half of the headline metric (Llama-3.2-1B TTFT / decode tokens/s, reported "
                          "under the extra key \"inference\")")
-    ap.add_argument("--families", nargs="?", const="gekazen", default="", choices=["gekazen", "rasodra", "gogalix", "vufasun", "tidavik"],
+    ap.add_argument("--families", nargs="?", const="gekazen", default="", choices=["gekazen", "rasodra", "gogalix", "vufasun", "tidavik", "mumazen"],
                     help="instead of the headline workload: serving throughput (prefill and decode tokens/s) of a "
                          "family next to the closest existing decoder at equal layer sizes (gekazen: the Mixtral-style "
                          "decoder; rasodra: the Llama decoder; gogalix: the Rasodra hybrid; vufasun: the Gogalix hybrid; tidavik: Rasodra's "
-                         "attention layers), and their like-for-like "
+                         "attention layers; mumazen: the Vufasun hybrid), and their like-for-like "
                          "kernels with roofline fractions "
                          "(1 GPU; one JSON line)")
     ap.add_argument("--profile", default="", help="diagnosis only: write a kernel timeline summary of 2 steps (rank 0) "
@@ -439,7 +439,8 @@ def main():
         sampler = ClockSampler(local_rank)
         sampler.start()
         bench_fn = {"rasodra": family_bench.run_hybrid, "gogalix": family_bench.run_delta,
-                    "vufasun": family_bench.run_retention, "tidavik": family_bench.run_scored}.get(args.families, family_bench.run)
+                    "vufasun": family_bench.run_retention, "tidavik": family_bench.run_scored,
+                    "mumazen": family_bench.run_state_space}.get(args.families, family_bench.run)
         out = bench_fn(steps=args.steps, warmup=args.warmup, device=dev)
         out["clocks"] = sampler.stop()
         print(json.dumps(out))

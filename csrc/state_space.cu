@@ -242,7 +242,8 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
                       const T* __restrict__ z, long long ld_z, const float* __restrict__ a_log, const float* __restrict__ dskip,
                       float* __restrict__ S, T* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
                       const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int C, int N, int async) {
-    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS > R ? SS_TS : R;
+    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS;
+    static_assert(TS % R == 0, "tokens come in groups of R");
     struct Buf {
         float B[TS][NP], Cm[TS][NP], dt[TS][CH];
         T x[TS][CH], z[TS][CH];
@@ -278,7 +279,7 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
             bufs[k].Cm[q / (NP - N)][N + q % (NP - N)] = 0.f;
         }
     constexpr int XV = 16 / sizeof(T);                       // elements of T per 16 bytes
-    constexpr int CX = CH / XV > 0 ? CH / XV : 1;            // such pieces per token (narrower CTAs never copy that way)
+    constexpr int CX = CH / XV;                              // such pieces per token
     auto fetch = [&](int t0, int k) {
         Buf& d = bufs[k];
         const int cnt = min(TS, n - t0);
@@ -394,7 +395,7 @@ int launch_selective(const void* x, long long ld_x, const float* dt, long long l
                      long long ld_bc, int b_off, int c_off, const void* z, long long ld_z, const float* a_log,
                      const float* dskip, float* S, void* out, long long ld_out, const int* q_start, const int* n_new,
                      const int* seq_ids, int B, int Tn, int C, int N, cudaStream_t st) {
-    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS > R ? SS_TS : R;
+    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS;
     constexpr size_t smem = 2 * (size_t)TS * (2 * NP * 4 + CH * 4 + 2 * CH * sizeof(T)) + 2 * (size_t)TS * CH * 4;
     auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
     constexpr int XV = 16 / sizeof(T);
@@ -980,7 +981,7 @@ NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const f
         if (N <= 64) NXD_SEL(T, 8, 8);                                                                                   \
         if (N <= 128) NXD_SEL(T, 16, 8);                                                                                 \
         if (N <= 256) NXD_SEL(T, 16, 16);                                                                                \
-        NXD_SEL(T, 16, 32);                                                                                              \
+        NXD_SEL(T, 32, 16);                                                                                              \
     } while (0)
     if (dtype == 0) NXD_SEL_T(bf16);
     NXD_SEL_T(float);

@@ -167,6 +167,10 @@ __global__ void qk_norm_cache_write_kernel(const T* __restrict__ qkv, long long 
             const float c = cs[i], s = sn[i];
             stf(dst + iu, u * c - v * s);
             stf(dst + iv, v * c + u * s);
+            if (back != nullptr) {               // this lane is the only one that reads the pair
+                stf(back + iu, u * c - v * s);
+                stf(back + iv, v * c + u * s);
+            }
         }
     }
     for (int i = rot + lane; i < dim; i += 32) {
@@ -1117,7 +1121,7 @@ NXD_API int nxd_qkv_prep_cache_write(int dtype, const void* qkv, long long ld, v
     NXD_REQUIRE(!value_from_key || Dv == D, "values taken from the keys need equal sizes (%d, %d)", D, Dv);
     NXD_REQUIRE(!(value_from_key && (bias != nullptr || value_norm)), "values taken from the keys: no bias or norm of their %s", "own");
     NXD_REQUIRE(!(writeback && whole_norm && normalize && row_stat == nullptr), "write-back under a whole-row norm needs %s", "row_stat");
-    NXD_REQUIRE(!(writeback && rope_cos != nullptr), "write-back of rotated keys is not %s", "supported");
+    NXD_REQUIRE(!(writeback && value_from_key), "write-back of keys that another warp reads as values is not %s", "supported");
     const CacheAddr ka = make_addr(k_stride_line, k_stride_head, block_table, page_size, table_cols, D);
     const CacheAddr va = make_addr(v_stride_line, v_stride_head, block_table, page_size, table_cols, Dv);
     const int wpb = 8;

@@ -948,3 +948,210 @@ def run_scored(steps: int = 10, warmup: int = 3, device=None, sizes=None) -> dic
         out["kernels"][s["name"]] = scored_kernel_cases(s, steps, warmup, dev)
     out["gpu_launches"] = _lib.kernel_launches() - before
     return out
+
+
+# ---- Mumazen next to Vufasun (attention over the cache beside a recurrent mixer, looped layers, gated feed-forward) -----------
+SSM_STATE, SSM_HEAD, SCAN_STATE = 128, 64, 16          # state-space heads of 128 x 64, selective scan of 16 states per channel
+
+
+def mumazen_config(s: dict):
+    from ..models.mumazen import MumazenConfig
+
+    ff = {"kind": "dense", "ff": (2 * s["ff"] // 3 + 127) // 128 * 128, "limit": 7.0}
+    inner = s["rec_heads"] * s["rec_vdim"]             # as wide as Vufasun's retention heads together
+    par = {"left": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"], "scale": s["dim"] ** -0.5,
+                    "softcap": 30.0, "rot": {"base": 500000.0, "dims": s["dim"] // 2, "scaling": {"factor": 4.0}}},
+           "right": {"heads": inner // SSM_HEAD, "vdim": SSM_HEAD, "state": SSM_STATE, "groups": 1, "conv": 4, "norm_groups": 1},
+           "left_scale": 1.0, "right_scale": 1.0}
+    scan = {"inner": s["width"], "state": SCAN_STATE, "dt_rank": s["width"] // 16, "conv": 4}
+    return MumazenConfig.from_dict({
+        "architecture": "Mumazen", "vocab": VOCAB, "width": s["width"], "embedding": {"scale": 1.0}, "residual_mult": 1.0,
+        "norm": {"eps": 1e-6}, "layers": [{"type": "parallel", "mixer": par, "mlp": ff},
+                                          {"type": "mamba1", "mixer": scan, "mlp": ff},
+                                          {"type": "parallel", "mixer": par, "mlp": ff}]}, torch_dtype=torch.bfloat16)
+
+
+def state_space_serve_case(s: dict, steps: int, warmup: int, dev) -> dict:
+    from .hybrid import MumazenInferenceModel, VufasunInferenceModel
+
+    timer = _Timer(dev)
+    out = {"size": dict(s)}
+    ic = dict(batch_size=s["decode_batch"], max_batch_size=s["decode_batch"], max_context_length=s["prompt"],
+              seq_len=s["prompt"] + 64, is_continuous_batching=True, use_cuda_graphs=False)
+    for name, make in (("mumazen", lambda: MumazenInferenceModel(mumazen_config(s), InferenceConfig(**ic), device=dev)),
+                       ("vufasun", lambda: VufasunInferenceModel(vufasun_config(s), InferenceConfig(**ic), device=dev))):
+        torch.manual_seed(0)
+        model = make()
+        model.init_kv_cache(device=dev)
+        out[name] = _serve(model, s, timer, steps, warmup, dev)
+        out[name]["parameters"] = sum(p.numel() for p in model.parameters())
+        del model
+        torch.cuda.empty_cache()
+    out["mumazen_over_vufasun"] = {k: out["mumazen"][k] / out["vufasun"][k]
+                                   for k in ("prefill_tokens_per_s", "decode_tokens_per_s")}
+    return out
+
+
+def state_space_kernel_cases(s: dict, steps: int, warmup: int, dev) -> List[dict]:
+    """Mumazen's own kernels on the shapes of ``s``, alone, with roofline fractions, each next to the like kernel of the Vufasun
+    family (of Gogalix where Vufasun has none).  The selective scan is as wide as in a layer of its own (twice the width)."""
+    from ..ops import delta_rule as dr
+    from ..ops import hyper_connection as hc_ops
+    from ..ops import mlstm as ml
+    from ..ops import retention as rt
+    from ..ops import rope as rope_ops
+    from ..ops import state_space as ss
+    from ..ops import stream_norm as sn
+
+    pk = peaks()
+    timer = _Timer(dev)
+    bf = torch.bfloat16
+    B, T, H, G, D, W, Bd = s["prefill_batch"], s["prompt"], s["heads"], s["kv_heads"], s["dim"], s["width"], s["decode_batch"]
+    rows = []
+
+    def row(kernel, like, fn, flops=None, nbytes=None):
+        ms = timer(fn, steps, warmup)
+        r = {"kernel": kernel, "like": like, "ms": ms, "peak": pk["source"]}
+        if flops is not None:
+            r["tflops"] = flops / ms / 1e9
+            r["of_peak"] = r["tflops"] / pk["bf16_tflops"]
+        if nbytes is not None:
+            r["gbs"] = nbytes / ms / 1e6
+            r["of_peak"] = r["gbs"] / pk["hbm_gbs"]
+        rows.append(r)
+
+    S, N = T + 64, B * T
+    lines = max(B, Bd)
+    zero = torch.zeros(B, dtype=torch.int32, device=dev)
+    pairs = T * (T + 1) // 2
+    fl = 4.0 * D * pairs * H * B
+    # attention with the cap, next to the same kernels without it
+    q = torch.randn(B, T, H, D, device=dev, dtype=bf)
+    kv = torch.randn(2, B, T, G, D, device=dev, dtype=bf)
+    qp, kp, vp = q.permute(0, 2, 1, 3), kv[0].permute(0, 2, 1, 3), kv[1].permute(0, 2, 1, 3)
+    row("capped attention prefill, tcgen05", "prefill attention", lambda: wa.window_attention_tc(qp, kp, vp, D ** -0.5, softcap=30.0), flops=fl)
+    row("causal attention prefill, tcgen05 (the like kernel)", "prefill attention",
+        lambda: attn_ops.flash_attn_func(qp, kp, vp, softmax_scale=D ** -0.5, causal=True), flops=fl)
+    ck = torch.randn(lines, G, S, D, device=dev, dtype=bf)
+    cv = torch.randn(lines, G, S, D, device=dev, dtype=bf)
+    for name, cap in (("capped attention prefill over the cache, mma.sync", 30.0), ("causal attention prefill over the cache (the like kernel)", None)):
+        row(name, "prefill attention", lambda: wa.window_attention_prefill(q, ck, cv, zero, D ** -0.5, softcap=cap), flops=fl)
+    qd = torch.randn(Bd, H, D, device=dev, dtype=bf)
+    posd = torch.full((Bd,), T, dtype=torch.int32, device=dev)
+    for name, cap in (("capped attention decode", 30.0), ("causal attention decode (the like kernel)", None)):
+        row(name, "decode attention", lambda: wa.window_attention_decode(qd, ck, cv, posd, D ** -0.5, softcap=cap),
+            nbytes=2.0 * (T + 1) * G * 2 * D * Bd)
+    del kv, ck, cv
+    n_qkv = H * D + 2 * G * D
+    wide = torch.randn(B, T, n_qkv, device=dev, dtype=bf)
+    ckw, cvw = torch.zeros(B, G, S, D, device=dev, dtype=bf), torch.zeros(B, G, S, D, device=dev, dtype=bf)
+    rope = rope_ops.build_interleaved_rope_cache(S, D // 2, 500000.0, device=dev, factor=4.0)
+    for name, back in (("slowed rotation of halves + cache write + write-back", True), ("rotation of halves + cache write (the like kernel)", False)):
+        row(name, "projection epilogue", lambda: wa.qk_norm_cache_write(wide, ckw, cvw, zero, H, G, D, D, 1e-6, normalize=False, rope=rope,
+                                                                       rope_layout="halves", writeback=back),
+            nbytes=2.0 * N * (2 * H * D + (5 if back else 4) * G * D))
+    g = torch.randn(N, H * D, device=dev, dtype=bf)
+    o = q.view(N, H * D)
+    row("attention output gate, one number per element", "norm", lambda: ss.gate_norm(o, g, act="sigmoid", mul=0.7), nbytes=2.0 * N * 3 * H * D)
+    del wide, ckw, cvw, q, g
+    # state-space heads next to retention
+    Hr, Dk, Dvr = s["rec_heads"], s["rec_dim"], s["rec_vdim"]
+    inner = Hr * Dvr
+    Hs, Ns, P = inner // SSM_HEAD, SSM_STATE, SSM_HEAD
+    C = inner + 2 * Ns
+    xbc = torch.randn(B, T, C, device=dev, dtype=bf)
+    cw, cb, cst = torch.randn(C, 4, device=dev), torch.randn(C, device=dev), torch.zeros(lines, 3, C, device=dev)
+    row("short convolution + bias + silu + state", "convolution", lambda: ss.conv_silu(xbc, cw, cb, cst, zero), nbytes=4.0 * N * C)
+    Gd, Hd = max(1, C // (4 * Dk) // 2), max(1, C // 2 // Dvr)            # about as many channels
+    Cd = 2 * Gd * Dk + (Hd // Gd * Gd or Gd) * Dvr
+    Hd = Hd // Gd * Gd or Gd
+    big = torch.randn(B, T, Cd, device=dev, dtype=bf)
+    cwd, cstd = torch.randn(Cd, 4, device=dev), torch.zeros(lines, 3, Cd, device=dev)
+    row("short convolution + silu + unit norm + state of the delta rule (the like kernel; fp32 output)", "convolution",
+        lambda: dr.delta_prep(big, (0, Gd * Dk, 2 * Gd * Dk), cwd, cstd, zero, Hd, Gd, Dk, Dvr, 1.0), nbytes=6.0 * N * Cd)
+    del big
+    dt = torch.randn(B, T, Hs, device=dev)
+    vec = [torch.randn(Hs, device=dev) for _ in range(3)]
+    st = torch.zeros(lines, Hs, Ns, P, device=dev)
+    offs = (0, inner, inner + Ns)
+    row("state-space heads, prompt, chunks on tensor cores", "prefill recurrence",
+        lambda: ss.state_space_heads(xbc, offs, dt, *vec, st, zero, 1), flops=4.0 * Ns * P * Hs * N)
+    row("state-space heads, prompt, token by token", "prefill recurrence",
+        lambda: ss.state_space_heads(xbc, offs, dt, *vec, st, zero, 1, impl="scan"), flops=4.0 * Ns * P * Hs * N)
+    ld = 2 * Hr * Dk + 2 * Hr * Dvr
+    pr = torch.randn(B, T, ld, device=dev, dtype=bf) * 0.3
+    dec = torch.full((Hr,), 0.99, device=dev)
+    rst = torch.zeros(lines, Hr, Dk, Dvr, device=dev)
+    rrope = rope_ops.build_interleaved_rope_cache(S, Dk, 500000.0, device=dev)
+    roffs = (0, Hr * Dk, 2 * Hr * Dk)
+    row("retention prompt, chunk-wise (the like kernel)", "prefill recurrence",
+        lambda: rt.retention_chunkwise(pr, roffs, dec, rst, zero, Hr, Dk, Dvr, Dk ** -0.5, rope=rrope), flops=4.0 * Dk * Dvr * Hr * N)
+    xd, dtd = xbc[:1, :1].expand(Bd, 1, C).contiguous(), torch.randn(Bd, 1, Hs, device=dev)
+    row("state-space heads, one token (state read + written)", "decode recurrence",
+        lambda: ss.state_space_heads(xd, offs, dtd, *vec, st, posd, 1), nbytes=8.0 * Ns * P * Hs * Bd)
+    prd = torch.randn(Bd, 1, ld, device=dev, dtype=bf) * 0.3
+    row("retention, one token (the like kernel)", "decode recurrence",
+        lambda: rt.retention_scan(prd, roffs, dec, rst, posd, Hr, Dk, Dvr, Dk ** -0.5, rope=rrope), nbytes=8.0 * Dk * Dvr * Hr * Bd)
+    y, w = torch.randn(N, inner, device=dev), torch.ones(inner, device=dev)
+    row("silu gate, then RMS norm over the row", "norm", lambda: ss.gate_norm(y, pr.view(N, ld)[:, :inner], w, 1, 1e-6), nbytes=8.0 * N * inner)
+    yh = y.view(N, Hr, Dvr)
+    row("unit head norm * silu gate (the like kernel)", "norm",
+        lambda: ml.head_norm_gate(yh, pr.view(N, ld), 0, Hr, Dvr, None, 1e-6, True, bf, gate_act="silu"), nbytes=8.0 * N * inner)
+    del xbc, pr, y, st, rst
+    # selective scan
+    Ci, n = 2 * W, SCAN_STATE
+    x, z = torch.randn(B, T, Ci, device=dev, dtype=bf), torch.randn(B, T, Ci, device=dev, dtype=bf)
+    dts, bc = torch.randn(B, T, Ci, device=dev), torch.randn(B, T, 2 * n, device=dev)
+    a_log, dv = torch.rand(Ci, n, device=dev), torch.randn(2, Ci, device=dev)
+    sst = torch.zeros(lines, Ci, n, device=dev)
+    row("selective scan + gate, prompt", "prefill recurrence",
+        lambda: ss.selective_scan(x, dts, dv[0], bc, 0, n, z, a_log, dv[1], sst, zero), nbytes=float(N * (10 * Ci + 8 * n)))
+    xd, zd, dtd, bcd = (t[:1, :1].expand(Bd, 1, t.shape[2]).contiguous() for t in (x, z, dts, bc))
+    row("selective scan + gate, one token (state read + written)", "decode recurrence",
+        lambda: ss.selective_scan(xd, dtd, dv[0], bcd, 0, n, zd, a_log, dv[1], sst, posd), nbytes=8.0 * Ci * n * Bd)
+    del x, z, dts, bc, sst
+    # the stream
+    x32 = torch.randn(N, W, device=dev)
+    y1 = torch.randn(N, W, device=dev, dtype=bf)
+    v = [torch.ones(W, device=dev) for _ in range(4)]
+    table, ids = torch.randn(VOCAB, W, device=dev, dtype=bf), torch.randint(0, VOCAB, (N,), device=dev)
+    row("layer-scaled residual + output bias + next norm", "norm",
+        lambda: sn.stream_update_(x32, y1, v[0], v[1], w_next=v[2], out_dtype=bf), nbytes=float(N * W * 12))
+    row("the same with the embedding and a pass vector added", "norm",
+        lambda: sn.stream_update_(x32, y1, v[0], v[1], table, ids, 1.0, v[3], v[2], out_dtype=bf), nbytes=float(N * W * 14))
+    xs = torch.randn(N, VUFASUN_STREAMS, W, device=dev)
+    mix, ow = torch.eye(VUFASUN_STREAMS, device=dev), torch.ones(VUFASUN_STREAMS, device=dev)
+    row(f"stream write + mixing + next read and norm, {VUFASUN_STREAMS} streams (the like kernel)", "norm",
+        lambda: hc_ops.hc_step(xs, y1, mix, ow, ow, v[2], 1e-6, bf), nbytes=float(N * W * (8 * VUFASUN_STREAMS + 4)))
+    del xs, x32
+    F = (2 * s["ff"] // 3 + 127) // 128 * 128
+    src, gb = torch.randn(N, 2 * F, device=dev, dtype=bf), torch.zeros(F, device=dev)
+    row("clamped gated activation with biases", "activation",
+        lambda: moe_sparse.glu_bias(src, 0, F, F, gb, gb, limit=7.0, alpha=moe_sparse.GLU_ALPHA, up_shift=1.0), nbytes=6.0 * N * F)
+    row("gelu_tanh(gate) * up (the like kernel)", "activation", lambda: moe_sparse.glu_bias(src, 0, F, F, act="gelu_tanh"), nbytes=6.0 * N * F)
+    del src
+    # sparse feed-forward of token generation: 8 experts, two of them per token
+    E, Fe = 8, W // 2
+    h = torch.randn(Bd, W, device=dev, dtype=bf)
+    wr, corr = torch.randn(E + 4, W, device=dev) * W ** -0.5, torch.zeros(E + 4, device=dev)
+    row("router: normalised scores with identity experts", "router", lambda: moe_sparse.route(h, wr, corr, 2, 1.0, normalize=True), nbytes=4.0 * (E + 4) * W)
+    row("router: sigmoid scores (the like kernel)", "router", lambda: moe_sparse.route(h, wr, None, 2, 1.0, score="sigmoid"), nbytes=4.0 * (E + 4) * W)
+    idx = torch.stack([torch.arange(Bd, device=dev) % E, (torch.arange(Bd, device=dev) + 3) % E], dim=1).to(torch.int32).contiguous()
+    wu, wg = torch.randn(E, W, Fe, device=dev, dtype=bf), torch.randn(E, W, 2 * Fe, device=dev, dtype=bf)
+    row("expert up products + squared relu, per pair", "expert", lambda: moe_sparse.up_act(h, wu, idx), nbytes=2.0 * Bd * 2 * W * Fe)
+    row("expert gate / up products + silu, per pair (the like kernel)", "expert",
+        lambda: moe_sparse.gate_up_act(h, wg, idx, float("inf"), 1.0, 0.0), nbytes=2.0 * Bd * 2 * W * 2 * Fe)
+    return rows
+
+
+def run_state_space(steps: int = 10, warmup: int = 3, device=None, sizes=None) -> dict:
+    dev = device or torch.device("cuda", torch.cuda.current_device())
+    before = _lib.kernel_launches()
+    out = {"metric": "Mumazen vs Vufasun, serving throughput at equal layer sizes", "dtype": "bf16",
+           "data": "synthetic token ids, random-init weights", "steps": steps, "warmup": max(warmup, 3),
+           "l2": "192 MB written between timed runs", "peaks": peaks(), "cases": [], "kernels": {}}
+    for s in (sizes or HYBRID_SIZES):
+        out["cases"].append(state_space_serve_case(s, steps, warmup, dev))
+        out["kernels"][s["name"]] = state_space_kernel_cases(s, steps, warmup, dev)
+    out["gpu_launches"] = _lib.kernel_launches() - before
+    return out
