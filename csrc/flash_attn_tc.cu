@@ -441,10 +441,20 @@ fa_fwd_tc_kernel(const __grid_constant__ CUtensorMap tmap_q, const __grid_consta
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
                 uint32_t w[4];
+                float eg[8];
+                if (WIN && p.mod.gate_cols > 0) {                // one gate number per element
+                    const long long at = ((long long)b * p.Sq + min(grow, p.Sq - 1)) * p.mod.gate_ld + (long long)hq * D + g * 64 + c * 8;
+                    unpack8(*reinterpret_cast<const bf16x8*>(reinterpret_cast<const bf16*>(p.mod.gate) + at), eg);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) eg[e] = p.mod.gate_mul * score::sigmoid(eg[e]) * inv;
+                } else {
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) eg[e] = inv;
+                }
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
-                    bf162 t = __floats2bfloat162_rn(__uint_as_float(o[8 * c + 2 * e]) * inv,
-                                                    __uint_as_float(o[8 * c + 2 * e + 1]) * inv);
+                    bf162 t = __floats2bfloat162_rn(__uint_as_float(o[8 * c + 2 * e]) * eg[2 * e],
+                                                    __uint_as_float(o[8 * c + 2 * e + 1]) * eg[2 * e + 1]);
                     w[e] = *reinterpret_cast<uint32_t*>(&t);
                 }
                 st_shared_v4(dst + ((c ^ (row & 7)) << 4), w[0], w[1], w[2], w[3]);
@@ -555,7 +565,9 @@ NXD_API int nxd_flash_attn_fwd_tc_scored(const void* q, const void* k, const voi
                                          int B, int Hq, int Hkv, int Sq, int Sk, int D, float scale, int window,
                                          int keep_first, const float* slopes, const float* sinks, float softcap,
                                          const float* log_r1, const float* log_r2, const float* sigmoid_bias,
-                                         const void* gate, long long gate_ld, void* stream) {
+                                         const void* gate, long long gate_ld, int gate_cols, float gate_mul, void* stream) {
+    NXD_REQUIRE(gate_cols == 0 || (gate_cols == D && gate != nullptr && gate_ld % 8 == 0 && ((uintptr_t)gate & 15) == 0),
+                "flash_attn_tc: a gate of %d columns per head of %d", gate_cols, D);
     NXD_REQUIRE((log_r1 == nullptr) == (log_r2 == nullptr), "flash_attn_tc: the logarithmic bias needs %s", "both vectors");
     NXD_REQUIRE(sigmoid_bias == nullptr || sinks == nullptr, "flash_attn_tc: sigmoid weights have no %s", "sink");
     NXD_REQUIRE(D == 64 || D == 128, "flash_attn_tc_window: head dim %d not supported (64 or 128)", D);
@@ -575,7 +587,7 @@ NXD_API int nxd_flash_attn_fwd_tc_scored(const void* q, const void* k, const voi
     p.keep_first = keep_first > 0 ? keep_first : 0;
     p.slopes = slopes;
     p.sinks = sinks;
-    p.mod = ScoreMod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld};
+    p.mod = ScoreMod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld, gate_cols, gate_mul, 0};
     const int mode = p.mod.mode();
     if (mode > 0 && (log_r1 != nullptr || slopes != nullptr)) {
         const int span = (window > 0 && window < Sk && p.keep_first == 0) ? window : Sk;      // distances that can be visible
@@ -597,5 +609,5 @@ NXD_API int nxd_flash_attn_fwd_tc_window(const void* q, const void* k, const voi
                                          int B, int Hq, int Hkv, int Sq, int Sk, int D, float scale, int window,
                                          int keep_first, const float* slopes, void* stream) {
     return nxd_flash_attn_fwd_tc_scored(q, k, v, o, strides, B, Hq, Hkv, Sq, Sk, D, scale, window, keep_first, slopes, nullptr,
-                                        0.f, nullptr, nullptr, nullptr, nullptr, 0, stream);
+                                        0.f, nullptr, nullptr, nullptr, nullptr, 0, 0, 1.f, stream);
 }

@@ -414,7 +414,7 @@ NXD_API int nxd_latent_decode(const void* q, const void* cache, long long stride
                               const int* positions, const int* seq_ids, const float* sinks, int B, int H, int D, int Dv,
                               float scale, int nsplit, int window, const void* gate, long long gate_ld, void* stream) {
     if (B == 0) return 0;
-    const ScoreMod mod{0.f, nullptr, nullptr, nullptr, gate, gate_ld};
+    const ScoreMod mod{0.f, nullptr, nullptr, nullptr, gate, gate_ld, 0, 1.f, 0};
     if ((stride_line % 8) || (row_pitch % 8) || ((uintptr_t)cache % 16) || ((uintptr_t)q % 16)) return 2;
     cudaStream_t st = (cudaStream_t)stream;
 #define NXD_LD_CASE(DD, DDV)                                                                                            \

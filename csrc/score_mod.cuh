@@ -5,6 +5,7 @@
 //   log distance     s <- s - r1_h * ln(1 + r2_h * (i - j))                          (r1, r2 != NULL)
 //   sigmoid weights  weight = sigmoid(s + pb_h), not normalised over the keys        (pb != NULL; no softmax, no sink)
 //   output gate      o <- o * sigmoid(gate[row, h])                                  (gate != NULL; one number per head)
+//                    o[c] <- o[c] * sigmoid(gate[row, h, c]) * gate_mul                 (gate_cols > 0: one number per element)
 //
 // tanh in fp32 for |x| < 0.4 is the odd power series up to x^9 (next term below 1e-6 of the value), beyond that
 // 1 - 2 / (1 + exp(2 |x|)); the kernels choose once per tile where they can.  The fp32 kernels take two more terms of the series
@@ -19,6 +20,9 @@ struct ScoreMod {
     const float* pb;
     const void* gate;        // activation dtype; pre-activation of (row n, head h) at gate[n * gate_ld + h]
     long long gate_ld;
+    int gate_cols;           // > 0: value size; pre-activation of (row n, head h, column c) at gate[n * gate_ld + h * gate_cols + c]
+    float gate_mul;          // of the gate per element
+    long long out_ld;        // elements between output rows (0: the heads of a row are all there is in it)
     __host__ __device__ int mode() const { return pb != nullptr ? 2 : ((cap > 0.f || r1 != nullptr) ? 1 : 0); }
 };
 
@@ -65,7 +69,19 @@ __device__ __forceinline__ float ldg(const float* p) { return *p; }
 __device__ __forceinline__ float ldg(const bf16* p) { return __bfloat162float(*p); }
 template <typename T>
 __device__ __forceinline__ float out_gate(const ScoreMod& m, long long row, int h) {
-    return m.gate == nullptr ? 1.f : sigmoid(ldg(reinterpret_cast<const T*>(m.gate) + row * m.gate_ld + h));
+    return (m.gate == nullptr || m.gate_cols > 0) ? 1.f : sigmoid(ldg(reinterpret_cast<const T*>(m.gate) + row * m.gate_ld + h));
 }
+
+template <typename T>
+__device__ __forceinline__ float elem_gate(const ScoreMod& m, long long row, int h, int c) {
+    return m.gate_cols <= 0 ? 1.f : m.gate_mul * sigmoid(ldg(reinterpret_cast<const T*>(m.gate) + row * m.gate_ld + (long long)h * m.gate_cols + c));
+}
+// two neighbouring columns (c even) of a 16-bit gate
+__device__ __forceinline__ float2 elem_gate2(const ScoreMod& m, long long row, int h, int c) {
+    if (m.gate_cols <= 0) return make_float2(1.f, 1.f);
+    const bf16* p = reinterpret_cast<const bf16*>(m.gate) + row * m.gate_ld + (long long)h * m.gate_cols + c;
+    return make_float2(m.gate_mul * sigmoid(ldg(p)), m.gate_mul * sigmoid(ldg(p + 1)));
+}
+__device__ __forceinline__ long long out_pitch(const ScoreMod& m, int columns) { return m.out_ld > 0 ? m.out_ld : columns; }
 
 }  // namespace score

@@ -13,9 +13,10 @@
 // Kernels:
 //   conv_silu          convolution + silu of a column range of a projection; also moves the line's convolution state (the
 //                      last taps - 1 raw inputs) when one thread sees the whole step, else conv_state does it afterwards
-//   selective_scan     states of a channel split over R lanes of NS registers, tokens in double-buffered blocks of 16 through
-//                      shared memory (cp.async); the R partial sums of R consecutive tokens are summed by one transposing
-//                      butterfly; gate, skip term and store once per block.  Prompts and single tokens
+//   selective_scan     states of a channel split over R lanes of NS registers (two channels per thread share the loads of B and
+//                      C), tokens in double-buffered blocks through shared memory (cp.async); the R partial sums of R
+//                      consecutive tokens are summed by one transposing butterfly; step sizes ahead of a block, gate, skip term
+//                      and store behind it.  Prompts and single tokens
 //   ssd_step           one token: a thread owns four neighbouring columns of a head's state, the rows are spread over the
 //                      CTA; the state is read and written once
 //   ssd_scan           token by token, a column's rows split over R lanes (fp32 prompts, short steps, unusual sizes)
@@ -23,7 +24,7 @@
 //                      head with the fp32 state in accumulator registers.  Operands that are products of fp32 numbers (decayed
 //                      scores, scaled inputs, the state) go in as the sum of two bf16 numbers, so that their relative error
 //                      is 2^-17, not 2^-9
-//   gate_norm          y act(z) [* constant], or divided by the root mean square over equal groups of columns and weighted
+//   gate_norm          y act(z), divided by the root mean square over equal groups of columns and weighted
 // This file is compiled without fast-math: the state lives for thousands of steps.
 #include "common.cuh"
 #include "mma_sync.cuh"
@@ -69,9 +70,39 @@ struct ScanDecay<float> {
     static __device__ __forceinline__ float at(float dt, float rate) { return decay_exp(dt * rate); }
 };
 
+// The arithmetic around the recurrences.  fp32 serving takes the library functions; 16-bit serving forms built on the hardware's
+// 2^x and reciprocal, whose relative errors stay near 2^-21: softplus(z) = max(z, 0) + log1p(e^-|z|) with log1p(t) = 2 atanh(t / (2 + t))
+// by its odd power series (t / (2 + t) <= 1/3, next term below 1e-8 of the value)
+template <typename T>
+struct ScanMath {
+    static __device__ __forceinline__ float softplus(float z) {
+        const float t = exp2_ftz(-fabsf(z) * LOG2E);
+        const float s = __fdividef(t, 2.f + t), q = s * s;
+        float p = fmaf(q, 2.f / 15.f, 2.f / 13.f);
+        p = fmaf(q, p, 2.f / 11.f);
+        p = fmaf(q, p, 2.f / 9.f);
+        p = fmaf(q, p, 2.f / 7.f);
+        p = fmaf(q, p, 2.f / 5.f);
+        p = fmaf(q, p, 2.f / 3.f);
+        p = fmaf(q, p, 2.f);
+        return fmaf(s, p, fmaxf(z, 0.f));
+    }
+    static __device__ __forceinline__ float sigmoid(float z) { return __fdividef(1.f, 1.f + exp2_ftz(fminf(-z * LOG2E, 100.f))); }
+    static __device__ __forceinline__ float silu(float z) { return z * sigmoid(z); }
+};
+template <>
+struct ScanMath<float> {
+    static __device__ __forceinline__ float softplus(float z) { return softplus_f(z); }
+    static __device__ __forceinline__ float sigmoid(float z) { return sigmoid_f(z); }
+    static __device__ __forceinline__ float silu(float z) { return silu_f(z); }
+};
+
 template <int VEC>
 __device__ __forceinline__ void ldv(const float* p, float* v) {
-    if (VEC == 4) {
+    if (VEC == 8) {
+        const float4 t = *reinterpret_cast<const float4*>(p), u = *reinterpret_cast<const float4*>(p + 4);
+        v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w, v[4] = u.x, v[5] = u.y, v[6] = u.z, v[7] = u.w;
+    } else if (VEC == 4) {
         const float4 t = *reinterpret_cast<const float4*>(p);
         v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w;
     } else {
@@ -80,7 +111,9 @@ __device__ __forceinline__ void ldv(const float* p, float* v) {
 }
 template <int VEC>
 __device__ __forceinline__ void ldv(const bf16* p, float* v) {
-    if (VEC == 4) {
+    if (VEC == 8) {
+        unpack8(*reinterpret_cast<const bf16x8*>(p), v);
+    } else if (VEC == 4) {
         const uint2 raw = *reinterpret_cast<const uint2*>(p);
         const float2 a = __bfloat1622float2(*reinterpret_cast<const bf162*>(&raw.x));
         const float2 b = __bfloat1622float2(*reinterpret_cast<const bf162*>(&raw.y));
@@ -91,12 +124,17 @@ __device__ __forceinline__ void ldv(const bf16* p, float* v) {
 }
 template <int VEC>
 __device__ __forceinline__ void stv(float* p, const float* v) {
-    if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    if (VEC == 8) {
+        *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+        *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+    } else if (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
     else *p = v[0];
 }
 template <int VEC>
 __device__ __forceinline__ void stv(bf16* p, const float* v) {
-    if (VEC == 4) {
+    if (VEC == 8) {
+        *reinterpret_cast<bf16x8*>(p) = pack8(v);
+    } else if (VEC == 4) {
         uint2 raw;
         *reinterpret_cast<bf162*>(&raw.x) = __floats2bfloat162_rn(v[0], v[1]);
         *reinterpret_cast<bf162*>(&raw.y) = __floats2bfloat162_rn(v[2], v[3]);
@@ -178,7 +216,7 @@ conv_silu_kernel(const T* __restrict__ proj, long long ld, const float* __restri
                 acc[i] = bv[i];
 #pragma unroll
                 for (int j = 0; j < NT; ++j) acc[i] = fmaf(w[j][i], win[j][i], acc[i]);
-                acc[i] = silu_f(acc[i]);
+                acc[i] = ScanMath<TO>::silu(acc[i]);
             }
             stv<VEC>(orow + (long long)t * ld_out, acc);
         }
@@ -193,7 +231,7 @@ conv_silu_kernel(const T* __restrict__ proj, long long ld, const float* __restri
                 for (int i = 0; i < VEC; ++i) acc[i] = fmaf(conv_w[(long long)(c + i) * (K + 1) + j], v[i], acc[i]);
             }
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) acc[i] = silu_f(acc[i]);
+            for (int i = 0; i < VEC; ++i) acc[i] = ScanMath<TO>::silu(acc[i]);
             stv<VEC>(orow + (long long)t * ld_out, acc);
         }
     }
@@ -233,27 +271,33 @@ __device__ __forceinline__ float transpose_sum(float (&v)[R], int r) {
     return v[0];
 }
 
-constexpr int SS_THREADS = 128, SS_TS = 16;
+constexpr int SS_THREADS = 128;
 
-template <typename T, int NS, int R>
+// NS states of each of CPT neighbouring channels per thread, R neighbouring lanes share them; TS tokens per block
+template <typename T, int NS, int R, int CPT, int TS>
+struct ScanSmem {
+    static constexpr int CH = SS_THREADS / R * CPT, NP = NS * R;
+    struct Buf {
+        float B[TS][NP], Cm[TS][NP], dt[TS][CH];
+        T x[TS][CH], z[TS][CH];
+    } buf[2];
+    float u[TS][CH];                                       // dt * x, then sum_n S C
+};
+
+template <typename T, int NS, int R, int CPT, int TS>
 __global__ void __launch_bounds__(SS_THREADS)
 selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __restrict__ dt, long long ld_dt,
                       const float* __restrict__ dt_bias, const float* __restrict__ bc, long long ld_bc, int b_off, int c_off,
                       const T* __restrict__ z, long long ld_z, const float* __restrict__ a_log, const float* __restrict__ dskip,
                       float* __restrict__ S, T* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
                       const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int C, int N, int async) {
-    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS;
+    using Sm = ScanSmem<T, NS, R, CPT, TS>;
+    constexpr int CH = Sm::CH, NP = Sm::NP;
     static_assert(TS % R == 0, "tokens come in groups of R");
-    struct Buf {
-        float B[TS][NP], Cm[TS][NP], dt[TS][CH];
-        T x[TS][CH], z[TS][CH];
-    };
     extern __shared__ __align__(16) unsigned char smem_raw[];
-    Buf* bufs = reinterpret_cast<Buf*>(smem_raw);
-    float(*us)[CH] = reinterpret_cast<float(*)[CH]>(smem_raw + 2 * sizeof(Buf));           // dt * x
-    float(*ys)[CH] = us + TS;                                                                // sum_n S C
-    const int tid = threadIdx.x, r = tid % R, cl = tid / R;
-    const int c0 = blockIdx.x * CH, c = c0 + cl, b = blockIdx.y;
+    Sm& sm = *reinterpret_cast<Sm*>(smem_raw);
+    const int tid = threadIdx.x, r = tid % R, cl = tid / R * CPT;
+    const int c0 = blockIdx.x * CH, b = blockIdx.y;
     const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
     const long long row0 = (long long)b * Tn;
     const int nch = min(CH, C - c0);
@@ -261,27 +305,29 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
         stf(out + (row0 + max(n, 0) + idx / nch) * ld_out + c0 + idx % nch, 0.f);
     if (n <= 0) return;
     const int line = seq_ids != nullptr ? seq_ids[b] : b;
-    float* Sc = S + ((long long)line * C + c) * N;
+    float* Sc = S + ((long long)line * C + c0 + cl) * N;
     const bool fresh = q_start[b] == 0;
-    float s[NS], a2[NS];
+    float s[CPT][NS], a2[CPT][NS];
 #pragma unroll
-    for (int j = 0; j < NS; ++j) {
-        const int i = r * NS + j;
-        const bool ok = c < C && i < N;
-        s[j] = (ok && !fresh) ? Sc[i] : 0.f;
-        a2[j] = ok ? ScanDecay<T>::rate(-expf(a_log[(long long)c * N + i])) : 0.f;
-    }
+    for (int k = 0; k < CPT; ++k)
+#pragma unroll
+        for (int j = 0; j < NS; ++j) {
+            const int i = r * NS + j;
+            const bool ok = cl + k < nch && i < N;
+            s[k][j] = (ok && !fresh) ? Sc[(long long)k * N + i] : 0.f;
+            a2[k][j] = ok ? ScanDecay<T>::rate(-expf(a_log[(long long)(c0 + cl + k) * N + i])) : 0.f;
+        }
     // columns N .. NP - 1 of B and C are zeros in both buffers and stay so
     if (N < NP)
         for (int idx = tid; idx < 2 * TS * (NP - N); idx += SS_THREADS) {
             const int k = idx / (TS * (NP - N)), q = idx % (TS * (NP - N));
-            bufs[k].B[q / (NP - N)][N + q % (NP - N)] = 0.f;
-            bufs[k].Cm[q / (NP - N)][N + q % (NP - N)] = 0.f;
+            sm.buf[k].B[q / (NP - N)][N + q % (NP - N)] = 0.f;
+            sm.buf[k].Cm[q / (NP - N)][N + q % (NP - N)] = 0.f;
         }
     constexpr int XV = 16 / sizeof(T);                       // elements of T per 16 bytes
     constexpr int CX = CH / XV;                              // such pieces per token
     auto fetch = [&](int t0, int k) {
-        Buf& d = bufs[k];
+        typename Sm::Buf& d = sm.buf[k];
         const int cnt = min(TS, n - t0);
         if (async) {
             for (int idx = tid; idx < cnt * (N / 4); idx += SS_THREADS) {
@@ -321,9 +367,19 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
         mma::cp_async_commit();
     };
     fetch(0, 0);
+    // a thread prepares and finishes VP neighbouring channels of every (128 VP / CH)-th token, always the same channels
+    constexpr int VP = 2, PT = CH / VP, ROWS = SS_THREADS / PT;
+    static_assert(SS_THREADS % PT == 0 && CH % VP == 0, "channel slices");
+    const int pi = tid % PT * VP, prow = tid / PT;
+    float bias[VP], dsk[VP];
+#pragma unroll
+    for (int v = 0; v < VP; ++v) {
+        bias[v] = (dt_bias != nullptr && pi + v < nch) ? dt_bias[c0 + pi + v] : 0.f;
+        dsk[v] = pi + v < nch ? dskip[c0 + pi + v] : 0.f;
+    }
     int k = 0;
     for (int t0 = 0; t0 < n; t0 += TS, k ^= 1) {
-        const int cnt = min(TS, n - t0);
+        const int cnt = min(TS, n - t0), top = (cnt + R - 1) / R * R;
         if (t0 + TS < n) {
             fetch(t0 + TS, k ^ 1);
             mma::cp_async_wait<1>();
@@ -331,79 +387,93 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
             mma::cp_async_wait<0>();
         }
         __syncthreads();
-        Buf& d = bufs[k];
-        for (int idx = tid; idx < TS * CH; idx += SS_THREADS) {          // step sizes; tokens past the end: no step
-            const int tt = idx / CH, i = idx % CH;
-            float v = 0.f, u = 0.f;
-            if (tt < cnt && i < nch) {
-                v = softplus_f(d.dt[tt][i] + (dt_bias != nullptr ? dt_bias[c0 + i] : 0.f));
-                u = v * ldf(&d.x[tt][i]);
+        typename Sm::Buf& d = sm.buf[k];
+        for (int tt = prow; tt < top; tt += ROWS) {                      // step sizes; tokens past the end: no step
+#pragma unroll
+            for (int v = 0; v < VP; ++v) {
+                const bool ok = tt < cnt && pi + v < nch;
+                const float step = ok ? ScanMath<T>::softplus(d.dt[tt][pi + v] + bias[v]) : 0.f;
+                d.dt[tt][pi + v] = step;
+                sm.u[tt][pi + v] = ok ? step * ldf(&d.x[tt][pi + v]) : 0.f;
             }
-            d.dt[tt][i] = v;
-            us[tt][i] = u;
         }
-        if (cnt < TS)                                                    // rows that no copy has filled
-            for (int idx = tid; idx < (TS - cnt) * N; idx += SS_THREADS) {
-                d.B[cnt + idx / N][idx % N] = 0.f;
-                d.Cm[cnt + idx / N][idx % N] = 0.f;
-            }
+        for (int idx = tid; idx < (top - cnt) * N; idx += SS_THREADS) {  // rows that no copy has filled
+            d.B[cnt + idx / N][idx % N] = 0.f;
+            d.Cm[cnt + idx / N][idx % N] = 0.f;
+        }
         __syncthreads();
-        for (int g0 = 0; g0 < cnt; g0 += R) {
-            float y[R];
+        for (int g0 = 0; g0 < top; g0 += R) {
+            float y[CPT][R];
 #pragma unroll
             for (int q = 0; q < R; ++q) {
-                const float dv = d.dt[g0 + q][cl], u = us[g0 + q][cl];
-                float acc[2] = {0.f, 0.f};
+                float dv[CPT], u[CPT], acc[CPT];
+#pragma unroll
+                for (int m = 0; m < CPT; ++m) dv[m] = d.dt[g0 + q][cl + m], u[m] = sm.u[g0 + q][cl + m], acc[m] = 0.f;
 #pragma unroll
                 for (int j = 0; j < NS; j += 4) {
                     const float4 bv = *reinterpret_cast<const float4*>(&d.B[g0 + q][r * NS + j]);
                     const float4 cv = *reinterpret_cast<const float4*>(&d.Cm[g0 + q][r * NS + j]);
-                    s[j] = fmaf(ScanDecay<T>::at(dv, a2[j]), s[j], u * bv.x);
-                    s[j + 1] = fmaf(ScanDecay<T>::at(dv, a2[j + 1]), s[j + 1], u * bv.y);
-                    s[j + 2] = fmaf(ScanDecay<T>::at(dv, a2[j + 2]), s[j + 2], u * bv.z);
-                    s[j + 3] = fmaf(ScanDecay<T>::at(dv, a2[j + 3]), s[j + 3], u * bv.w);
-                    acc[0] = fmaf(s[j], cv.x, acc[0]);
-                    acc[1] = fmaf(s[j + 1], cv.y, acc[1]);
-                    acc[0] = fmaf(s[j + 2], cv.z, acc[0]);
-                    acc[1] = fmaf(s[j + 3], cv.w, acc[1]);
+#pragma unroll
+                    for (int m = 0; m < CPT; ++m) {
+                        s[m][j] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j]), s[m][j], u[m] * bv.x);
+                        s[m][j + 1] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j + 1]), s[m][j + 1], u[m] * bv.y);
+                        s[m][j + 2] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j + 2]), s[m][j + 2], u[m] * bv.z);
+                        s[m][j + 3] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j + 3]), s[m][j + 3], u[m] * bv.w);
+                        acc[m] += fmaf(s[m][j], cv.x, s[m][j + 1] * cv.y) + fmaf(s[m][j + 2], cv.z, s[m][j + 3] * cv.w);
+                    }
                 }
-                y[q] = acc[0] + acc[1];
+#pragma unroll
+                for (int m = 0; m < CPT; ++m) y[m][q] = acc[m];
             }
-            ys[g0 + r][cl] = transpose_sum<R>(y, r);
+            // every lane of the channel has read its u of these tokens (the shuffles wait for them): y takes their place
+#pragma unroll
+            for (int m = 0; m < CPT; ++m) {
+                const float v = transpose_sum<R>(y[m], r);
+                if (R == 1) __syncwarp();
+                sm.u[g0 + r][cl + m] = v;
+            }
         }
         __syncthreads();
-        for (int idx = tid; idx < cnt * CH; idx += SS_THREADS) {
-            const int tt = idx / CH, i = idx % CH;
-            if (i < nch) {
-                const float xv = ldf(&d.x[tt][i]);
-                stf(out + (row0 + t0 + tt) * ld_out + c0 + i, (ys[tt][i] + dskip[c0 + i] * xv) * silu_f(ldf(&d.z[tt][i])));
+        for (int tt = prow; tt < cnt; tt += ROWS) {
+            float v[VP];
+#pragma unroll
+            for (int w = 0; w < VP; ++w)
+                v[w] = fmaf(dsk[w], ldf(&d.x[tt][pi + w]), sm.u[tt][pi + w]) * ScanMath<T>::silu(ldf(&d.z[tt][pi + w]));
+            T* dst = out + (row0 + t0 + tt) * ld_out + c0 + pi;
+            if (async && pi + 1 < nch) {
+                if (sizeof(T) == 4) *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
+                else *reinterpret_cast<uint32_t*>(dst) = mma::pack2(v[0], v[1]);
+            } else {
+#pragma unroll
+                for (int w = 0; w < VP; ++w)
+                    if (pi + w < nch) stf(dst + w, v[w]);
             }
         }
-        __syncthreads();                                                 // everyone is done with this buffer, us and ys
+        __syncthreads();                                                 // everyone is done with this buffer and with u
     }
-    if (c < C) {
+#pragma unroll
+    for (int m = 0; m < CPT; ++m)
 #pragma unroll
         for (int j = 0; j < NS; ++j) {
             const int i = r * NS + j;
-            if (i < N) Sc[i] = s[j];
+            if (cl + m < nch && i < N) Sc[(long long)m * N + i] = s[m][j];
         }
-    }
 }
 
-template <typename T, int NS, int R>
+template <typename T, int NS, int R, int CPT, int TS>
 int launch_selective(const void* x, long long ld_x, const float* dt, long long ld_dt, const float* dt_bias, const float* bc,
                      long long ld_bc, int b_off, int c_off, const void* z, long long ld_z, const float* a_log,
                      const float* dskip, float* S, void* out, long long ld_out, const int* q_start, const int* n_new,
                      const int* seq_ids, int B, int Tn, int C, int N, cudaStream_t st) {
-    constexpr int CH = SS_THREADS / R, NP = NS * R, TS = SS_TS;
-    constexpr size_t smem = 2 * (size_t)TS * (2 * NP * 4 + CH * 4 + 2 * CH * sizeof(T)) + 2 * (size_t)TS * CH * 4;
+    using Sm = ScanSmem<T, NS, R, CPT, TS>;
+    constexpr size_t smem = sizeof(Sm);
     auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
     constexpr int XV = 16 / sizeof(T);
-    const int async = CH % XV == 0 && C % XV == 0 && ld_x % XV == 0 && ld_z % XV == 0 && ld_dt % 4 == 0 && ld_bc % 4 == 0 &&
-                      b_off % 4 == 0 && c_off % 4 == 0 && N % 4 == 0 && al(x) && al(z) && al(dt) && al(bc);
-    auto kern = selective_scan_kernel<T, NS, R>;
+    const int async = Sm::CH % XV == 0 && C % XV == 0 && ld_x % XV == 0 && ld_z % XV == 0 && ld_out % XV == 0 && ld_dt % 4 == 0 &&
+                      ld_bc % 4 == 0 && b_off % 4 == 0 && c_off % 4 == 0 && N % 4 == 0 && al(x) && al(z) && al(dt) && al(bc) && al(out);
+    auto kern = selective_scan_kernel<T, NS, R, CPT, TS>;
     if (smem > 48 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    dim3 grid((C + CH - 1) / CH, B);
+    dim3 grid((C + Sm::CH - 1) / Sm::CH, B);
     kern<<<grid, SS_THREADS, smem, st>>>((const T*)x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, (const T*)z, ld_z, a_log,
                                          dskip, S, (T*)out, ld_out, q_start, n_new, seq_ids, Tn, C, N, async);
     NXD_LAUNCH_CHECK();
@@ -411,13 +481,15 @@ int launch_selective(const void* x, long long ld_x, const float* dt, long long l
 }
 
 // ---- state-space heads: one token ------------------------------------------------------------------------------------------
-// blockIdx.x: slice of 32 columns, y: head, z: row.  A thread owns VEC neighbouring columns and every ROWS-th state row.
+// blockIdx.x: slice of 32 columns, y: head, z: row.  A thread owns VEC neighbouring columns and every ROWS-th state row.  With
+// dt == NULL the CTA makes its head's step size itself, <dt_w[h], hin[row]> over the layer's W inputs.
 template <typename T, typename TY, int VEC>
 __global__ void __launch_bounds__(128)
 ssd_step_kernel(const T* __restrict__ xbc, long long ld, int x_off, int b_off, int c_off, const float* __restrict__ dt,
                 long long ld_dt, const float* __restrict__ dt_bias, const float* __restrict__ a_log,
                 const float* __restrict__ dskip, float* __restrict__ S, TY* __restrict__ y, const int* __restrict__ q_start,
-                const int* __restrict__ seq_ids, int H, int G, int N, int P) {
+                const int* __restrict__ seq_ids, int H, int G, int N, int P, const T* __restrict__ hin,
+                const T* __restrict__ dt_w, int W) {
     constexpr int LC = 32 / VEC, ROWS = 128 / LC;              // lanes per row, rows in flight
     extern __shared__ float smem[];
     float* Bs = smem;                                          // [N]
@@ -430,7 +502,28 @@ ssd_step_kernel(const T* __restrict__ xbc, long long ld, int x_off, int b_off, i
         Bs[i] = ldf(row + b_off + g * N + i);
         Cs[i] = ldf(row + c_off + g * N + i);
     }
-    const float step = softplus_f(dt[(long long)b * ld_dt + h] + (dt_bias != nullptr ? dt_bias[h] : 0.f));
+    float pre = 0.f;
+    if (dt != nullptr) {
+        pre = dt[(long long)b * ld_dt + h];
+    } else {
+        const T* hr = hin + (long long)b * W;
+        const T* wr = dt_w + (long long)h * W;
+        if (W % 8 == 0) {
+#pragma unroll 2
+            for (int c = tid * 8; c < W; c += 128 * 8) {
+                float u8[8], w8[8];
+                ldv<8>(hr + c, u8);
+                ldv<8>(wr + c, w8);
+#pragma unroll
+                for (int i = 0; i < 8; ++i) pre = fmaf(u8[i], w8[i], pre);
+            }
+        } else {
+            for (int c = tid; c < W; c += 128) pre = fmaf(ldf(hr + c), ldf(wr + c), pre);
+        }
+        pre = block_sum(pre, &red[0][0]);
+        __syncthreads();                                       // red is used again below
+    }
+    const float step = softplus_f(pre + (dt_bias != nullptr ? dt_bias[h] : 0.f));
     const float decay = decay_exp(-expf(a_log[h]) * step);
     const bool fresh = q_start[b] == 0, ok = p0 < P;
     const int line = seq_ids != nullptr ? seq_ids[b] : b;
@@ -844,7 +937,7 @@ __global__ void gate_norm_kernel(const TY* __restrict__ y, long long ld_y, const
         ldv<VEC>(yr + c, t);
         ldv<VEC>(zr + c, g);
 #pragma unroll
-        for (int i = 0; i < VEC; ++i) t[i] *= act == 1 ? silu_f(g[i]) : sigmoid_f(g[i]);
+        for (int i = 0; i < VEC; ++i) t[i] *= act == 1 ? ScanMath<T>::silu(g[i]) : ScanMath<T>::sigmoid(g[i]);
     };
 #pragma unroll
     for (int k = 0; k < RV; ++k) {
@@ -881,37 +974,15 @@ __global__ void gate_norm_kernel(const TY* __restrict__ y, long long ld_y, const
     }
 }
 
-// out = y act(z) mul, no norm
-template <typename TY, typename T, int VEC>
-__global__ void gate_mul_kernel(const TY* __restrict__ y, long long ld_y, const T* __restrict__ z, long long ld_z,
-                                T* __restrict__ out, long long ld_out, int n, float mul, int act) {
-    const long long row = blockIdx.x;
-    for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC; c < n; c += gridDim.y * blockDim.x * VEC) {
-        float t[VEC], g[VEC];
-        ldv<VEC>(y + row * ld_y + c, t);
-        ldv<VEC>(z + row * ld_z + c, g);
-#pragma unroll
-        for (int i = 0; i < VEC; ++i) t[i] *= (act == 1 ? silu_f(g[i]) : sigmoid_f(g[i])) * mul;
-        stv<VEC>(out + row * ld_out + c, t);
-    }
-}
-
 template <typename TY, typename T>
 int launch_gate(const void* y, long long ld_y, const void* z, long long ld_z, const float* w, void* out, long long ld_out,
-                long long rows, int n, int groups, float eps, float mul, int act, bool vec, cudaStream_t st) {
-    const int gs = groups > 0 ? n / groups : n;
-    if (groups > 0) {
-        const int per = vec ? 4 : 1;
-        int threads = 32;
-        while (threads < 256 && threads * per * 2 < gs) threads <<= 1;
-        dim3 grid((unsigned)rows, groups);
-        if (vec) gate_norm_kernel<TY, T, 4><<<grid, threads, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, w, (T*)out, ld_out, gs, eps, act);
-        else gate_norm_kernel<TY, T, 1><<<grid, threads, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, w, (T*)out, ld_out, gs, eps, act);
-    } else {
-        dim3 grid((unsigned)rows, (n + 1023) / 1024);
-        if (vec) gate_mul_kernel<TY, T, 4><<<grid, 256, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, (T*)out, ld_out, n, mul, act);
-        else gate_mul_kernel<TY, T, 1><<<grid, 256, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, (T*)out, ld_out, n, mul, act);
-    }
+                long long rows, int n, int groups, float eps, int act, bool vec, cudaStream_t st) {
+    const int gs = n / groups, per = vec ? 4 : 1;
+    int threads = 32;
+    while (threads < 256 && threads * per * 2 < gs) threads <<= 1;
+    dim3 grid((unsigned)rows, groups);
+    if (vec) gate_norm_kernel<TY, T, 4><<<grid, threads, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, w, (T*)out, ld_out, gs, eps, act);
+    else gate_norm_kernel<TY, T, 1><<<grid, threads, 0, st>>>((const TY*)y, ld_y, (const T*)z, ld_z, w, (T*)out, ld_out, gs, eps, act);
     NXD_LAUNCH_CHECK();
     return 0;
 }
@@ -933,7 +1004,9 @@ NXD_API int nxd_conv_silu(int dtype, int out_dtype, const void* proj, long long 
     const bool vec = C % 4 == 0 && ld % 4 == 0 && ld_out % 4 == 0 && al(proj) && al(out) && al(conv_state);
     // few tokens: one thread walks the whole step and moves the state itself
     const int TT = Tn <= 64 ? Tn : 32, move = Tn <= 64 ? 1 : 0;
-    dim3 grid((C + 128 * (vec ? 4 : 1) - 1) / (128 * (vec ? 4 : 1)), (Tn + TT - 1) / TT, B);
+    const bool wide = vec && !move && dtype == 0 && out_dtype == 0 && taps == 4 && C % 8 == 0 && ld % 8 == 0 && ld_out % 8 == 0;
+    const int width = 128 * (wide ? 8 : (vec ? 4 : 1));
+    dim3 grid((C + width - 1) / width, (Tn + TT - 1) / TT, B);
     NXD_REQUIRE(grid.y < 65536, "short convolution: %d tokens", Tn);
 #define NXD_CONV(T, TO, V, K)                                                                                            \
     conv_silu_kernel<T, TO, V, K><<<grid, 128, 0, st>>>((const T*)proj, ld, conv_w, bias, conv_state, (TO*)out, ld_out,    \
@@ -943,7 +1016,8 @@ NXD_API int nxd_conv_silu(int dtype, int out_dtype, const void* proj, long long 
         if (taps == 4) { if (vec) NXD_CONV(T, TO, 4, 4); else NXD_CONV(T, TO, 1, 4); }                                    \
         else { if (vec) NXD_CONV(T, TO, 4, 0); else NXD_CONV(T, TO, 1, 0); }                                              \
     } while (0)
-    if (dtype == 0 && out_dtype == 0) NXD_CONV_T(bf16, bf16);
+    if (wide) NXD_CONV(bf16, bf16, 8, 4);
+    else if (dtype == 0 && out_dtype == 0) NXD_CONV_T(bf16, bf16);
     else if (dtype == 0) NXD_CONV_T(bf16, float);
     else { NXD_REQUIRE(out_dtype == 1, "short convolution: fp32 input, 16-bit output"); NXD_CONV_T(float, float); }
 #undef NXD_CONV_T
@@ -969,19 +1043,20 @@ NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const f
     NXD_REQUIRE(N >= 1 && N <= 512, "selective scan: %d states per channel", N);
     NXD_REQUIRE(B < 65536, "selective scan: %d rows", B);
     cudaStream_t st = (cudaStream_t)stream;
-#define NXD_SEL(T, NS_, R_)                                                                                              \
-    return launch_selective<T, NS_, R_>(x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, z, ld_z, a_log, dskip, S, out, \
-                                        ld_out, q_start, n_new, seq_ids, B, Tn, C, N, st)
+#define NXD_SEL(T, NS_, R_, CPT_, TS_)                                                                                   \
+    return launch_selective<T, NS_, R_, CPT_, TS_>(x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, z, ld_z, a_log,  \
+                                                   dskip, S, out, ld_out, q_start, n_new, seq_ids, B, Tn, C, N, st)
 #define NXD_SEL_T(T)                                                                                                     \
     do {                                                                                                                 \
-        if (N <= 4) NXD_SEL(T, 4, 1);                                                                                    \
-        if (N <= 8) NXD_SEL(T, 4, 2);                                                                                    \
-        if (N <= 16) NXD_SEL(T, 4, 4);                                                                                   \
-        if (N <= 32) NXD_SEL(T, 8, 4);                                                                                   \
-        if (N <= 64) NXD_SEL(T, 8, 8);                                                                                   \
-        if (N <= 128) NXD_SEL(T, 16, 8);                                                                                 \
-        if (N <= 256) NXD_SEL(T, 16, 16);                                                                                \
-        NXD_SEL(T, 32, 16);                                                                                              \
+        if (N <= 4) NXD_SEL(T, 4, 1, 1, 16);                                                                             \
+        if (N <= 8) NXD_SEL(T, 4, 2, 2, 16);                                                                             \
+        if (N <= 16 && Tn > 1) NXD_SEL(T, 4, 4, 2, 32);                                                                  \
+        if (N <= 16) NXD_SEL(T, 4, 4, 1, 16);                                                                            \
+        if (N <= 32) NXD_SEL(T, 8, 4, 1, 16);                                                                            \
+        if (N <= 64) NXD_SEL(T, 8, 8, 1, 16);                                                                            \
+        if (N <= 128) NXD_SEL(T, 16, 8, 1, 16);                                                                          \
+        if (N <= 256) NXD_SEL(T, 16, 16, 1, 16);                                                                         \
+        NXD_SEL(T, 32, 16, 1, 16);                                                                                       \
     } while (0)
     if (dtype == 0) NXD_SEL_T(bf16);
     NXD_SEL_T(float);
@@ -991,11 +1066,13 @@ NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const f
 
 // xbc [B * Tn, ld] (dtype): x [H, P] at column x_off, B and C [G, N] at b_off and c_off (after the convolution); dt fp32
 // pre-activations [B * Tn, ld_dt], one per head; dt_bias (or NULL), a_log, dskip fp32 [H]; S fp32 [lines, H, N, P] in place;
-// y [B * Tn, H, P] (y_dtype).  impl: 0 choose, 1 token by token, 2 chunks on the tensor cores (an error where they do not apply).
+// y [B * Tn, H, P] (y_dtype).  dt NULL (one token per row): the pre-activations are hin [B, W] times the rows of dt_w [H, W], both
+// of the type of xbc.  impl: 0 choose, 1 token by token, 2 chunks on the tensor cores (an error where they do not apply).
 NXD_API int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long long ld, int x_off, int b_off, int c_off,
                                   const float* dt, long long ld_dt, const float* dt_bias, const float* a_log,
                                   const float* dskip, float* S, void* y, const int* q_start, const int* n_new,
-                                  const int* seq_ids, int B, int Tn, int H, int G, int N, int P, int impl, void* stream) {
+                                  const int* seq_ids, int B, int Tn, int H, int G, int N, int P, int impl,
+                                  const void* hin, const void* dt_w, int W, void* stream) {
     if ((long long)B * Tn * H * P == 0) return 0;
     NXD_REQUIRE(G > 0 && H % G == 0, "state-space heads: %d heads over %d groups", H, G);
     NXD_REQUIRE(N >= 1 && N <= 1024, "state-space heads: state size %d", N);
@@ -1003,13 +1080,16 @@ NXD_API int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long 
     NXD_REQUIRE(y_dtype == 1 || y_dtype == dtype, "state-space heads: output type");
     cudaStream_t st = (cudaStream_t)stream;
     auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
-    if (Tn == 1 && n_new == nullptr && impl == 0) {
+    const bool single = Tn == 1 && n_new == nullptr && impl == 0;
+    NXD_REQUIRE(dt != nullptr || (single && hin != nullptr && dt_w != nullptr), "state-space heads: %s", "no step sizes");
+    NXD_REQUIRE(dt != nullptr || W % 8 != 0 || (al(hin) && al(dt_w)), "state-space heads: %s", "unaligned inputs of the step sizes");
+    if (single) {
         const bool vec = P % 4 == 0 && al(S);
         dim3 grid((P + 31) / 32, H, B);
         const size_t smem = (size_t)2 * N * sizeof(float);
 #define NXD_STEP(T, TY, V)                                                                                               \
     ssd_step_kernel<T, TY, V><<<grid, 128, smem, st>>>((const T*)xbc, ld, x_off, b_off, c_off, dt, ld_dt, dt_bias, a_log, \
-                                                       dskip, S, (TY*)y, q_start, seq_ids, H, G, N, P)
+                                                       dskip, S, (TY*)y, q_start, seq_ids, H, G, N, P, (const T*)hin, (const T*)dt_w, W)
         if (dtype == 1) { if (vec) NXD_STEP(float, float, 4); else NXD_STEP(float, float, 1); }
         else if (y_dtype == 1) { if (vec) NXD_STEP(bf16, float, 4); else NXD_STEP(bf16, float, 1); }
         else { if (vec) NXD_STEP(bf16, bf16, 4); else NXD_STEP(bf16, bf16, 1); }
@@ -1066,19 +1146,18 @@ NXD_API int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long 
     return 0;
 }
 
-// y [rows, ld_y] (y_dtype: 0 bf16, 1 fp32), z and out [rows, ...] (dtype): act 0 sigmoid, 1 silu.  groups > 0: v = y act(z),
-// every one of the groups of n / groups columns divided by sqrt(mean(v^2) + eps), times w fp32 [n].  groups == 0: y act(z) mul.
+// y [rows, ld_y] (y_dtype: 0 bf16, 1 fp32), z and out [rows, ...] (dtype): v = y act(z) (act 0 sigmoid, 1 silu), every one of the
+// groups of n / groups columns divided by sqrt(mean(v^2) + eps), times w fp32 [n].
 NXD_API int nxd_gate_norm(int y_dtype, int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w,
-                          void* out, long long ld_out, long long rows, int n, int groups, float eps, float mul, int act,
-                          void* stream) {
+                          void* out, long long ld_out, long long rows, int n, int groups, float eps, int act, void* stream) {
     if (rows * n == 0) return 0;
     NXD_REQUIRE(rows < (1ll << 31), "gate: %lld rows", rows);
-    NXD_REQUIRE(groups == 0 || (n % groups == 0 && groups < 65536), "gate: %d columns in %d groups", n, groups);
+    NXD_REQUIRE(groups > 0 && n % groups == 0 && groups < 65536, "gate: %d columns in %d groups", n, groups);
+    NXD_REQUIRE(dtype == 0 || y_dtype == 1, "gate: %s", "16-bit input, fp32 gate");
     auto al = [](const void* p) { return ((uintptr_t)p % 16) == 0; };
-    const int gs = groups > 0 ? n / groups : n;
-    const bool vec = gs % 4 == 0 && ld_y % 4 == 0 && ld_z % 4 == 0 && ld_out % 4 == 0 && al(y) && al(z) && al(out) && al(w);
+    const bool vec = (n / groups) % 4 == 0 && ld_y % 4 == 0 && ld_z % 4 == 0 && ld_out % 4 == 0 && al(y) && al(z) && al(out) && al(w);
     cudaStream_t st = (cudaStream_t)stream;
-    if (dtype == 1) { NXD_REQUIRE(y_dtype == 1, "gate: 16-bit input, fp32 gate"); return launch_gate<float, float>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, mul, act, vec, st); }
-    if (y_dtype == 1) return launch_gate<float, bf16>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, mul, act, vec, st);
-    return launch_gate<bf16, bf16>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, mul, act, vec, st);
+    if (dtype == 1) return launch_gate<float, float>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, act, vec, st);
+    if (y_dtype == 1) return launch_gate<float, bf16>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, act, vec, st);
+    return launch_gate<bf16, bf16>(y, ld_y, z, ld_z, w, out, ld_out, rows, n, groups, eps, act, vec, st);
 }

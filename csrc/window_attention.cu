@@ -204,7 +204,7 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
     const int nb = n_new != nullptr ? min(n_new[b], Tn) : Tn;
     const int qi = tid >> 3, sub = tid & 7;
     const int nc = (Dv + 7) >> 3;
-    T* orow = out + (((long long)b * Tn + q0 + qi) * H + h) * Dv;
+    T* orow = out + ((long long)b * Tn + q0 + qi) * score::out_pitch(mod, H * Dv) + (long long)h * Dv;
     if (q0 >= nb) {                          // a tile of padding rows: defined output, no work
         if (q0 + qi < Tn)
             for (int m = 0; m < nc; ++m) {
@@ -309,7 +309,7 @@ window_attn_prefill_kernel(const T* __restrict__ q, const T* __restrict__ cache_
         for (int m = 0; m < MAXC; ++m) {
             if (m < nc) {
                 const int c = sub + 8 * m;
-                if (c < Dv) stf(orow + c, acc[m] * inv);
+                if (c < Dv) stf(orow + c, acc[m] * inv * score::elem_gate<T>(mod, (long long)b * Tn + q0 + qi, h, c));
             }
         }
     }
@@ -349,7 +349,7 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
         for (int idx = tid; idx < MQ * (DV / 2); idx += M_THREADS) {
             const int r = idx / (DV / 2), c = idx - r * (DV / 2);
             if (q0 + r < Tn)
-                *reinterpret_cast<uint32_t*>(out + (((long long)b * Tn + q0 + r) * H + h) * DV + 2 * c) = 0u;
+                *reinterpret_cast<uint32_t*>(out + ((long long)b * Tn + q0 + r) * score::out_pitch(mod, H * DV) + (long long)h * DV + 2 * c) = 0u;
         }
         return;
     }
@@ -604,12 +604,18 @@ window_attn_prefill_mma_kernel(const bf16* __restrict__ q, const bf16* __restric
         if (ok0) i0 *= score::out_gate<bf16>(mod, (long long)b * Tn + q0 + r_lo, h);
         if (ok1) i1 *= score::out_gate<bf16>(mod, (long long)b * Tn + q0 + r_lo + 8, h);
     }
-    bf16* out0 = out + (((long long)b * Tn + q0 + r_lo) * H + h) * DV + (lane & 3) * 2;
-    bf16* out1 = out0 + (long long)8 * H * DV;
+    const long long pitch = score::out_pitch(mod, H * DV), row_a = (long long)b * Tn + q0 + r_lo;
+    bf16* out0 = out + row_a * pitch + (long long)h * DV + (lane & 3) * 2;
+    bf16* out1 = out0 + 8 * pitch;
 #pragma unroll
     for (int i = 0; i < DV / 8; ++i) {
-        if (q0 + r_lo < Tn) *reinterpret_cast<uint32_t*>(out0 + i * 8) = mma::pack2(o[i][0] * i0, o[i][1] * i0);
-        if (q0 + r_lo + 8 < Tn) *reinterpret_cast<uint32_t*>(out1 + i * 8) = mma::pack2(o[i][2] * i1, o[i][3] * i1);
+        float2 ga = make_float2(1.f, 1.f), gb = ga;
+        if (mod.gate_cols > 0) {
+            if (ok0) ga = score::elem_gate2(mod, row_a, h, (lane & 3) * 2 + i * 8);
+            if (ok1) gb = score::elem_gate2(mod, row_a + 8, h, (lane & 3) * 2 + i * 8);
+        }
+        if (q0 + r_lo < Tn) *reinterpret_cast<uint32_t*>(out0 + i * 8) = mma::pack2(o[i][0] * i0 * ga.x, o[i][1] * i0 * ga.y);
+        if (q0 + r_lo + 8 < Tn) *reinterpret_cast<uint32_t*>(out1 + i * 8) = mma::pack2(o[i][2] * i1 * gb.x, o[i][3] * i1 * gb.y);
     }
 }
 
@@ -743,7 +749,8 @@ window_attn_decode_kernel(const T* __restrict__ q, const T* __restrict__ cache_k
         if (sinks != nullptr) den += expf(sinks[h0 + r] - (mx == -INFINITY ? 0.f : mx));
         if (sig) den = 1.f;
         const float y = den > 0.f ? num / den : 0.f;
-        stf(out + ((long long)b * H + h0 + r) * Dv + c, y * score::out_gate<T>(mod, b, h0 + r));
+        stf(out + (long long)b * score::out_pitch(mod, H * Dv) + (long long)(h0 + r) * Dv + c,
+            y * score::out_gate<T>(mod, b, h0 + r) * score::elem_gate<T>(mod, b, h0 + r, c));
     }
 }
 
@@ -983,7 +990,8 @@ window_attn_decode_mma_kernel(const bf16* __restrict__ q, const bf16* __restrict
         if (sinks != nullptr) den += exp2f(sinks[h0 + r] * LOG2E - (mx == -INFINITY ? 0.f : mx));
         if (MODE == 2) den = 1.f;
         const float y = den > 0.f ? num / den : 0.f;
-        out[((long long)b * H + h0 + r) * DV + vz + c] = __float2bfloat16_rn(y * score::out_gate<bf16>(mod, b, h0 + r));
+        out[(long long)b * score::out_pitch(mod, H * DV) + (long long)(h0 + r) * DV + vz + c] =
+            __float2bfloat16_rn(y * score::out_gate<bf16>(mod, b, h0 + r) * score::elem_gate<bf16>(mod, b, h0 + r, vz + c));
     }
 }
 
@@ -1185,7 +1193,8 @@ NXD_API int nxd_qk_norm_cache_write(int dtype, const void* qkv, long long ld, vo
 // tensors of their own; v_row == k_row when the values are columns of the key rows).
 // impl: 0 = choose, 1 = the generic kernel, 2 = the tensor-core kernel (an error when it does not apply).
 // softcap <= 0: none; log_r1 / log_r2 [H] fp32 or NULL: logarithmic distance bias; sigmoid_bias [H] fp32 or NULL: sigmoid
-// weights instead of the softmax; gate (activation dtype, rows gate_ld elements apart) or NULL: output gate per head.
+// weights instead of the softmax; gate (activation dtype, rows gate_ld elements apart) or NULL: output gate per head, or
+// (gate_cols == Dv) per element, times gate_mul; out_ld: elements between output rows (0: H * Dv).
 NXD_API int nxd_scored_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v,
                                     long long k_stride_line, long long k_stride_head, long long k_row,
                                     long long v_stride_line, long long v_stride_head, long long v_row,
@@ -1193,10 +1202,13 @@ NXD_API int nxd_scored_attn_prefill(int dtype, const void* q, const void* cache_
                                     const int* n_new, const int* seq_ids, const float* slopes, const float* sinks, int B,
                                     int Tn, int H, int G, int D, int Dv, float scale, int window, int keep_first, int chunk,
                                     int impl, int value_heads, float softcap, const float* log_r1, const float* log_r2,
-                                    const float* sigmoid_bias, const void* gate, long long gate_ld, void* stream) {
+                                    const float* sigmoid_bias, const void* gate, long long gate_ld, int gate_cols,
+                                    float gate_mul, long long out_ld, void* stream) {
     NXD_REQUIRE((log_r1 == nullptr) == (log_r2 == nullptr), "attention: the logarithmic bias needs %s", "both vectors");
     NXD_REQUIRE(sigmoid_bias == nullptr || sinks == nullptr, "attention: sigmoid weights have no %s", "sink");
-    const ScoreMod mod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld};
+    NXD_REQUIRE(gate_cols == 0 || (gate_cols == Dv && gate != nullptr), "attention: a gate of %d columns per head of %d", gate_cols, Dv);
+    NXD_REQUIRE(out_ld == 0 || (out_ld >= (long long)H * Dv && out_ld % 2 == 0), "attention: output rows %lld apart", out_ld);
+    const ScoreMod mod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld, gate_cols, gate_mul, out_ld};
     const int mode = mod.mode();
     NXD_REQUIRE(G > 0 && H % G == 0, "attention: %d query heads over %d key/value heads", H, G);
     NXD_REQUIRE(Dv <= MAXC * 8, "attention: value size %d above %d", Dv, MAXC * 8);
@@ -1258,7 +1270,7 @@ NXD_API int nxd_masked_attn_prefill(int dtype, const void* q, const void* cache_
     return nxd_scored_attn_prefill(dtype, q, cache_k, cache_v, k_stride_line, k_stride_head, k_row, v_stride_line,
                                    v_stride_head, v_row, block_table, page_size, table_cols, out, q_start, n_new, seq_ids,
                                    slopes, sinks, B, Tn, H, G, D, Dv, scale, window, keep_first, chunk, impl, value_heads,
-                                   0.f, nullptr, nullptr, nullptr, nullptr, 0, stream);
+                                   0.f, nullptr, nullptr, nullptr, nullptr, 0, 0, 1.f, 0, stream);
 }
 
 NXD_API int nxd_window_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v,
@@ -1280,10 +1292,13 @@ NXD_API int nxd_scored_attn_decode(int dtype, const void* q, const void* cache_k
                                    const int* seq_ids, const float* slopes, const float* sinks, int B, int H, int G, int D,
                                    int Dv, float scale, int window, int keep_first, int chunk, int impl, int value_heads,
                                    float softcap, const float* log_r1, const float* log_r2, const float* sigmoid_bias,
-                                   const void* gate, long long gate_ld, void* stream) {
+                                   const void* gate, long long gate_ld, int gate_cols, float gate_mul, long long out_ld,
+                                   void* stream) {
     NXD_REQUIRE((log_r1 == nullptr) == (log_r2 == nullptr), "attention: the logarithmic bias needs %s", "both vectors");
     NXD_REQUIRE(sigmoid_bias == nullptr || sinks == nullptr, "attention: sigmoid weights have no %s", "sink");
-    const ScoreMod mod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld};
+    NXD_REQUIRE(gate_cols == 0 || (gate_cols == Dv && gate != nullptr), "attention: a gate of %d columns per head of %d", gate_cols, Dv);
+    NXD_REQUIRE(out_ld == 0 || (out_ld >= (long long)H * Dv && out_ld % 2 == 0), "attention: output rows %lld apart", out_ld);
+    const ScoreMod mod{softcap > 0.f ? softcap : 0.f, log_r1, log_r2, sigmoid_bias, gate, gate_ld, gate_cols, gate_mul, out_ld};
     const int mode = mod.mode();
     NXD_REQUIRE(G > 0 && H % G == 0, "attention: %d query heads over %d key/value heads", H, G);
     NXD_REQUIRE(Dv <= 512, "attention: value size %d above %d", Dv, 512);
@@ -1345,7 +1360,7 @@ NXD_API int nxd_masked_attn_decode(int dtype, const void* q, const void* cache_k
     return nxd_scored_attn_decode(dtype, q, cache_k, cache_v, k_stride_line, k_stride_head, k_row, v_stride_line,
                                   v_stride_head, v_row, block_table, page_size, table_cols, out, positions, seq_ids, slopes,
                                   sinks, B, H, G, D, Dv, scale, window, keep_first, chunk, impl, value_heads, 0.f, nullptr,
-                                  nullptr, nullptr, nullptr, 0, stream);
+                                  nullptr, nullptr, nullptr, 0, 0, 1.f, 0, stream);
 }
 
 NXD_API int nxd_window_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v,

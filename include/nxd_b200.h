@@ -332,7 +332,8 @@ int nxd_masked_attn_decode(int dtype, const void* q, const void* cache_k, const 
                            int value_heads, void* stream);
 /* The attention entry points with changes to the score and the head output (csrc/score_mod.cuh): softcap (<= 0: none),
  * logarithmic distance bias log_r1_h * ln(1 + log_r2_h * (i - j)) (fp32 [H], both or neither), sigmoid_bias (fp32 [H]: weights
- * sigmoid(score + b_h) instead of the softmax), gate (activation dtype, rows gate_ld apart: head h times sigmoid(gate)). */
+ * sigmoid(score + b_h) instead of the softmax), gate (activation dtype, rows gate_ld apart: head h times sigmoid(gate); with
+ * gate_cols == Dv one number per element, times gate_mul); out_ld: elements between output rows (0: H * Dv). */
 int nxd_scored_attn_prefill(int dtype, const void* q, const void* cache_k, const void* cache_v, long long k_stride_line,
                             long long k_stride_head, long long k_row, long long v_stride_line, long long v_stride_head,
                             long long v_row, const int* block_table, int page_size, int table_cols, void* out,
@@ -340,14 +341,15 @@ int nxd_scored_attn_prefill(int dtype, const void* q, const void* cache_k, const
                             const float* sinks, int B, int Tn, int H, int G, int D, int Dv, float scale, int window,
                             int keep_first, int chunk, int impl, int value_heads, float softcap, const float* log_r1,
                             const float* log_r2, const float* sigmoid_bias, const void* gate, long long gate_ld,
-                            void* stream);
+                            int gate_cols, float gate_mul, long long out_ld, void* stream);
 int nxd_scored_attn_decode(int dtype, const void* q, const void* cache_k, const void* cache_v, long long k_stride_line,
                            long long k_stride_head, long long k_row, long long v_stride_line, long long v_stride_head,
                            long long v_row, const int* block_table, int page_size, int table_cols, void* out,
                            const int* positions, const int* seq_ids, const float* slopes, const float* sinks, int B, int H,
                            int G, int D, int Dv, float scale, int window, int keep_first, int chunk, int impl,
                            int value_heads, float softcap, const float* log_r1, const float* log_r2,
-                           const float* sigmoid_bias, const void* gate, long long gate_ld, void* stream);
+                           const float* sigmoid_bias, const void* gate, long long gate_ld, int gate_cols, float gate_mul,
+                           long long out_ld, void* stream);
 /* nxd_qk_prep_cache_write with a projection bias (fp32, one number per column of the row, or NULL) and unit-RMS values */
 int nxd_qkv_prep_cache_write(int dtype, const void* qkv, long long ld, void* q_out, void* cache_k, void* cache_v,
                              long long k_stride_line, long long k_stride_head, long long v_stride_line,
@@ -362,7 +364,7 @@ int nxd_flash_attn_fwd_tc_scored(const void* q, const void* k, const void* v, vo
                                  int Hkv, int Sq, int Sk, int D, float scale, int window, int keep_first,
                                  const float* slopes, const float* sinks, float softcap, const float* log_r1,
                                  const float* log_r2, const float* sigmoid_bias, const void* gate, long long gate_ld,
-                                 void* stream);
+                                 int gate_cols, float gate_mul, void* stream);
 /* differential attention: maps [N, 2 * H, Dv] (first H heads = map 1, last H = map 2) -> out [N, H * Dv] =
  * rms_head(a1 - lambda * a2) * (1 - diff), lambda = exp(<lq1, lk1>) - exp(<lq2, lk2>) + diff (vectors fp32 [D]) */
 int nxd_diff_attn_combine(int dtype, const void* maps, void* out, const float* lq1, const float* lk1, const float* lq2,
@@ -502,16 +504,14 @@ int nxd_selective_scan(int dtype, const void* x, long long ld_x, const float* dt
                        const float* a_log, const float* dskip, float* S, void* out, long long ld_out, const int* q_start,
                        const int* n_new, const int* seq_ids, int B, int Tn, int C, int N, void* stream);
 /* S <- exp(-exp(a_log_h) dt) S + dt B x^T, y = S^T C + D_h x per head, B and C shared by the H / G heads of a group;
- * S [lines, H, N, P].  impl: 0 choose, 1 token by token, 2 chunks of 64 tokens on the tensor cores (bf16) */
+ * S [lines, H, N, P].  dt NULL with one token per row: the products of hin [B, W] with dt_w [H, W].  impl: 0 choose, 1 token by token, 2 chunks of 64 tokens on the tensor cores (bf16) */
 int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long long ld, int x_off, int b_off, int c_off,
                           const float* dt, long long ld_dt, const float* dt_bias, const float* a_log, const float* dskip,
                           float* S, void* y, const int* q_start, const int* n_new, const int* seq_ids, int B, int Tn, int H,
-                          int G, int N, int P, int impl, void* stream);
-/* v = y act(z) (act 0 sigmoid, 1 silu); groups > 0: every group of n / groups columns divided by its root mean square, times w;
- * groups == 0: v * mul */
+                          int G, int N, int P, int impl, const void* hin, const void* dt_w, int W, void* stream);
+/* v = y act(z) (act 0 sigmoid, 1 silu), every group of n / groups columns divided by its root mean square, times w */
 int nxd_gate_norm(int y_dtype, int dtype, const void* y, long long ld_y, const void* z, long long ld_z, const float* w,
-                  void* out, long long ld_out, long long rows, int n, int groups, float eps, float mul, int act,
-                  void* stream);
+                  void* out, long long ld_out, long long rows, int n, int groups, float eps, int act, void* stream);
 
 #ifdef __cplusplus
 }

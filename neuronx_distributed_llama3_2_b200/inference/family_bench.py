@@ -1029,19 +1029,25 @@ def state_space_kernel_cases(s: dict, steps: int, warmup: int, dev) -> List[dict
     q = torch.randn(B, T, H, D, device=dev, dtype=bf)
     kv = torch.randn(2, B, T, G, D, device=dev, dtype=bf)
     qp, kp, vp = q.permute(0, 2, 1, 3), kv[0].permute(0, 2, 1, 3), kv[1].permute(0, 2, 1, 3)
-    row("capped attention prefill, tcgen05", "prefill attention", lambda: wa.window_attention_tc(qp, kp, vp, D ** -0.5, softcap=30.0), flops=fl)
+    gate = torch.randn(B, T, H * D, device=dev, dtype=bf)
+    gd = gate.view(-1, H * D)[:Bd]
+    row("capped attention prefill + gate per element, tcgen05", "prefill attention",
+        lambda: wa.window_attention_tc(qp, kp, vp, D ** -0.5, softcap=30.0, gate=gate, gate_elements=True), flops=fl)
     row("causal attention prefill, tcgen05 (the like kernel)", "prefill attention",
         lambda: attn_ops.flash_attn_func(qp, kp, vp, softmax_scale=D ** -0.5, causal=True), flops=fl)
     ck = torch.randn(lines, G, S, D, device=dev, dtype=bf)
     cv = torch.randn(lines, G, S, D, device=dev, dtype=bf)
-    for name, cap in (("capped attention prefill over the cache, mma.sync", 30.0), ("causal attention prefill over the cache (the like kernel)", None)):
-        row(name, "prefill attention", lambda: wa.window_attention_prefill(q, ck, cv, zero, D ** -0.5, softcap=cap), flops=fl)
+    for name, cap in (("capped attention prefill over the cache + gate per element, mma.sync", 30.0),
+                      ("causal attention prefill over the cache (the like kernel)", None)):
+        kw = dict(gate=gate, gate_elements=True) if cap else {}
+        row(name, "prefill attention", lambda: wa.window_attention_prefill(q, ck, cv, zero, D ** -0.5, softcap=cap, **kw), flops=fl)
     qd = torch.randn(Bd, H, D, device=dev, dtype=bf)
     posd = torch.full((Bd,), T, dtype=torch.int32, device=dev)
-    for name, cap in (("capped attention decode", 30.0), ("causal attention decode (the like kernel)", None)):
-        row(name, "decode attention", lambda: wa.window_attention_decode(qd, ck, cv, posd, D ** -0.5, softcap=cap),
+    for name, cap in (("capped attention decode + gate per element", 30.0), ("causal attention decode (the like kernel)", None)):
+        kw = dict(gate=gd, gate_elements=True) if cap else {}
+        row(name, "decode attention", lambda: wa.window_attention_decode(qd, ck, cv, posd, D ** -0.5, softcap=cap, **kw),
             nbytes=2.0 * (T + 1) * G * 2 * D * Bd)
-    del kv, ck, cv
+    del kv, ck, cv, gate, gd
     n_qkv = H * D + 2 * G * D
     wide = torch.randn(B, T, n_qkv, device=dev, dtype=bf)
     ckw, cvw = torch.zeros(B, G, S, D, device=dev, dtype=bf), torch.zeros(B, G, S, D, device=dev, dtype=bf)
@@ -1050,10 +1056,7 @@ def state_space_kernel_cases(s: dict, steps: int, warmup: int, dev) -> List[dict
         row(name, "projection epilogue", lambda: wa.qk_norm_cache_write(wide, ckw, cvw, zero, H, G, D, D, 1e-6, normalize=False, rope=rope,
                                                                        rope_layout="halves", writeback=back),
             nbytes=2.0 * N * (2 * H * D + (5 if back else 4) * G * D))
-    g = torch.randn(N, H * D, device=dev, dtype=bf)
-    o = q.view(N, H * D)
-    row("attention output gate, one number per element", "norm", lambda: ss.gate_norm(o, g, act="sigmoid", mul=0.7), nbytes=2.0 * N * 3 * H * D)
-    del wide, ckw, cvw, q, g
+    del wide, ckw, cvw, q
     # state-space heads next to retention
     Hr, Dk, Dvr = s["rec_heads"], s["rec_dim"], s["rec_vdim"]
     inner = Hr * Dvr

@@ -773,10 +773,10 @@ class MumazenInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, MumazenForCau
         scaled embedding; a sublayer's result (with its output bias) times layer scale and ``residual_mult``; ahead of a
         pass of the looped range also the embedding once more (gathered from the table again) and the pass's vector;
       * ONE matrix product of the mixer's input gives all its projections (``layer.in_proj``, parts at ``layer.columns``); the
-        products that become step sizes stay fp32 (``dt_proj``);
-      * ``parallel``: rotation + cache write, capped softmax attention over the cache, the output gate; convolution,
-        state-space heads on the line's fp32 state, gate + grouped norm; both branches write their half of one buffer, which one
-        output projection reads (the branch scales sit in the gate's and the norm's fp32 epilogues);
+        products that become step sizes stay fp32 (``dt_proj``; of single tokens inside the recurrence's kernel);
+      * ``parallel``: rotation + cache write, capped softmax attention over the cache with the output gate in its epilogue;
+        convolution, state-space heads on the line's fp32 state, gate + grouped norm; both branches write their half of one
+        buffer, which one output projection reads (the branch scales sit in the gate's and the norm's fp32 epilogues);
       * ``mamba1``: convolution, the fp32 product for step sizes, B and C, the low-rank step sizes' second half, selective scan
         with the gate inside, output projection;
       * a looped layer appears once per pass in the run list: same modules, cache / state of the run's own index.
@@ -864,25 +864,27 @@ class MumazenInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, MumazenForCau
                                      out_dtype=self.config.torch_dtype)[1], None
 
     # -- mixers: big [B, T, n_out] = the fused projection of the normed input h [N, W] -> [N, W] ---------------------------
-    def _attention_heads(self, run, m, layer, big, B, T, q_start, n_new, seq_ids):
+    def _attention_heads(self, run, m, layer, big, out, mul, B, T, q_start, n_new, seq_ids) -> None:
+        """The gated heads times ``mul`` into ``out [N, heads * vdim]``."""
         ck, cv = self.kv_cache.layer(run)
-        paged = self._paged()
-        at, n = layer.columns["qkv"]
+        paged, cols = self._paged(), layer.columns
+        at, n = cols["qkv"]
         qkv = big[..., at: at + n]
         tc = (T >= self.TC_PREFILL_MIN_TOKENS and not self._step_past_context
               and wa_ops.tc_prefill_applies(qkv, m.dim, m.vdim, qkv.stride(-2)))
         q = wa_ops.qk_norm_cache_write(qkv, ck, cv, q_start, m.heads, m.kv_heads, m.dim, m.vdim, self.config.rms_norm_eps,
                                        n_new=n_new, seq_ids=seq_ids, normalize=False,
                                        rope=self._rotary_tables(m.rot, big.device), rope_layout="halves", writeback=tc, **paged)
+        gate = big[..., cols["g"][0]: cols["g"][0] + m.width]
+        kw = dict(softcap=m.softcap, gate_elements=True, gate_mul=mul, out=out)
         if T == 1:
-            return wa_ops.window_attention_decode(q[:, 0], ck, cv, q_start, m.scale, seq_ids=seq_ids, softcap=m.softcap, **paged)
-        if tc:                              # q, and k / v as views of the projection (the rotated keys were written back)
+            wa_ops.window_attention_decode(q[:, 0], ck, cv, q_start, m.scale, seq_ids=seq_ids, gate=gate[:, 0], **kw, **paged)
+        elif tc:                            # q, and k / v as views of the projection (the rotated keys were written back)
             k = qkv[..., m.heads * m.dim: (m.heads + m.kv_heads) * m.dim].unflatten(-1, (m.kv_heads, m.dim))
             v = qkv[..., (m.heads + m.kv_heads) * m.dim:].unflatten(-1, (m.kv_heads, m.vdim))
-            return wa_ops.window_attention_tc(q.permute(0, 2, 1, 3), k.permute(0, 2, 1, 3), v.permute(0, 2, 1, 3), m.scale,
-                                              softcap=m.softcap).permute(0, 2, 1, 3)
-        return wa_ops.window_attention_prefill(q, ck, cv, q_start, m.scale, n_new=n_new, seq_ids=seq_ids, softcap=m.softcap,
-                                               **paged)
+            wa_ops.window_attention_tc(q.permute(0, 2, 1, 3), k.permute(0, 2, 1, 3), v.permute(0, 2, 1, 3), m.scale, gate=gate, **kw)
+        else:
+            wa_ops.window_attention_prefill(q, ck, cv, q_start, m.scale, n_new=n_new, seq_ids=seq_ids, gate=gate, **kw, **paged)
 
     def _mix_parallel(self, run, layer, h, big, q_start, n_new, seq_ids):
         mixer, m, cfg = layer.mixer, layer.mixer.cfg, self.config
@@ -892,18 +894,16 @@ class MumazenInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, MumazenForCau
         joint = torch.empty(N, width, dtype=h.dtype, device=h.device)
         if a.width != right or r.inner != width - right:      # columns that pad a half meet zero rows of the projection
             joint.zero_()
-        rows = big.view(N, -1)
-        part = lambda n: rows[:, cols[n][0]: cols[n][0] + cols[n][1]]                      # noqa: E731
-        o = self._attention_heads(run, a, layer, big, B, T, q_start, n_new, seq_ids)
-        ss_ops.gate_norm(o.reshape(N, a.width), part("g"), act="sigmoid", mul=m.left_scale, out=joint[:, : a.width])
+        self._attention_heads(run, a, layer, big, joint[:, : a.width], m.left_scale, B, T, q_start, n_new, seq_ids)
         st = self.kv_cache.state(run)
-        dt = gemm_nt(h, mixer.dt_proj, out_dtype=torch.float32).view(B, T, -1)[..., : r.heads]
         at = cols["xbc"][0]
         xbc = ss_ops.conv_silu(big[..., at: at + r.channels], mixer.conv_weight, mixer.conv_bias, st["conv"], q_start,
                                n_new=n_new, seq_ids=seq_ids, out_pitch=(r.channels + 7) // 8 * 8)
-        y = ss_ops.state_space_heads(xbc, (0, r.inner, r.inner + r.groups * r.state), dt, mixer.dt_bias, mixer.a_log,
-                                     mixer.d_skip, st["S"], q_start, r.groups, n_new=n_new, seq_ids=seq_ids)
-        ss_ops.gate_norm(y.view(N, r.inner), part("z"), mixer.out_norm, r.norm_groups, cfg.rms_norm_eps,
+        y = ss_ops.state_space_heads(xbc, (0, r.inner, r.inner + r.groups * r.state), None, mixer.dt_bias, mixer.a_log,
+                                     mixer.d_skip, st["S"], q_start, r.groups, n_new=n_new, seq_ids=seq_ids,
+                                     dt_from=(h, mixer.dt_proj))
+        z = big.view(N, -1)[:, cols["z"][0]: cols["z"][0] + r.inner]
+        ss_ops.gate_norm(y.view(N, r.inner), z, mixer.out_norm, r.norm_groups, cfg.rms_norm_eps,
                          out=joint[:, right: right + r.inner])
         return gemm_nt(joint, mixer.o_proj.weight)
 

@@ -25,6 +25,7 @@ import torch
 import torch.nn.functional as F
 
 from . import _lib
+from .linear import gemm_nt
 
 GROUP = "state_space_serving"
 IMPLS = {"auto": 0, "scan": 1, "chunks": 2}
@@ -141,21 +142,32 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, dt_bias: Optional[torch.Te
     return out
 
 
-def state_space_heads(xbc: torch.Tensor, offsets: Tuple[int, int, int], dt: torch.Tensor, dt_bias: Optional[torch.Tensor],
+def state_space_heads(xbc: torch.Tensor, offsets: Tuple[int, int, int], dt: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor],
                       a_log: torch.Tensor, d: torch.Tensor, S: torch.Tensor, q_start: torch.Tensor, groups: int,
                       n_new: Optional[torch.Tensor] = None, seq_ids: Optional[torch.Tensor] = None,
-                      out_dtype: torch.dtype = torch.float32, impl: str = "auto") -> torch.Tensor:
+                      out_dtype: torch.dtype = torch.float32, impl: str = "auto",
+                      dt_from: Optional[Tuple[torch.Tensor, torch.Tensor]] = None) -> torch.Tensor:
     """``xbc [B, T, ld]`` holds, at columns ``offsets = (x, B, C)``, the heads' inputs ``[H, P]`` and the groups' ``B, C [G, N]``
     (after the convolution); ``dt [B, T, H]`` fp32 pre-activations of the step sizes (may be a column range); ``dt_bias,
     a_log, d [H]`` fp32; ``S [lines, H, N, P]`` fp32, updated in place -> ``y [B, T, H, P]`` in ``out_dtype``.  ``impl``: ``auto`` |
-    ``scan`` (token by token) | ``chunks`` (tensor cores, bf16; an error where it does not apply)."""
+    ``scan`` (token by token) | ``chunks`` (tensor cores, bf16; an error where it does not apply).  ``dt_from = (h [B * T, W],
+    w [>= H, W])`` instead of ``dt``: the pre-activations are ``h w^T`` (fp32), of a step of one token per row made inside the
+    recurrence's kernel."""
     B, T, _ = xbc.shape
     H, N, P = S.shape[1:]
-    assert H % groups == 0 and a_log.shape == (H,) and dt.dtype == torch.float32
+    assert H % groups == 0 and a_log.shape == (H,)
+    hin = dt_w = None
+    if dt is None:
+        hin, dt_w = dt_from
+        if T > 1 or n_new is not None or impl != "auto" or not _use_kernel(xbc):
+            dt, hin, dt_w = gemm_nt(hin, dt_w, out_dtype=torch.float32).view(B, T, -1)[..., :H], None, None
+    assert dt is None or dt.dtype == torch.float32
     x_off, b_off, c_off = offsets
     if _use_kernel(xbc):
         assert S.is_contiguous() and out_dtype in (torch.float32, xbc.dtype)
-        (xbc, ld), (dt, ldd) = _rows(xbc), _rows(dt)
+        xbc, ld = _rows(xbc)
+        dt, ldd = _rows(dt) if dt is not None else (None, 0)
+        assert hin is None or (hin.is_contiguous() and dt_w.is_contiguous() and hin.dtype == dt_w.dtype == xbc.dtype)
         y = torch.empty(B, T, H, P, dtype=out_dtype, device=xbc.device)
         qs, nn_, sid = _i32(q_start), _i32(n_new), _i32(seq_ids)
         L = _lib.lib(GROUP)
@@ -164,6 +176,7 @@ def state_space_heads(xbc: torch.Tensor, offsets: Tuple[int, int, int], dt: torc
                                      _c.c_longlong(ldd), _lib.ptr(dt_bias), _lib.ptr(a_log), _lib.ptr(d), _lib.ptr(S),
                                      _lib.ptr(y), _lib.ptr(qs), _lib.ptr(nn_), _lib.ptr(sid), _c.c_int(B), _c.c_int(T),
                                      _c.c_int(H), _c.c_int(groups), _c.c_int(N), _c.c_int(P), _c.c_int(IMPLS[impl]),
+                                     _lib.ptr(hin), _lib.ptr(dt_w), _c.c_int(hin.shape[1] if hin is not None else 0),
                                      _lib.stream_ptr())
         _lib.check(rc, "nxd_state_space_heads", L)
         return y
@@ -187,31 +200,26 @@ def state_space_heads(xbc: torch.Tensor, offsets: Tuple[int, int, int], dt: torc
     return y
 
 
-def gate_norm(y: torch.Tensor, z: torch.Tensor, weight: Optional[torch.Tensor] = None, groups: int = 0, eps: float = 0.0,
-              act: str = "silu", mul: float = 1.0, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``y, z [N, n]`` (rows may be column ranges of wider buffers) -> ``v = y * act(z)`` (``silu`` or ``sigmoid``), then, with
-    ``groups > 0``, every one of the ``groups`` equal parts of the columns divided by its root mean square (fp32, ``eps`` inside
-    the root) times ``weight [n]``; with ``groups == 0`` ``v * mul``.  Result in the dtype of ``z``, into ``out`` (a column
-    range of a wider buffer) when given."""
+def gate_norm(y: torch.Tensor, z: torch.Tensor, weight: torch.Tensor, groups: int, eps: float, act: str = "silu",
+              out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``y, z [N, n]`` (rows may be column ranges of wider buffers) -> ``v = y * act(z)`` (``silu`` or ``sigmoid``), every one of the
+    ``groups`` equal parts of the columns divided by its root mean square (fp32, ``eps`` inside the root), times ``weight [n]``.
+    Result in the dtype of ``z``, into ``out`` (a column range of a wider buffer) when given."""
     N, n = y.shape
-    assert z.shape == (N, n) and (groups == 0 or (n % groups == 0 and weight is not None))
+    assert z.shape == (N, n) and n % groups == 0
     if out is None:
         out = torch.empty(N, n, dtype=z.dtype, device=z.device)
     assert out.shape == (N, n) and out.dtype == z.dtype
-    if (_use_kernel(z) and y.dtype in (torch.float32, z.dtype) and y.stride(1) == 1 and z.stride(1) == 1 and out.stride(1) == 1):
+    if _use_kernel(z) and y.dtype in (torch.float32, z.dtype) and y.stride(1) == 1 and z.stride(1) == 1 and out.stride(1) == 1:
         L = _lib.lib(GROUP)
         rc = L.nxd_gate_norm(_c.c_int(_code(y.dtype)), _c.c_int(_code(z.dtype)), _lib.ptr(y), _c.c_longlong(y.stride(0)),
                              _lib.ptr(z), _c.c_longlong(z.stride(0)), _lib.ptr(weight), _lib.ptr(out),
                              _c.c_longlong(out.stride(0)), _c.c_longlong(N), _c.c_int(n), _c.c_int(groups), _c.c_float(eps),
-                             _c.c_float(mul), _c.c_int(1 if act == "silu" else 0), _lib.stream_ptr())
+                             _c.c_int(1 if act == "silu" else 0), _lib.stream_ptr())
         _lib.check(rc, "nxd_gate_norm", L)
         return out
     zf = z.float()
-    v = y.float() * (F.silu(zf) if act == "silu" else torch.sigmoid(zf))
-    if groups:
-        v = v.reshape(N, groups, n // groups)
-        v = (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(N, n) * weight.float()
-    else:
-        v = v * mul
+    v = (y.float() * (F.silu(zf) if act == "silu" else torch.sigmoid(zf))).reshape(N, groups, n // groups)
+    v = (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)).reshape(N, n) * weight.float()
     out.copy_(v.to(z.dtype))
     return out

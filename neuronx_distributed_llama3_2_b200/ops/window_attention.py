@@ -8,7 +8,8 @@
 
 ``log_bias = (r1, r2)``: ``score -= r1_h * ln(1 + r2_h * (i - j))``; ``softcap``: ``score = cap * tanh(score / cap)`` ahead
 of the distance biases; ``sigmoid_bias``: the weights are ``sigmoid(score + b_h)``, not normalised over the keys, instead of
-the softmax; ``gate``: the output of head ``h`` is multiplied by ``sigmoid`` of that head's pre-activation.
+the softmax; ``gate``: the output of head ``h`` is multiplied by ``sigmoid`` of that head's pre-activation, or (``gate_elements``)
+every element by ``gate_mul * sigmoid`` of its own.  ``out``: where the result goes, a column range of a wider buffer.
 
 ``sinks``: a learned per-head logit that is attached to no position and only takes probability mass.  The value rows may be
 a column range of the key rows (``cache_v`` a view of ``cache_k``): the cache of a compressed key/value projection.
@@ -191,7 +192,8 @@ def window_attention_ref(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_po
                          window: Optional[int], keep_first: int, slopes: Optional[torch.Tensor],
                          chunk: Optional[int] = None, sinks: Optional[torch.Tensor] = None,
                          softcap: Optional[float] = None, log_bias: Optional[tuple] = None,
-                         sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                         sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                         gate_elements: bool = False, gate_mul: float = 1.0) -> torch.Tensor:
     """One sequence in fp32: ``q [Tq, H, D]`` at positions ``q_pos [Tq]`` over keys ``k [G, Tk, D]`` / ``v [Gv, Tk, Dv]``
     at positions ``0 .. Tk - 1``; with fewer value heads than key heads, key head ``g`` reads value head ``g % Gv``."""
     H, G = q.shape[1], k.shape[0]
@@ -216,7 +218,10 @@ def window_attention_ref(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_po
         r1, r2 = (t.float().reshape(H, 1, 1) for t in log_bias)
         s = s - r1 * torch.log(1.0 + r2 * dist.clamp(min=0).float())
     s = s.masked_fill(~vis, float("-inf"))
-    g = torch.sigmoid(gate.float()).unsqueeze(-1) if gate is not None else 1.0          # [Tq, H, 1]
+    g = 1.0
+    if gate is not None:                                                                # [Tq, H, 1] or [Tq, H, Dv]
+        g = (gate_mul * torch.sigmoid(gate.float()).unflatten(-1, (H, v.shape[-1])) if gate_elements
+             else torch.sigmoid(gate.float()).unsqueeze(-1))
     if sigmoid_bias is not None:
         assert sinks is None
         p = torch.sigmoid(s + sigmoid_bias.float().reshape(H, 1, 1))                      # masked scores: weight 0
@@ -230,8 +235,9 @@ def window_attention_ref(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_po
     return torch.einsum("hqk,hkd->qhd", p, vf) * g
 
 
-def _mod_args(softcap, log_bias, sigmoid_bias, gate, x):
-    """The score / output modifications of an attention call as C arguments (and the tensors to keep alive)."""
+def _mod_args(softcap, log_bias, sigmoid_bias, gate, x, gate_cols: int = 0, gate_mul: float = 1.0, out_ld: Optional[int] = None):
+    """The score / output modifications of an attention call as C arguments (and the tensors to keep alive); ``out_ld``:
+    elements between output rows, for the entry points that take them."""
     r1, r2 = (t.float().contiguous() for t in log_bias) if log_bias is not None else (None, None)
     pb = sigmoid_bias.float().contiguous() if sigmoid_bias is not None else None
     if gate is not None:
@@ -239,8 +245,16 @@ def _mod_args(softcap, log_bias, sigmoid_bias, gate, x):
         assert gate.dim() == 2 or gate.shape[0] == 1 or gate.stride(0) == gate.shape[1] * gate.stride(1)
     ld = gate.stride(-2) if gate is not None else 0
     return (_c.c_float(float(softcap) if softcap else 0.0), _lib.ptr(r1), _lib.ptr(r2), _lib.ptr(pb), _lib.ptr(gate),
-            _c.c_longlong(ld)), (r1, r2, pb)
+            _c.c_longlong(ld), _c.c_int(gate_cols), _c.c_float(gate_mul)) + (
+        (_c.c_longlong(out_ld),) if out_ld is not None else ()), (r1, r2, pb)
 
+
+def _out_rows(out: Optional[torch.Tensor], q: torch.Tensor, rows: int, H: int, Dv: int):
+    """The output ``[rows, H * Dv]`` of an attention call (given, or new) and the distance between its rows."""
+    if out is None:
+        return torch.empty(rows, H * Dv, dtype=q.dtype, device=q.device), 0
+    assert out.shape == (rows, H * Dv) and out.dtype == q.dtype and out.stride(1) == 1
+    return out, out.stride(0)
 
 
 def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tensor, q_start: torch.Tensor,
@@ -250,8 +264,11 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
                              page_size: int = 0, impl: str = "auto", chunk: Optional[int] = None,
                              sinks: Optional[torch.Tensor] = None, value_heads: Optional[int] = None,
                              softcap: Optional[float] = None, log_bias: Optional[tuple] = None,
-                             sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """``gate [B, T, H]``: output gate pre-activations (may be a column range of a projection output).
+                             sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                             gate_elements: bool = False, gate_mul: float = 1.0,
+                             out: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """``gate [B, T, H]``: output gate pre-activations (may be a column range of a projection output); ``gate_elements``:
+    ``[B, T, H * Dv]``.  ``out [B * T, H * Dv]``: a buffer (or a column range of one) for the result.
 
     ``impl``: ``auto`` | ``generic`` (fp32-math tile kernel, any sizes) | ``mma`` (bf16 tensor-core kernel, an error
     where it does not apply) -- for tests and measurements.
@@ -263,12 +280,12 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
     w = int(window) if window else 0
     if _use_kernel(q):
         q = q if q.is_contiguous() else q.contiguous()
-        out = torch.empty(B, T, H, Dv, dtype=q.dtype, device=q.device)
+        out, out_ld = _out_rows(out, q, B * T, H, Dv)
         qs, nn_, sid = _i32(q_start), _i32(n_new), _i32(seq_ids)
         cargs, bt = _cache_args(cache_k, cache_v, block_table, page_size, rows=True)
         sk = sinks.float().contiguous() if sinks is not None else None
         L = _lib.lib(GROUP)
-        margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q)
+        margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q, Dv if gate_elements else 0, gate_mul, out_ld)
         rc = L.nxd_scored_attn_prefill(_c.c_int(_code(q.dtype)), _lib.ptr(q), _lib.ptr(cache_k), _lib.ptr(cache_v),
                                        *cargs, _lib.ptr(out), _lib.ptr(qs), _lib.ptr(nn_), _lib.ptr(sid),
                                        _lib.ptr(slopes), _lib.ptr(sk), _c.c_int(B), _c.c_int(T), _c.c_int(H), _c.c_int(G),
@@ -277,8 +294,8 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
                                        _c.c_int({"auto": 0, "generic": 1, "mma": 2}[impl]),
                                        _c.c_int(int(value_heads) if value_heads else 0), *margs, _lib.stream_ptr())
         _lib.check(rc, "nxd_scored_attn_prefill", L)
-        return out
-    out = torch.zeros(B, T, H, Dv, dtype=q.dtype, device=q.device)
+        return out.view(B, T, H, Dv) if out_ld == 0 else out
+    given, out = out, torch.zeros(B, T, H, Dv, dtype=q.dtype, device=q.device)
     for b in range(B):
         n = T if n_new is None else int(n_new[b])
         if n == 0:
@@ -289,8 +306,9 @@ def window_attention_prefill(q: torch.Tensor, cache_k: torch.Tensor, cache_v: to
         vv = _cache_rows(cache_v, line, p0 + n, block_table, page_size)
         pos = torch.arange(p0, p0 + n, device=q.device)
         out[b, :n] = window_attention_ref(q[b, :n], kk, vv, pos, scale, w, keep_first, slopes, chunk, sinks,
-                                          softcap, log_bias, sigmoid_bias, gate[b, :n] if gate is not None else None).to(q.dtype)
-    return out
+                                          softcap, log_bias, sigmoid_bias, gate[b, :n] if gate is not None else None,
+                                          gate_elements, gate_mul).to(q.dtype)
+    return given.copy_(out.view(B * T, H * Dv)) if given is not None else out
 
 
 def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: torch.Tensor, positions: torch.Tensor,
@@ -300,19 +318,22 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
                             impl: str = "auto", chunk: Optional[int] = None,
                             sinks: Optional[torch.Tensor] = None, value_heads: Optional[int] = None,
                             softcap: Optional[float] = None, log_bias: Optional[tuple] = None,
-                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                            sigmoid_bias: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None,
+                            gate_elements: bool = False, gate_mul: float = 1.0,
+                            out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """One new token per row: ``q [B, H, D]`` at ``positions[b]`` -> ``[B, H, Dv]``; only the kept first rows and the
-    window's rows of the cache line are read.  ``gate [B, H]``: output gate pre-activations."""
+    window's rows of the cache line are read.  ``gate [B, H]`` (``gate_elements``: ``[B, H * Dv]``): output gate
+    pre-activations.  ``out [B, H * Dv]``: a buffer (or a column range of one) for the result."""
     B, H, D = q.shape
     G, Dv = cache_k.shape[1], cache_v.shape[3]
     w = int(window) if window else 0
     if _use_kernel(q):
         q = q if q.is_contiguous() else q.contiguous()
-        out = torch.empty(B, H, Dv, dtype=q.dtype, device=q.device)
+        out, out_ld = _out_rows(out, q, B, H, Dv)
         pos, sid = _i32(positions), _i32(seq_ids)
         cargs, bt = _cache_args(cache_k, cache_v, block_table, page_size, rows=True)
         sk = sinks.float().contiguous() if sinks is not None else None
-        plain = not softcap and log_bias is None and sigmoid_bias is None
+        plain = not softcap and log_bias is None and sigmoid_bias is None and not gate_elements and out_ld == 0
         if (impl == "auto" and q.dtype == torch.bfloat16 and G == 1 and not keep_first and not chunk and slopes is None and plain
                 and cache_v.data_ptr() == cache_k.data_ptr() and cache_v.stride(2) == cache_k.stride(2)
                 and cache_v.stride(0) == cache_k.stride(0)):
@@ -320,10 +341,10 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
             # rows once per 16 query heads, with the context split over CTAs when the batch alone does not fill the GPU
             from . import latent_attention as la
 
-            if la.latent_decode(q, cache_k, Dv, out, pos, sid, sk, scale, bt, page_size, w, gate):
-                return out
+            if la.latent_decode(q, cache_k, Dv, out.view(B, H, Dv), pos, sid, sk, scale, bt, page_size, w, gate):
+                return out.view(B, H, Dv)
         L = _lib.lib(GROUP)
-        margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q)
+        margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q, Dv if gate_elements else 0, gate_mul, out_ld)
         rc = L.nxd_scored_attn_decode(_c.c_int(_code(q.dtype)), _lib.ptr(q), _lib.ptr(cache_k), _lib.ptr(cache_v), *cargs,
                                       _lib.ptr(out), _lib.ptr(pos), _lib.ptr(sid), _lib.ptr(slopes), _lib.ptr(sk),
                                       _c.c_int(B), _c.c_int(H), _c.c_int(G), _c.c_int(D), _c.c_int(Dv), _c.c_float(scale),
@@ -331,8 +352,8 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
                                       _c.c_int({"auto": 0, "generic": 1, "mma": 2}[impl]),
                                       _c.c_int(int(value_heads) if value_heads else 0), *margs, _lib.stream_ptr())
         _lib.check(rc, "nxd_scored_attn_decode", L)
-        return out
-    out = torch.empty(B, H, Dv, dtype=q.dtype, device=q.device)
+        return out.view(B, H, Dv) if out_ld == 0 else out
+    given, out = out, torch.empty(B, H, Dv, dtype=q.dtype, device=q.device)
     for b in range(B):
         line = b if seq_ids is None else int(seq_ids[b])
         p = int(positions[b])
@@ -340,8 +361,8 @@ def window_attention_decode(q: torch.Tensor, cache_k: torch.Tensor, cache_v: tor
         vv = _cache_rows(cache_v, line, p + 1, block_table, page_size)
         out[b] = window_attention_ref(q[b:b + 1], kk, vv, torch.tensor([p], device=q.device), scale, w, keep_first,
                                       slopes, chunk, sinks, softcap, log_bias, sigmoid_bias,
-                                      gate[b:b + 1] if gate is not None else None)[0].to(q.dtype)
-    return out
+                                      gate[b:b + 1] if gate is not None else None, gate_elements, gate_mul)[0].to(q.dtype)
+    return given.copy_(out.view(B, H * Dv)) if given is not None else out
 
 
 def diff_attention_combine(maps: torch.Tensor, lq1: torch.Tensor, lk1: torch.Tensor, lq2: torch.Tensor,
@@ -381,19 +402,25 @@ def window_attention_tc(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale
                         keep_first: int = 0, slopes: Optional[torch.Tensor] = None,
                         sinks: Optional[torch.Tensor] = None, softcap: Optional[float] = None,
                         log_bias: Optional[tuple] = None, sigmoid_bias: Optional[torch.Tensor] = None,
-                        gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        gate: Optional[torch.Tensor] = None, gate_elements: bool = False, gate_mul: float = 1.0,
+                        out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Prefill from position 0 on the tcgen05 flash-attention kernel (``csrc/flash_attn_tc.cu``, windowed
     instantiation): ``q [B, H, T, D]``, ``k / v [B, G, T, D]`` as (strided) views with unit stride on ``D`` ->
     ``[B, H, T, D]`` stored as ``[B, T, H, D]``.  All rows are taken as ``T`` tokens long (right padding only ever
-    sits behind the real tokens of a causal row).  ``gate [B, T, H]``: output gate pre-activations."""
+    sits behind the real tokens of a causal row).  ``gate [B, T, H]`` (``gate_elements``: ``[B, T, H * D]``): output gate
+    pre-activations.  ``out [B * T, H * D]``: a buffer (or a column range of one, rows a multiple of 8 elements apart)."""
     from .flash_attn import _fix, _strides
 
     q, k, v = _fix(q), _fix(k), _fix(v)
     B, H, T, D = q.shape
     G = k.shape[1]
-    o = torch.empty(B, T, H, D, dtype=q.dtype, device=q.device).permute(0, 2, 1, 3)
+    if out is None:
+        o = torch.empty(B, T, H, D, dtype=q.dtype, device=q.device).permute(0, 2, 1, 3)
+    else:
+        assert out.shape == (B * T, H * D) and out.stride(1) == 1
+        o = out.as_strided((B, H, T, D), (T * out.stride(0), D, out.stride(0), 1))
     L = _lib.lib()
-    margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q)
+    margs, _keep = _mod_args(softcap, log_bias, sigmoid_bias, gate, q, D if gate_elements else 0, gate_mul)
     sk = sinks.float().contiguous() if sinks is not None else None
     rc = L.nxd_flash_attn_fwd_tc_scored(_lib.ptr(q), _lib.ptr(k), _lib.ptr(v), _lib.ptr(o), _strides(q, k, v, o),
                                         _c.c_int(B), _c.c_int(H), _c.c_int(G), _c.c_int(T), _c.c_int(T), _c.c_int(D),

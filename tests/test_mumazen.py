@@ -309,7 +309,7 @@ def test_chunks_on_the_tensor_cores_equal_the_token_walk(H, G, N, P):
 
 @case
 @pytest.mark.parametrize("n,groups", [(12, 3), (40, 1), (33, 3), (64, 8), (2048, 2), (1500, 1), (9000, 1)])
-def test_gate_then_grouped_norm_and_plain_gate(dev, dt, n, groups):
+def test_gate_then_grouped_norm(dev, dt, n, groups):
     torch.manual_seed(n)
     N = 5
     y, zs = torch.randn(N, n) * 3, torch.randn(N, n + 24).to(dt)
@@ -319,8 +319,9 @@ def test_gate_then_grouped_norm_and_plain_gate(dev, dt, n, groups):
     got = ss.gate_norm(y.to(dev), zs.to(dev)[:, 8: 8 + n], w.to(dev), groups, 1e-2, out=buf[:, 16: 16 + n])
     close(got, O.gated_group_norm(y.to(F64), z, w.to(F64), groups, 1e-2), dt, scale=3.0)
     assert float(buf[:, :16].abs().max()) == 0.0 and float(buf[:, 16 + n:].abs().max()) == 0.0
-    yt = y.to(dt)
-    close(ss.gate_norm(yt.to(dev), zs.to(dev)[:, 8: 8 + n], act="sigmoid", mul=0.7), 0.7 * yt.to(F64) * torch.sigmoid(z), dt, scale=3.0)
+    got = ss.gate_norm(y.to(dt).to(dev), zs.to(dev)[:, 8: 8 + n], w.to(dev), groups, 1e-2, act="sigmoid")
+    v = (y.to(dt).to(F64) * torch.sigmoid(z)).reshape(N, groups, -1)
+    close(got, O.rms(v, 1e-2).reshape(N, n) * w.to(F64), dt, scale=3.0)
 
 
 @case
@@ -331,6 +332,7 @@ def test_slowed_rotation_and_capped_attention(dev, dt, H, G, D, Dv, rot, cap):
     torch.manual_seed(D + Dv)
     T, lens = 40, [40, 23]
     qkv = torch.randn(2, T, H * D + G * (D + Dv) + 8).to(dt)
+    gates = torch.randn(2, T, H * Dv + 8).to(dt)
     r = {"base": 500.0, "dims": rot, "scaling": {"factor": 3.0}} if rot else None
     rope = tuple(t.to(dev) for t in rp.build_interleaved_rope_cache(64, rot, 500.0, factor=3.0)) if rot else None
     scale = 6.0 / D ** 0.5                                       # scores on both sides of the cap
@@ -341,7 +343,10 @@ def test_slowed_rotation_and_capped_attention(dev, dt, H, G, D, Dv, rot, cap):
         rd = lambda t: t.to(dt).to(F64)                                                 # noqa: E731  as the cache holds it
         q = rd(O.rotate(x[:, : H * D].reshape(n, H, D), pos, r))
         kk = rd(O.rotate(x[:, H * D: (H + G) * D].reshape(n, G, D), pos, r))
-        ref.append(O.capped_attention(q, kk, x[:, (H + G) * D: (H + G) * D + G * Dv].reshape(n, G, Dv), scale, cap))
+        o = O.capped_attention(q, kk, x[:, (H + G) * D: (H + G) * D + G * Dv].reshape(n, G, Dv), scale, cap)
+        g = torch.sigmoid(gates[k, :n, 8:].to(F64)).reshape(n, H, Dv)
+        ref.append((o, 0.7 * o * g))
+    pad = H * Dv % 2
     at = 0
     for n in (17, 2, 20, 1):
         left = [max(0, min(n, L - at)) for L in lens]
@@ -350,14 +355,58 @@ def test_slowed_rotation_and_capped_attention(dev, dt, H, G, D, Dv, rot, cap):
         start = i32(at, at, dev=dev)
         q = wa.qk_norm_cache_write(rows, ck, cv, start, H, G, D, Dv, 1e-6, n_new=i32(*left, dev=dev), normalize=False, rope=rope,
                                    rope_layout="halves", **kw)
-        if n == 1:
-            o = wa.window_attention_decode(q[:, 0], ck, cv, start, scale, softcap=cap, **kw).unsqueeze(1)
-        else:
-            o = wa.window_attention_prefill(q, ck, cv, start, scale, n_new=i32(*left, dev=dev), softcap=cap, **kw)
-        for k in range(2):
-            if left[k]:
-                close(o[k, :left[k]], ref[k][at: at + left[k]], dt, scale=2.0)
+        gate = gates[:, at: at + n].contiguous().to(dev)[..., 8:]
+        for gated in (False, True):
+            buf = torch.zeros(2 * n, H * Dv + 32 + pad, dtype=dt, device=dev)
+            gk = dict(gate_elements=True, gate_mul=0.7, out=buf[:, 16: 16 + H * Dv]) if gated else {}
+            if n == 1:
+                o = wa.window_attention_decode(q[:, 0], ck, cv, start, scale, softcap=cap, gate=gate[:, 0] if gated else None, **gk, **kw)
+            else:
+                o = wa.window_attention_prefill(q, ck, cv, start, scale, n_new=i32(*left, dev=dev), softcap=cap,
+                                                gate=gate if gated else None, **gk, **kw)
+            o = (buf[:, 16: 16 + H * Dv] if gated else o).reshape(2, n, H, Dv)
+            assert float(buf[:, :16].abs().max()) == 0.0 and float(buf[:, 16 + H * Dv:].abs().max()) == 0.0
+            for k in range(2):
+                if left[k]:
+                    close(o[k, :left[k]], ref[k][int(gated)][at: at + left[k]], dt, scale=2.0)
         at += n
+
+
+@pytest.mark.gpu
+@pytest.mark.parametrize("D,T", [(64, 40), (64, 300), (128, 257)])
+def test_capped_gated_attention_on_tcgen05_into_a_column_range(D, T):
+    torch.manual_seed(T)
+    H, G = 4, 2
+    qkv = torch.randn(2, T, (H + 2 * G) * D).bfloat16().cuda()
+    gates = torch.randn(2, T, H * D + 16).bfloat16().cuda()
+    q, k, v = (qkv[..., lo * D: hi * D].unflatten(-1, (hi - lo, D)).permute(0, 2, 1, 3) for lo, hi in ((0, H), (H, H + G), (H + G, H + 2 * G)))
+    buf = torch.zeros(2 * T, H * D + 24, dtype=torch.bfloat16, device="cuda")
+    wa.window_attention_tc(q, k, v, 4.0 / D ** 0.5, softcap=6.0, gate=gates[..., 8: 8 + H * D], gate_elements=True, gate_mul=1.5,
+                           out=buf[:, 8: 8 + H * D])
+    assert float(buf[:, :8].abs().max()) == 0.0 and float(buf[:, 8 + H * D:].abs().max()) == 0.0
+    for b in range(2):
+        o = O.capped_attention(*(t[b].permute(1, 0, 2).cpu().to(F64) for t in (q, k, v)), 4.0 / D ** 0.5, 6.0)
+        g = torch.sigmoid(gates[b, :, 8: 8 + H * D].cpu().to(F64)).reshape(T, H, D)
+        close(buf.view(2, T, -1)[b, :, 8: 8 + H * D].reshape(T, H, D), 1.5 * o * g, torch.bfloat16)
+
+
+@case
+@pytest.mark.parametrize("W", [24, 30, 1040])
+def test_step_sizes_of_single_tokens_made_inside_the_recurrence(dev, dt, W):
+    torch.manual_seed(W)
+    H, G, N, P, B = 5, 1, 20, 12, 3
+    h, w = torch.randn(B, W).to(dt), (torch.randn(8, W) * W ** -0.5).to(dt)
+    xbc = torch.randn(B, 1, H * P + 2 * G * N).to(dt).to(dev)
+    vecs = [torch.randn(H).to(dev) * 0.5 for _ in range(3)]
+    S0 = torch.randn(B, H, N, P).to(dev)
+    outs = []
+    for kw in (dict(dt=(h.float() @ w.float().T)[:, :H].reshape(B, 1, H).contiguous().to(dev)), dict(dt=None, dt_from=(h.to(dev), w.to(dev)))):
+        S = S0.clone()
+        dtv = kw.pop("dt")
+        y = ss.state_space_heads(xbc, (0, H * P, H * P + G * N), dtv, *vecs, S, i32(4, 9, 1, dev=dev), G, **kw)
+        outs.append((y, S))
+    close(outs[1][0], outs[0][0].cpu(), torch.float32)
+    close(outs[1][1], outs[0][1].cpu(), torch.float32)
 
 
 def test_scaled_rotation_tables():
