@@ -14,9 +14,9 @@
 //   conv_silu          convolution + silu of a column range of a projection; also moves the line's convolution state (the
 //                      last taps - 1 raw inputs) when one thread sees the whole step, else conv_state does it afterwards
 //   selective_scan     states of a channel split over R lanes of NS registers (two channels per thread share the loads of B and
-//                      C), tokens in double-buffered blocks through shared memory (cp.async); the R partial sums of R
-//                      consecutive tokens are summed by one transposing butterfly; step sizes ahead of a block, gate, skip term
-//                      and store behind it.  Prompts and single tokens
+//                      C), tokens in blocks through four shared-memory buffers (cp.async); the R partial sums of R
+//                      consecutive tokens are summed by one transposing butterfly; the other half of the CTA makes the step
+//                      sizes ahead of a block and applies skip term and gate behind it.  Prompts and single tokens
 //   ssd_step           one token: a thread owns four neighbouring columns of a head's state, the rows are spread over the
 //                      CTA; the state is read and written once
 //   ssd_scan           token by token, a column's rows split over R lanes (fp32 prompts, short steps, unusual sizes)
@@ -58,16 +58,42 @@ __device__ __forceinline__ float decay_exp(float y) {
     return fmaf(y, p, 1.f);
 }
 constexpr float LOG2E = 1.4426950408889634f;
-// the decay of a state in the selective scan: fp32 serving rounds it as above, 16-bit serving takes the hardware's 2^x
+// packed fp32 arithmetic on two neighbouring states
+__device__ __forceinline__ uint64_t pair2(float lo, float hi) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(lo), "f"(hi));
+    return r;
+}
+__device__ __forceinline__ void unpair2(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v)); }
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+
+// the decays of two states in the selective scan: fp32 serving rounds it as above, 16-bit serving takes the hardware's 2^x
 template <typename T>
 struct ScanDecay {
     static __device__ __forceinline__ float rate(float a) { return a * LOG2E; }
-    static __device__ __forceinline__ float at(float dt, float rate) { return exp2_ftz(dt * rate); }
+    static __device__ __forceinline__ uint64_t at2(uint64_t dt, uint64_t rate) {
+        float lo, hi;
+        unpair2(mul2(dt, rate), lo, hi);
+        return pair2(exp2_ftz(lo), exp2_ftz(hi));
+    }
 };
 template <>
 struct ScanDecay<float> {
     static __device__ __forceinline__ float rate(float a) { return a; }
-    static __device__ __forceinline__ float at(float dt, float rate) { return decay_exp(dt * rate); }
+    static __device__ __forceinline__ uint64_t at2(uint64_t dt, uint64_t rate) {
+        float lo, hi;
+        unpair2(mul2(dt, rate), lo, hi);
+        return pair2(decay_exp(lo), decay_exp(hi));
+    }
 };
 
 // The arithmetic around the recurrences.  fp32 serving takes the library functions; 16-bit serving forms built on the hardware's
@@ -271,77 +297,150 @@ __device__ __forceinline__ float transpose_sum(float (&v)[R], int r) {
     return v[0];
 }
 
-constexpr int SS_THREADS = 128;
+// Half of the CTA scans block i while the other half prepares block i + 1 (step sizes), finishes block i - 1 (skip term, gate,
+// store) and fetches block i + 2: one barrier per block of TS tokens.
+constexpr int SS_SCAN = 128, SS_HELP = 128, SS_BUFS = 4;
 
-// NS states of each of CPT neighbouring channels per thread, R neighbouring lanes share them; TS tokens per block
+// NS states of each of CPT neighbouring channels per scanning thread, R neighbouring lanes share them
 template <typename T, int NS, int R, int CPT, int TS>
 struct ScanSmem {
-    static constexpr int CH = SS_THREADS / R * CPT, NP = NS * R;
+    static constexpr int CH = SS_SCAN / R * CPT, NP = NS * R;
     struct Buf {
-        float B[TS][NP], Cm[TS][NP], dt[TS][CH];
+        float B[TS][NP], Cm[TS][NP];
+        float dt[TS][CH];                                  // pre-activations, then step sizes
+        float u[TS][CH];                                   // dt * x, then sum_n S C
         T x[TS][CH], z[TS][CH];
-    } buf[2];
-    float u[TS][CH];                                       // dt * x, then sum_n S C
+    } buf[SS_BUFS];
 };
 
 template <typename T, int NS, int R, int CPT, int TS>
-__global__ void __launch_bounds__(SS_THREADS)
+__global__ void __launch_bounds__(SS_SCAN + SS_HELP)
 selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __restrict__ dt, long long ld_dt,
                       const float* __restrict__ dt_bias, const float* __restrict__ bc, long long ld_bc, int b_off, int c_off,
                       const T* __restrict__ z, long long ld_z, const float* __restrict__ a_log, const float* __restrict__ dskip,
                       float* __restrict__ S, T* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
                       const int* __restrict__ n_new, const int* __restrict__ seq_ids, int Tn, int C, int N, int async) {
     using Sm = ScanSmem<T, NS, R, CPT, TS>;
-    constexpr int CH = Sm::CH, NP = Sm::NP;
-    static_assert(TS % R == 0, "tokens come in groups of R");
+    constexpr int CH = Sm::CH, NP = Sm::NP, THREADS = SS_SCAN + SS_HELP;
+    static_assert(TS % R == 0 && NS % 4 == 0, "tokens come in groups of R, states in groups of 4");
     extern __shared__ __align__(16) unsigned char smem_raw[];
     Sm& sm = *reinterpret_cast<Sm*>(smem_raw);
-    const int tid = threadIdx.x, r = tid % R, cl = tid / R * CPT;
+    const int tid = threadIdx.x;
+    const bool helper = tid >= SS_SCAN;
     const int c0 = blockIdx.x * CH, b = blockIdx.y;
     const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
     const long long row0 = (long long)b * Tn;
     const int nch = min(CH, C - c0);
-    for (int idx = tid; idx < (Tn - max(n, 0)) * nch; idx += SS_THREADS)                     // padding rows
+    for (int idx = tid; idx < (Tn - max(n, 0)) * nch; idx += THREADS)                        // padding rows
         stf(out + (row0 + max(n, 0) + idx / nch) * ld_out + c0 + idx % nch, 0.f);
     if (n <= 0) return;
     const int line = seq_ids != nullptr ? seq_ids[b] : b;
-    float* Sc = S + ((long long)line * C + c0 + cl) * N;
     const bool fresh = q_start[b] == 0;
-    float s[CPT][NS], a2[CPT][NS];
-#pragma unroll
-    for (int k = 0; k < CPT; ++k)
-#pragma unroll
-        for (int j = 0; j < NS; ++j) {
-            const int i = r * NS + j;
-            const bool ok = cl + k < nch && i < N;
-            s[k][j] = (ok && !fresh) ? Sc[(long long)k * N + i] : 0.f;
-            a2[k][j] = ok ? ScanDecay<T>::rate(-expf(a_log[(long long)(c0 + cl + k) * N + i])) : 0.f;
-        }
-    // columns N .. NP - 1 of B and C are zeros in both buffers and stay so
+    const int tiles = (n + TS - 1) / TS;
+    // columns N .. NP - 1 of B and C are zeros in all buffers and stay so
     if (N < NP)
-        for (int idx = tid; idx < 2 * TS * (NP - N); idx += SS_THREADS) {
+        for (int idx = tid; idx < SS_BUFS * TS * (NP - N); idx += THREADS) {
             const int k = idx / (TS * (NP - N)), q = idx % (TS * (NP - N));
             sm.buf[k].B[q / (NP - N)][N + q % (NP - N)] = 0.f;
             sm.buf[k].Cm[q / (NP - N)][N + q % (NP - N)] = 0.f;
         }
+    if (!helper) {
+        const int r = tid % R, cl = tid / R * CPT;
+        float* Sc = S + ((long long)line * C + c0 + cl) * N;
+        uint64_t s[CPT][NS / 2], a2[CPT][NS / 2];
+#pragma unroll
+        for (int m = 0; m < CPT; ++m)
+#pragma unroll
+            for (int j = 0; j < NS / 2; ++j) {
+                float sv[2], av[2];
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const int i = r * NS + 2 * j + e;
+                    const bool ok = cl + m < nch && i < N;
+                    sv[e] = (ok && !fresh) ? Sc[(long long)m * N + i] : 0.f;
+                    av[e] = ok ? ScanDecay<T>::rate(-expf(a_log[(long long)(c0 + cl + m) * N + i])) : 0.f;
+                }
+                s[m][j] = pair2(sv[0], sv[1]);
+                a2[m][j] = pair2(av[0], av[1]);
+            }
+        __syncthreads();
+        for (int it = 0; it <= tiles + 1; ++it) {
+            if (it >= 1 && it <= tiles) {
+                typename Sm::Buf& d = sm.buf[(it - 1) & (SS_BUFS - 1)];
+                const int top = (min(TS, n - (it - 1) * TS) + R - 1) / R * R;
+                for (int g0 = 0; g0 < top; g0 += R) {
+                    float y[CPT][R];
+#pragma unroll
+                    for (int q = 0; q < R; ++q) {
+                        uint64_t dv[CPT], u[CPT], acc[CPT];
+#pragma unroll
+                        for (int m = 0; m < CPT; ++m) {
+                            const float dvs = d.dt[g0 + q][cl + m], us = d.u[g0 + q][cl + m];
+                            dv[m] = pair2(dvs, dvs), u[m] = pair2(us, us), acc[m] = 0ull;
+                        }
+#pragma unroll
+                        for (int j = 0; j < NS; j += 4) {
+                            const ulonglong2 bv = *reinterpret_cast<const ulonglong2*>(&d.B[g0 + q][r * NS + j]);
+                            const ulonglong2 cv = *reinterpret_cast<const ulonglong2*>(&d.Cm[g0 + q][r * NS + j]);
+#pragma unroll
+                            for (int m = 0; m < CPT; ++m) {
+                                const uint64_t g01 = ScanDecay<T>::at2(dv[m], a2[m][j / 2]);
+                                const uint64_t g23 = ScanDecay<T>::at2(dv[m], a2[m][j / 2 + 1]);
+                                s[m][j / 2] = fma2(g01, s[m][j / 2], mul2(u[m], bv.x));
+                                s[m][j / 2 + 1] = fma2(g23, s[m][j / 2 + 1], mul2(u[m], bv.y));
+                                acc[m] = fma2(s[m][j / 2], cv.x, acc[m]);
+                                acc[m] = fma2(s[m][j / 2 + 1], cv.y, acc[m]);
+                            }
+                        }
+#pragma unroll
+                        for (int m = 0; m < CPT; ++m) {
+                            float lo, hi;
+                            unpair2(acc[m], lo, hi);
+                            y[m][q] = lo + hi;
+                        }
+                    }
+                    // every lane of the channel has read its u of these tokens (the shuffles wait for them): y takes their place
+#pragma unroll
+                    for (int m = 0; m < CPT; ++m) {
+                        const float v = transpose_sum<R>(y[m], r);
+                        d.u[g0 + r][cl + m] = v;
+                    }
+                }
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int m = 0; m < CPT; ++m)
+#pragma unroll
+            for (int j = 0; j < NS / 2; ++j) {
+                float lo, hi;
+                unpair2(s[m][j], lo, hi);
+                const int i = r * NS + 2 * j;
+                if (cl + m < nch && i < N) Sc[(long long)m * N + i] = lo;
+                if (cl + m < nch && i + 1 < N) Sc[(long long)m * N + i + 1] = hi;
+            }
+        return;
+    }
     constexpr int XV = 16 / sizeof(T);                       // elements of T per 16 bytes
     constexpr int CX = CH / XV;                              // such pieces per token
-    auto fetch = [&](int t0, int k) {
-        typename Sm::Buf& d = sm.buf[k];
-        const int cnt = min(TS, n - t0);
+    const int ht = tid - SS_SCAN;
+    auto fetch = [&](int tile) {
+        typename Sm::Buf& d = sm.buf[tile & (SS_BUFS - 1)];
+        const int t0 = tile * TS, cnt = min(TS, n - t0);
         if (async) {
-            for (int idx = tid; idx < cnt * (N / 4); idx += SS_THREADS) {
-                const int tt = idx / (N / 4), i = (idx % (N / 4)) * 4;
+            const int n4 = N / 4;
+            for (int idx = ht; idx < cnt * n4; idx += SS_HELP) {
+                const int tt = idx / n4, i = (idx - tt * n4) * 4;
                 const float* src = bc + (row0 + t0 + tt) * ld_bc + i;
                 mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.B[tt][i]), src + b_off, true);
                 mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.Cm[tt][i]), src + c_off, true);
             }
-            for (int idx = tid; idx < cnt * (CH / 4); idx += SS_THREADS) {
+            for (int idx = ht; idx < cnt * (CH / 4); idx += SS_HELP) {
                 const int tt = idx / (CH / 4), i = (idx % (CH / 4)) * 4;
                 const bool ok = i < nch;
                 mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.dt[tt][i]), dt + (row0 + t0 + tt) * ld_dt + c0 + (ok ? i : 0), ok);
             }
-            for (int idx = tid; idx < cnt * CX; idx += SS_THREADS) {
+            for (int idx = ht; idx < cnt * CX; idx += SS_HELP) {
                 const int tt = idx / CX, i = (idx % CX) * XV;
                 const bool ok = i < nch;
                 const long long at = row0 + t0 + tt;
@@ -349,13 +448,13 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
                 mma::cp_async16((uint32_t)__cvta_generic_to_shared(&d.z[tt][i]), z + at * ld_z + c0 + (ok ? i : 0), ok);
             }
         } else {
-            for (int idx = tid; idx < cnt * N; idx += SS_THREADS) {
+            for (int idx = ht; idx < cnt * N; idx += SS_HELP) {
                 const int tt = idx / N, i = idx % N;
                 const float* src = bc + (row0 + t0 + tt) * ld_bc + i;
                 d.B[tt][i] = src[b_off];
                 d.Cm[tt][i] = src[c_off];
             }
-            for (int idx = tid; idx < cnt * CH; idx += SS_THREADS) {
+            for (int idx = ht; idx < cnt * CH; idx += SS_HELP) {
                 const int tt = idx / CH, i = idx % CH;
                 const bool ok = i < nch;
                 const long long at = row0 + t0 + tt;
@@ -364,100 +463,63 @@ selective_scan_kernel(const T* __restrict__ x, long long ld_x, const float* __re
                 stf(&d.z[tt][i], ok ? ldf(z + at * ld_z + c0 + i) : 0.f);
             }
         }
-        mma::cp_async_commit();
     };
-    fetch(0, 0);
-    // a thread prepares and finishes VP neighbouring channels of every (128 VP / CH)-th token, always the same channels
-    constexpr int VP = 2, PT = CH / VP, ROWS = SS_THREADS / PT;
-    static_assert(SS_THREADS % PT == 0 && CH % VP == 0, "channel slices");
-    const int pi = tid % PT * VP, prow = tid / PT;
+    // a helper prepares and finishes VP neighbouring channels of every ROWS-th token, always the same channels
+    constexpr int VP = 2, PT = CH / VP, ROWS = SS_HELP / PT;
+    static_assert(SS_HELP % PT == 0 && CH % VP == 0, "channel slices");
+    const int pi = ht % PT * VP, prow = ht / PT;
     float bias[VP], dsk[VP];
 #pragma unroll
     for (int v = 0; v < VP; ++v) {
         bias[v] = (dt_bias != nullptr && pi + v < nch) ? dt_bias[c0 + pi + v] : 0.f;
         dsk[v] = pi + v < nch ? dskip[c0 + pi + v] : 0.f;
     }
-    int k = 0;
-    for (int t0 = 0; t0 < n; t0 += TS, k ^= 1) {
-        const int cnt = min(TS, n - t0), top = (cnt + R - 1) / R * R;
-        if (t0 + TS < n) {
-            fetch(t0 + TS, k ^ 1);
-            mma::cp_async_wait<1>();
-        } else {
-            mma::cp_async_wait<0>();
-        }
-        __syncthreads();
-        typename Sm::Buf& d = sm.buf[k];
-        for (int tt = prow; tt < top; tt += ROWS) {                      // step sizes; tokens past the end: no step
+    fetch(0);
+    mma::cp_async_commit();
+    __syncthreads();
+    for (int it = 0; it <= tiles + 1; ++it) {
+        if (it + 1 < tiles) fetch(it + 1);
+        mma::cp_async_commit();
+        mma::cp_async_wait<1>();
+        asm volatile("bar.sync 1, %0;" ::"n"(SS_HELP) : "memory");       // block `it` has arrived for every helper
+        if (it < tiles) {
+            typename Sm::Buf& d = sm.buf[it & (SS_BUFS - 1)];
+            const int cnt = min(TS, n - it * TS), top = (cnt + R - 1) / R * R;
+            for (int tt = prow; tt < top; tt += ROWS) {                  // step sizes; tokens past the end: no step
 #pragma unroll
-            for (int v = 0; v < VP; ++v) {
-                const bool ok = tt < cnt && pi + v < nch;
-                const float step = ok ? ScanMath<T>::softplus(d.dt[tt][pi + v] + bias[v]) : 0.f;
-                d.dt[tt][pi + v] = step;
-                sm.u[tt][pi + v] = ok ? step * ldf(&d.x[tt][pi + v]) : 0.f;
-            }
-        }
-        for (int idx = tid; idx < (top - cnt) * N; idx += SS_THREADS) {  // rows that no copy has filled
-            d.B[cnt + idx / N][idx % N] = 0.f;
-            d.Cm[cnt + idx / N][idx % N] = 0.f;
-        }
-        __syncthreads();
-        for (int g0 = 0; g0 < top; g0 += R) {
-            float y[CPT][R];
-#pragma unroll
-            for (int q = 0; q < R; ++q) {
-                float dv[CPT], u[CPT], acc[CPT];
-#pragma unroll
-                for (int m = 0; m < CPT; ++m) dv[m] = d.dt[g0 + q][cl + m], u[m] = sm.u[g0 + q][cl + m], acc[m] = 0.f;
-#pragma unroll
-                for (int j = 0; j < NS; j += 4) {
-                    const float4 bv = *reinterpret_cast<const float4*>(&d.B[g0 + q][r * NS + j]);
-                    const float4 cv = *reinterpret_cast<const float4*>(&d.Cm[g0 + q][r * NS + j]);
-#pragma unroll
-                    for (int m = 0; m < CPT; ++m) {
-                        s[m][j] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j]), s[m][j], u[m] * bv.x);
-                        s[m][j + 1] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j + 1]), s[m][j + 1], u[m] * bv.y);
-                        s[m][j + 2] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j + 2]), s[m][j + 2], u[m] * bv.z);
-                        s[m][j + 3] = fmaf(ScanDecay<T>::at(dv[m], a2[m][j + 3]), s[m][j + 3], u[m] * bv.w);
-                        acc[m] += fmaf(s[m][j], cv.x, s[m][j + 1] * cv.y) + fmaf(s[m][j + 2], cv.z, s[m][j + 3] * cv.w);
-                    }
+                for (int v = 0; v < VP; ++v) {
+                    const bool ok = tt < cnt && pi + v < nch;
+                    const float step = ok ? ScanMath<T>::softplus(d.dt[tt][pi + v] + bias[v]) : 0.f;
+                    d.dt[tt][pi + v] = step;
+                    d.u[tt][pi + v] = ok ? step * ldf(&d.x[tt][pi + v]) : 0.f;
                 }
-#pragma unroll
-                for (int m = 0; m < CPT; ++m) y[m][q] = acc[m];
             }
-            // every lane of the channel has read its u of these tokens (the shuffles wait for them): y takes their place
-#pragma unroll
-            for (int m = 0; m < CPT; ++m) {
-                const float v = transpose_sum<R>(y[m], r);
-                if (R == 1) __syncwarp();
-                sm.u[g0 + r][cl + m] = v;
+            for (int idx = ht; idx < (top - cnt) * N; idx += SS_HELP) {  // rows that no copy has filled
+                d.B[cnt + idx / N][idx % N] = 0.f;
+                d.Cm[cnt + idx / N][idx % N] = 0.f;
             }
         }
-        __syncthreads();
-        for (int tt = prow; tt < cnt; tt += ROWS) {
-            float v[VP];
-#pragma unroll
-            for (int w = 0; w < VP; ++w)
-                v[w] = fmaf(dsk[w], ldf(&d.x[tt][pi + w]), sm.u[tt][pi + w]) * ScanMath<T>::silu(ldf(&d.z[tt][pi + w]));
-            T* dst = out + (row0 + t0 + tt) * ld_out + c0 + pi;
-            if (async && pi + 1 < nch) {
-                if (sizeof(T) == 4) *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
-                else *reinterpret_cast<uint32_t*>(dst) = mma::pack2(v[0], v[1]);
-            } else {
+        if (it >= 2) {
+            typename Sm::Buf& d = sm.buf[(it - 2) & (SS_BUFS - 1)];
+            const int t0 = (it - 2) * TS, cnt = min(TS, n - t0);
+            for (int tt = prow; tt < cnt; tt += ROWS) {
+                float v[VP];
 #pragma unroll
                 for (int w = 0; w < VP; ++w)
-                    if (pi + w < nch) stf(dst + w, v[w]);
+                    v[w] = fmaf(dsk[w], ldf(&d.x[tt][pi + w]), d.u[tt][pi + w]) * ScanMath<T>::silu(ldf(&d.z[tt][pi + w]));
+                T* dst = out + (row0 + t0 + tt) * ld_out + c0 + pi;
+                if (async && pi + 1 < nch) {
+                    if (sizeof(T) == 4) *reinterpret_cast<float2*>(dst) = make_float2(v[0], v[1]);
+                    else *reinterpret_cast<uint32_t*>(dst) = mma::pack2(v[0], v[1]);
+                } else {
+#pragma unroll
+                    for (int w = 0; w < VP; ++w)
+                        if (pi + w < nch) stf(dst + w, v[w]);
+                }
             }
         }
-        __syncthreads();                                                 // everyone is done with this buffer and with u
+        __syncthreads();
     }
-#pragma unroll
-    for (int m = 0; m < CPT; ++m)
-#pragma unroll
-        for (int j = 0; j < NS; ++j) {
-            const int i = r * NS + j;
-            if (cl + m < nch && i < N) Sc[(long long)m * N + i] = s[m][j];
-        }
 }
 
 template <typename T, int NS, int R, int CPT, int TS>
@@ -474,7 +536,7 @@ int launch_selective(const void* x, long long ld_x, const float* dt, long long l
     auto kern = selective_scan_kernel<T, NS, R, CPT, TS>;
     if (smem > 48 * 1024) NXD_CHECK_CUDA(cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     dim3 grid((C + Sm::CH - 1) / Sm::CH, B);
-    kern<<<grid, SS_THREADS, smem, st>>>((const T*)x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, (const T*)z, ld_z, a_log,
+    kern<<<grid, SS_SCAN + SS_HELP, smem, st>>>((const T*)x, ld_x, dt, ld_dt, dt_bias, bc, ld_bc, b_off, c_off, (const T*)z, ld_z, a_log,
                                          dskip, S, (T*)out, ld_out, q_start, n_new, seq_ids, Tn, C, N, async);
     NXD_LAUNCH_CHECK();
     return 0;
@@ -1050,13 +1112,13 @@ NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const f
     do {                                                                                                                 \
         if (N <= 4) NXD_SEL(T, 4, 1, 1, 16);                                                                             \
         if (N <= 8) NXD_SEL(T, 4, 2, 2, 16);                                                                             \
-        if (N <= 16 && Tn > 1) NXD_SEL(T, 4, 4, 2, 32);                                                                  \
+        if (N <= 16 && Tn > 1) NXD_SEL(T, 4, 4, 2, 16);                                                                  \
         if (N <= 16) NXD_SEL(T, 4, 4, 1, 16);                                                                            \
         if (N <= 32) NXD_SEL(T, 8, 4, 1, 16);                                                                            \
         if (N <= 64) NXD_SEL(T, 8, 8, 1, 16);                                                                            \
         if (N <= 128) NXD_SEL(T, 16, 8, 1, 16);                                                                          \
-        if (N <= 256) NXD_SEL(T, 16, 16, 1, 16);                                                                         \
-        NXD_SEL(T, 32, 16, 1, 16);                                                                                       \
+        if (N <= 256) NXD_SEL(T, 32, 8, 1, 8);                                                                           \
+        NXD_SEL(T, 64, 8, 1, 8);                                                                                         \
     } while (0)
     if (dtype == 0) NXD_SEL_T(bf16);
     NXD_SEL_T(float);
