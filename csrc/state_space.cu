@@ -12,11 +12,13 @@
 //
 // Kernels:
 //   conv_silu          convolution + silu of a column range of a projection; also moves the line's convolution state (the
-//                      last taps - 1 raw inputs) when one thread sees the whole step, else conv_state does it afterwards
+//                      last taps - 1 raw inputs) when one thread sees the whole step, else conv_state does it afterwards;
+//                      conv_silu_strip is its form for long 16-bit steps
 //   selective_scan     states of a channel split over R lanes of NS registers (two channels per thread share the loads of B and
 //                      C), tokens in blocks through four shared-memory buffers (cp.async); the R partial sums of R
 //                      consecutive tokens are summed by one transposing butterfly; the other half of the CTA makes the step
 //                      sizes ahead of a block and applies skip term and gate behind it.  Prompts and single tokens
+//   selective_step     one token per row: the low-rank product that makes the step sizes, the recurrence and the gate
 //   ssd_step           one token: a thread owns four neighbouring columns of a head's state, the rows are spread over the
 //                      CTA; the state is read and written once
 //   ssd_scan           token by token, a column's rows split over R lanes (fp32 prompts, short steps, unusual sizes)
@@ -224,7 +226,7 @@ conv_silu_kernel(const T* __restrict__ proj, long long ld, const float* __restri
 #pragma unroll
         for (int j = 0; j < NT; ++j)
 #pragma unroll
-            for (int i = 0; i < VEC; ++i) w[j][i] = conv_w[(long long)(c + i) * NT + j];
+            for (int i = 0; i < VEC; ++i) w[j][i] = conv_w[(long long)j * C + c + i];
         if (t0 < te) {
 #pragma unroll
             for (int j = 0; j + 1 < NT; ++j) conv_input<T, VEC>(row0, ld, st, t0 - (NT - 1) + j, p0, K, C, c, win[j + 1]);
@@ -254,7 +256,7 @@ conv_silu_kernel(const T* __restrict__ proj, long long ld, const float* __restri
             for (int j = 0; j <= K; ++j) {
                 conv_input<T, VEC>(row0, ld, st, t - K + j, p0, K, C, c, v);
 #pragma unroll
-                for (int i = 0; i < VEC; ++i) acc[i] = fmaf(conv_w[(long long)(c + i) * (K + 1) + j], v[i], acc[i]);
+                for (int i = 0; i < VEC; ++i) acc[i] = fmaf(conv_w[(long long)j * C + c + i], v[i], acc[i]);
             }
 #pragma unroll
             for (int i = 0; i < VEC; ++i) acc[i] = ScanMath<TO>::silu(acc[i]);
@@ -266,6 +268,71 @@ conv_silu_kernel(const T* __restrict__ proj, long long ld, const float* __restri
     for (int i = 0; i < VEC; ++i) zero[i] = 0.f;
     for (int t = max(t0, n); t < t1; ++t) stv<VEC>(orow + (long long)t * ld_out, zero);
     if (move && n > 0) move_conv_state<T, VEC>(row0, ld, st, n, p0, K, C, c);
+}
+
+// Long 16-bit steps: a thread convolves STRIP tokens of eight channels, all of whose STRIP + TAPS - 1 rows it asks for at once
+// (the overlap between strips is served by the caches).  Does not move the state.
+constexpr int STRIP = 8;
+
+template <int TAPS>
+__global__ void __launch_bounds__(128)
+conv_silu_strip_kernel(const bf16* __restrict__ proj, long long ld, const float* __restrict__ conv_w,
+                       const float* __restrict__ bias, const float* __restrict__ conv_state, bf16* __restrict__ out,
+                       long long ld_out, const int* __restrict__ q_start, const int* __restrict__ n_new,
+                       const int* __restrict__ seq_ids, int Tn, int C) {
+    constexpr int K = TAPS - 1;
+    const int c = (blockIdx.x * 128 + threadIdx.x) * 8;
+    if (c >= C) return;
+    const int b = blockIdx.z, t0 = blockIdx.y * STRIP;
+    const int n = n_new != nullptr ? min(n_new[b], Tn) : Tn;
+    const bf16* row0 = proj + (long long)b * Tn * ld + c;
+    bf16* orow = out + (long long)b * Tn * ld_out + c;
+    bf16x8 raw[STRIP + K];
+#pragma unroll
+    for (int j = 0; j < STRIP + K; ++j) {
+        const int t = t0 - K + j;
+        if (t >= 0 && t < n) raw[j] = *reinterpret_cast<const bf16x8*>(row0 + (long long)t * ld);
+    }
+    float bv[8], w[TAPS][8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) bv[i] = 0.f;
+    if (bias != nullptr) ldv<8>(bias + c, bv);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) ldv<8>(conv_w + (long long)j * C + c, w[j]);
+    float win[TAPS][8];
+    const int line = seq_ids != nullptr ? seq_ids[b] : b;
+#pragma unroll
+    for (int j = 0; j < K; ++j) {
+        if (t0 - K + j >= 0) {
+            unpack8(raw[j], win[j + 1]);
+        } else {                                               // ahead of the step: the line's state, zeros ahead of the sequence
+            conv_input<bf16, 8>(nullptr, 0, conv_state + (long long)line * K * C, t0 - K + j, q_start[b], K, C, c, win[j + 1]);
+        }
+    }
+#pragma unroll
+    for (int g = 0; g < STRIP; ++g) {
+        const int t = t0 + g;
+        if (t >= Tn) break;
+        float acc[8];
+#pragma unroll
+        for (int j = 0; j < K; ++j)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) win[j][i] = win[j + 1][i];
+        if (t < n) {
+            unpack8(raw[g + K], win[K]);
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                acc[i] = bv[i];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc[i] = fmaf(w[j][i], win[j][i], acc[i]);
+                acc[i] = ScanMath<bf16>::silu(acc[i]);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < 8; ++i) acc[i] = 0.f;
+        }
+        stv<8>(orow + (long long)t * ld_out, acc);
+    }
 }
 
 template <typename T>
@@ -540,6 +607,81 @@ int launch_selective(const void* x, long long ld_x, const float* dt, long long l
                                          dskip, S, (T*)out, ld_out, q_start, n_new, seq_ids, Tn, C, N, async);
     NXD_LAUNCH_CHECK();
     return 0;
+}
+
+// One token per row.  A CTA takes 32 channels (four lanes each) of STEP_ROWS rows, so that the low-rank weights that make the step
+// sizes, dt_c = softplus(<dt_w[c], p[row]> + bias_c), are read once for those rows; every state is read and written once.
+constexpr int STEP_ROWS = 4, STEP_THREADS = 128;
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(STEP_THREADS)
+selective_step_kernel(const T* __restrict__ x, long long ld_x, const T* __restrict__ dt_w, int rank,
+                      const float* __restrict__ dt_bias, const float* __restrict__ p, long long ld_p, int b_off, int c_off,
+                      const T* __restrict__ z, long long ld_z, const float* __restrict__ a_log, const float* __restrict__ dskip,
+                      float* __restrict__ S, T* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
+                      const int* __restrict__ seq_ids, int B, int C, int N) {
+    extern __shared__ __align__(16) float smem[];              // [STEP_ROWS][rank + 2 N]
+    const int pitch = rank + 2 * N;
+    const int tid = threadIdx.x, r = tid & 3, c = blockIdx.x * 32 + (tid >> 2);
+    const int b0 = blockIdx.y * STEP_ROWS, nb = min(STEP_ROWS, B - b0);
+    for (int idx = tid; idx < nb * pitch; idx += STEP_THREADS) {
+        const int q = idx / pitch, i = idx - q * pitch;
+        const float* row = p + (long long)(b0 + q) * ld_p;
+        smem[idx] = i < rank ? row[i] : (i < rank + N ? row[b_off + i - rank] : row[c_off + i - rank - N]);
+    }
+    __syncthreads();
+    if (c >= C) return;                                        // whole groups of four lanes
+    const unsigned mask = __activemask();
+    float acc[STEP_ROWS];
+#pragma unroll
+    for (int q = 0; q < STEP_ROWS; ++q) acc[q] = 0.f;
+    const T* wr = dt_w + (long long)c * rank;                  // rank is a multiple of 8
+    for (int k = r * 8; k < rank; k += 32) {
+        float w[8];
+        ldv<8>(wr + k, w);
+#pragma unroll
+        for (int q = 0; q < STEP_ROWS; ++q)
+            if (q < nb) {
+#pragma unroll
+                for (int i = 0; i < 8; ++i) acc[q] = fmaf(w[i], smem[q * pitch + k + i], acc[q]);
+            }
+    }
+    const float bias = dt_bias != nullptr ? dt_bias[c] : 0.f, dsk = dskip[c];
+#pragma unroll
+    for (int q = 0; q < STEP_ROWS; ++q) {
+        if (q >= nb) break;
+        const int b = b0 + q, line = seq_ids != nullptr ? seq_ids[b] : b;
+        const bool fresh = q_start[b] == 0;
+        float v = acc[q];
+        v += __shfl_xor_sync(mask, v, 1);
+        v += __shfl_xor_sync(mask, v, 2);
+        const float step = softplus_f(v + bias), xv = ldf(x + (long long)b * ld_x + c), u = step * xv;
+        const float* Bs = smem + q * pitch + rank;
+        const float* Cs = Bs + N;
+        float* Sc = S + ((long long)line * C + c) * N;
+        const float* al = a_log + (long long)c * N;
+        constexpr int W = VEC ? 4 : 1;
+        float y = 0.f;
+        for (int i = r * W; i < N; i += 4 * W) {
+            float s[W], a[W];
+            if (fresh) {
+#pragma unroll
+                for (int e = 0; e < W; ++e) s[e] = 0.f;
+            } else {
+                ldv<W>(Sc + i, s);
+            }
+            ldv<W>(al + i, a);
+#pragma unroll
+            for (int e = 0; e < W; ++e) {
+                s[e] = fmaf(decay_exp(-expf(a[e]) * step), s[e], u * Bs[i + e]);
+                y = fmaf(s[e], Cs[i + e], y);
+            }
+            stv<W>(Sc + i, s);
+        }
+        y += __shfl_xor_sync(mask, y, 1);
+        y += __shfl_xor_sync(mask, y, 2);
+        if (r == 0) stf(out + (long long)b * ld_out + c, fmaf(dsk, xv, y) * silu_f(ldf(z + (long long)b * ld_z + c)));
+    }
 }
 
 // ---- state-space heads: one token ------------------------------------------------------------------------------------------
@@ -1051,7 +1193,7 @@ int launch_gate(const void* y, long long ld_y, const void* z, long long ld_z, co
 
 }  // namespace
 
-// dtypes: 0 bf16, 1 fp32.  proj [B * Tn, ld] points at the first of the C channels; conv_w fp32 [C, taps] (last column = the
+// dtypes: 0 bf16, 1 fp32.  proj [B * Tn, ld] points at the first of the C channels; conv_w fp32 [taps, C] (last row = the
 // current token), bias fp32 [C] or NULL; conv_state fp32 [lines, taps - 1, C], moved to the end of the step (zeros before
 // the start of the sequence; rows without real tokens keep theirs).  out [B * Tn, ld_out]: silu(convolution), zeros in padding
 // rows.  q_start [B], n_new [B] or NULL, seq_ids [B] or NULL as in the attention entry points.
@@ -1066,9 +1208,10 @@ NXD_API int nxd_conv_silu(int dtype, int out_dtype, const void* proj, long long 
     const bool vec = C % 4 == 0 && ld % 4 == 0 && ld_out % 4 == 0 && al(proj) && al(out) && al(conv_state);
     // few tokens: one thread walks the whole step and moves the state itself
     const int TT = Tn <= 64 ? Tn : 32, move = Tn <= 64 ? 1 : 0;
-    const bool wide = vec && !move && dtype == 0 && out_dtype == 0 && taps == 4 && C % 8 == 0 && ld % 8 == 0 && ld_out % 8 == 0;
-    const int width = 128 * (wide ? 8 : (vec ? 4 : 1));
-    dim3 grid((C + width - 1) / width, (Tn + TT - 1) / TT, B);
+    const bool wide = vec && !move && dtype == 0 && out_dtype == 0 && taps == 4 && C % 8 == 0 && ld % 8 == 0 && ld_out % 8 == 0 &&
+                      al(conv_w) && al(bias);
+    const int width = 128 * (wide ? 8 : (vec ? 4 : 1)), tokens = wide ? STRIP : TT;
+    dim3 grid((C + width - 1) / width, (Tn + tokens - 1) / tokens, B);
     NXD_REQUIRE(grid.y < 65536, "short convolution: %d tokens", Tn);
 #define NXD_CONV(T, TO, V, K)                                                                                            \
     conv_silu_kernel<T, TO, V, K><<<grid, 128, 0, st>>>((const T*)proj, ld, conv_w, bias, conv_state, (TO*)out, ld_out,    \
@@ -1078,7 +1221,9 @@ NXD_API int nxd_conv_silu(int dtype, int out_dtype, const void* proj, long long 
         if (taps == 4) { if (vec) NXD_CONV(T, TO, 4, 4); else NXD_CONV(T, TO, 1, 4); }                                    \
         else { if (vec) NXD_CONV(T, TO, 4, 0); else NXD_CONV(T, TO, 1, 0); }                                              \
     } while (0)
-    if (wide) NXD_CONV(bf16, bf16, 8, 4);
+    if (wide)
+        conv_silu_strip_kernel<4><<<grid, 128, 0, st>>>((const bf16*)proj, ld, conv_w, bias, conv_state, (bf16*)out, ld_out,
+                                                        q_start, n_new, seq_ids, Tn, C);
     else if (dtype == 0 && out_dtype == 0) NXD_CONV_T(bf16, bf16);
     else if (dtype == 0) NXD_CONV_T(bf16, float);
     else { NXD_REQUIRE(out_dtype == 1, "short convolution: fp32 input, 16-bit output"); NXD_CONV_T(float, float); }
@@ -1112,8 +1257,7 @@ NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const f
     do {                                                                                                                 \
         if (N <= 4) NXD_SEL(T, 4, 1, 1, 16);                                                                             \
         if (N <= 8) NXD_SEL(T, 4, 2, 2, 16);                                                                             \
-        if (N <= 16 && Tn > 1) NXD_SEL(T, 4, 4, 2, 16);                                                                  \
-        if (N <= 16) NXD_SEL(T, 4, 4, 1, 16);                                                                            \
+        if (N <= 16) NXD_SEL(T, 4, 4, 2, 16);                                                                            \
         if (N <= 32) NXD_SEL(T, 8, 4, 1, 16);                                                                            \
         if (N <= 64) NXD_SEL(T, 8, 8, 1, 16);                                                                            \
         if (N <= 128) NXD_SEL(T, 16, 8, 1, 16);                                                                          \
@@ -1124,6 +1268,32 @@ NXD_API int nxd_selective_scan(int dtype, const void* x, long long ld_x, const f
     NXD_SEL_T(float);
 #undef NXD_SEL_T
 #undef NXD_SEL
+}
+
+// One token per row of the same recurrence; the step sizes' pre-activations are the first `rank` columns of p (fp32 [B, ld_p], B and C
+// at b_off and c_off) times dt_w [C, rank] (dtype; rank a multiple of 8).
+NXD_API int nxd_selective_step(int dtype, const void* x, long long ld_x, const void* dt_w, int rank, const float* dt_bias,
+                               const float* p, long long ld_p, int b_off, int c_off, const void* z, long long ld_z,
+                               const float* a_log, const float* dskip, float* S, void* out, long long ld_out,
+                               const int* q_start, const int* seq_ids, int B, int C, int N, void* stream) {
+    if ((long long)B * C == 0) return 0;
+    auto al = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
+    NXD_REQUIRE(rank % 8 == 0 && al(dt_w), "selective scan: step sizes of rank %d", rank);
+    const size_t smem = (size_t)STEP_ROWS * (rank + 2 * N) * sizeof(float);
+    NXD_REQUIRE(N >= 1 && smem <= 48 * 1024, "selective scan: rank %d, %d states", rank, N);
+    dim3 grid((C + 31) / 32, (B + STEP_ROWS - 1) / STEP_ROWS);
+    NXD_REQUIRE(grid.y < 65536, "selective scan: %d rows", B);
+    const bool vec = N % 4 == 0 && al(S) && al(a_log);
+    cudaStream_t st = (cudaStream_t)stream;
+#define NXD_SSTEP(T, V)                                                                                                  \
+    selective_step_kernel<T, V><<<grid, STEP_THREADS, smem, st>>>((const T*)x, ld_x, (const T*)dt_w, rank, dt_bias, p, ld_p, \
+                                                                  b_off, c_off, (const T*)z, ld_z, a_log, dskip, S, (T*)out, \
+                                                                  ld_out, q_start, seq_ids, B, C, N)
+    if (dtype == 0) { if (vec) NXD_SSTEP(bf16, true); else NXD_SSTEP(bf16, false); }
+    else { if (vec) NXD_SSTEP(float, true); else NXD_SSTEP(float, false); }
+#undef NXD_SSTEP
+    NXD_LAUNCH_CHECK();
+    return 0;
 }
 
 // xbc [B * Tn, ld] (dtype): x [H, P] at column x_off, B and C [G, N] at b_off and c_off (after the convolution); dt fp32

@@ -503,6 +503,11 @@ int nxd_selective_scan(int dtype, const void* x, long long ld_x, const float* dt
                        const float* bc, long long ld_bc, int b_off, int c_off, const void* z, long long ld_z,
                        const float* a_log, const float* dskip, float* S, void* out, long long ld_out, const int* q_start,
                        const int* n_new, const int* seq_ids, int B, int Tn, int C, int N, void* stream);
+/* one token per row; dt = p[:, :rank] dt_w^T (rank a multiple of 8), B and C further columns of p (fp32 [B, ld_p]) */
+int nxd_selective_step(int dtype, const void* x, long long ld_x, const void* dt_w, int rank, const float* dt_bias,
+                       const float* p, long long ld_p, int b_off, int c_off, const void* z, long long ld_z,
+                       const float* a_log, const float* dskip, float* S, void* out, long long ld_out, const int* q_start,
+                       const int* seq_ids, int B, int C, int N, void* stream);
 /* S <- exp(-exp(a_log_h) dt) S + dt B x^T, y = S^T C + D_h x per head, B and C shared by the H / G heads of a group;
  * S [lines, H, N, P].  dt NULL with one token per row: the products of hin [B, W] with dt_w [H, W].  impl: 0 choose, 1 token by token, 2 chunks of 64 tokens on the tensor cores (bf16) */
 int nxd_state_space_heads(int dtype, int y_dtype, const void* xbc, long long ld, int x_off, int b_off, int c_off,

@@ -1063,7 +1063,7 @@ def state_space_kernel_cases(s: dict, steps: int, warmup: int, dev) -> List[dict
     Hs, Ns, P = inner // SSM_HEAD, SSM_STATE, SSM_HEAD
     C = inner + 2 * Ns
     xbc = torch.randn(B, T, C, device=dev, dtype=bf)
-    cw, cb, cst = torch.randn(C, 4, device=dev), torch.randn(C, device=dev), torch.zeros(lines, 3, C, device=dev)
+    cw, cb, cst = torch.randn(4, C, device=dev), torch.randn(C, device=dev), torch.zeros(lines, 3, C, device=dev)
     row("short convolution + bias + silu + state", "convolution", lambda: ss.conv_silu(xbc, cw, cb, cst, zero), nbytes=4.0 * N * C)
     Gd, Hd = max(1, C // (4 * Dk) // 2), max(1, C // 2 // Dvr)            # about as many channels
     Cd = 2 * Gd * Dk + (Hd // Gd * Gd or Gd) * Dvr
@@ -1109,9 +1109,12 @@ def state_space_kernel_cases(s: dict, steps: int, warmup: int, dev) -> List[dict
     sst = torch.zeros(lines, Ci, n, device=dev)
     row("selective scan + gate, prompt", "prefill recurrence",
         lambda: ss.selective_scan(x, dts, dv[0], bc, 0, n, z, a_log, dv[1], sst, zero), nbytes=float(N * (10 * Ci + 8 * n)))
-    xd, zd, dtd, bcd = (t[:1, :1].expand(Bd, 1, t.shape[2]).contiguous() for t in (x, z, dts, bc))
-    row("selective scan + gate, one token (state read + written)", "decode recurrence",
-        lambda: ss.selective_scan(xd, dtd, dv[0], bcd, 0, n, zd, a_log, dv[1], sst, posd), nbytes=8.0 * Ci * n * Bd)
+    rank = W // 16
+    xd, zd = (t[:1, :1].expand(Bd, 1, Ci).contiguous() for t in (x, z))
+    pd, dtw = torch.randn(Bd, 1, rank + 2 * n, device=dev), torch.randn(Ci, rank, device=dev, dtype=bf) * rank ** -0.5
+    row("step sizes + selective scan + gate, one token (weights read, state read + written)", "decode recurrence",
+        lambda: ss.selective_scan(xd, None, dv[0], pd, rank, rank + n, zd, a_log, dv[1], sst, posd, dt_w=dtw),
+        nbytes=8.0 * Ci * n * Bd + 2.0 * Ci * rank)
     del x, z, dts, bc, sst
     # the stream
     x32 = torch.randn(N, W, device=dev)

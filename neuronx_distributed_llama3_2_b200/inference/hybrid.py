@@ -777,8 +777,8 @@ class MumazenInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, MumazenForCau
       * ``parallel``: rotation + cache write, capped softmax attention over the cache with the output gate in its epilogue;
         convolution, state-space heads on the line's fp32 state, gate + grouped norm; both branches write their half of one
         buffer, which one output projection reads (the branch scales sit in the gate's and the norm's fp32 epilogues);
-      * ``mamba1``: convolution, the fp32 product for step sizes, B and C, the low-rank step sizes' second half, selective scan
-        with the gate inside, output projection;
+      * ``mamba1``: convolution, the fp32 product for step sizes, B and C, the low-rank step sizes' second half (of single tokens
+        inside the recurrence's kernel), selective scan with the gate inside, output projection;
       * a looped layer appears once per pass in the run list: same modules, cache / state of the run's own index.
     A step may start at any position: attention reads earlier keys from the cache, convolutions and recurrences continue from
     the line's state."""
@@ -914,11 +914,10 @@ class MumazenInferenceModel(CacheRowsMixin, KVCacheInferenceMixin, MumazenForCau
         st = self.kv_cache.state(run)
         part = lambda n: big[..., cols[n][0]: cols[n][0] + cols[n][1]]                     # noqa: E731
         x = ss_ops.conv_silu(part("x"), mixer.conv_weight, mixer.conv_bias, st["conv"], q_start, n_new=n_new, seq_ids=seq_ids)
-        r, b, c, _ = x_proj_columns(m)
+        _, b, c, _ = x_proj_columns(m)
         p = gemm_nt(x.view(N, m.inner), mixer.x_proj, out_dtype=torch.float32)
-        dt = gemm_nt(p[:, :r].to(h.dtype).contiguous(), mixer.dt_proj, out_dtype=torch.float32)
-        y = ss_ops.selective_scan(x, dt.view(B, T, m.inner), mixer.dt_bias, p.view(B, T, -1), b, c, part("z"), mixer.a_log,
-                                  mixer.d_skip, st["S"], q_start, n_new=n_new, seq_ids=seq_ids)
+        y = ss_ops.selective_scan(x, None, mixer.dt_bias, p.view(B, T, -1), b, c, part("z"), mixer.a_log, mixer.d_skip, st["S"],
+                                  q_start, n_new=n_new, seq_ids=seq_ids, dt_w=mixer.dt_proj)
         return gemm_nt(y.view(N, m.inner), mixer.o_proj.weight)
 
     _MIX = {"parallel": _mix_parallel, "mamba1": _mix_mamba1}

@@ -334,8 +334,9 @@ def _linear_out(config: MumazenConfig, n_in: int, device) -> RowParallelLinear:
 
 class ParallelMixer(nn.Module):
     """Both branches' own tensors (their input rows are part of the layer's ``in_proj``): rows that make the step sizes, the
-    convolution over x | B | C, decays, skip, norm weight (times ``right_scale``, as the norm's fp32 epilogue applies it); and ONE
-    output projection over [gated attention heads | normed state-space heads], whose inputs carry the branch scales."""
+    convolution ``[taps, channels]`` over x | B | C, decays, skip, norm weight (times ``right_scale``, as the norm's fp32 epilogue
+    applies it); and ONE output projection over [gated attention heads | normed state-space heads], whose inputs carry the
+    branch scales."""
 
     def __init__(self, config: MumazenConfig, m: ParallelMixerConfig, device=None):
         super().__init__()
@@ -343,7 +344,7 @@ class ParallelMixer(nn.Module):
         r = m.right
         f32 = dict(dtype=torch.float32, device=device)
         self.dt_proj = nn.Parameter(torch.zeros(_up8(r.heads), config.hidden_size, dtype=config.torch_dtype, device=device))
-        self.conv_weight = nn.Parameter(torch.empty(r.channels, r.conv, **f32).normal_(0.0, 0.3))
+        self.conv_weight = nn.Parameter(torch.empty(r.conv, r.channels, **f32).normal_(0.0, 0.3))
         self.conv_bias = nn.Parameter(torch.zeros(r.channels, **f32))
         self.dt_bias = nn.Parameter(torch.zeros(r.heads, **f32))
         self.a_log = nn.Parameter(torch.zeros(r.heads, **f32))
@@ -353,8 +354,8 @@ class ParallelMixer(nn.Module):
 
 
 class SelectiveScanMixer(nn.Module):
-    """Convolution, the projection of the convolved channels to [low-rank step sizes | B | C] (fp32 products), the step sizes'
-    second half, decays ``[inner, state]``, skip, output projection."""
+    """Convolution ``[taps, channels]``, the projection of the convolved channels to [low-rank step sizes | B | C] (fp32
+    products), the step sizes' second half, decays ``[inner, state]``, skip, output projection."""
 
     def __init__(self, config: MumazenConfig, m: SelectiveScanConfig, device=None):
         super().__init__()
@@ -363,7 +364,7 @@ class SelectiveScanMixer(nn.Module):
         f32 = dict(dtype=torch.float32, device=device)
         act = dict(dtype=config.torch_dtype, device=device)
         std = config.initializer_range
-        self.conv_weight = nn.Parameter(torch.empty(m.inner, m.conv, **f32).normal_(0.0, 0.3))
+        self.conv_weight = nn.Parameter(torch.empty(m.conv, m.inner, **f32).normal_(0.0, 0.3))
         self.conv_bias = nn.Parameter(torch.zeros(m.inner, **f32))
         self.x_proj = nn.Parameter(torch.empty(n, m.inner, **act).normal_(0.0, std))
         self.dt_proj = nn.Parameter(torch.empty(m.inner, r, **act).normal_(0.0, std))
@@ -476,7 +477,7 @@ def convert_mumazen_state_dict(sd: Dict[str, torch.Tensor], config: MumazenConfi
             xp[b: b + m.state], xp[c: c + m.state] = rows[m.dt_rank: m.dt_rank + m.state], rows[m.dt_rank + m.state:]
             out[to + "x_proj"], out[to + "dt_proj"] = xp, _padded(mix("dt"), m.inner, r)
             out[to + "dt_bias"] = mix("dt.b").float()
-            out[to + "conv_weight"], out[to + "conv_bias"] = mix("conv").float(), mix("conv.b").float()
+            out[to + "conv_weight"], out[to + "conv_bias"] = mix("conv").float().t(), mix("conv.b").float()
             out[to + "a_log"], out[to + "d_skip"] = mix("A_log").float(), mix("D").float()
             out[to + "o_proj.weight"] = mix("o")
         else:
@@ -486,7 +487,7 @@ def convert_mumazen_state_dict(sd: Dict[str, torch.Tensor], config: MumazenConfi
                      "z": win[: s.inner], "xbc": win[s.inner: s.inner + s.channels]}
             out[to + "dt_proj"] = _padded(win[s.inner + s.channels:], _up8(s.heads))
             out[to + "dt_bias"] = mix("right.dt_bias").float()
-            out[to + "conv_weight"], out[to + "conv_bias"] = mix("right.conv").float(), mix("right.conv.b").float()
+            out[to + "conv_weight"], out[to + "conv_bias"] = mix("right.conv").float().t(), mix("right.conv.b").float()
             out[to + "a_log"], out[to + "d_skip"] = mix("right.A_log").float(), mix("right.D").float()
             out[to + "out_norm"] = mix("right.norm").float() * m.right_scale
             at, n = out_proj_columns(m)
@@ -558,7 +559,7 @@ def export_mumazen_state_dict(model: MumazenForCausalLM) -> Dict[str, torch.Tens
             at, _ = out_proj_columns(m)
             o = sd[frm + "o_proj.weight"]
             out[x + "left.o"], out[x + "right.o"] = o[:, : a.width], o[:, at: at + s.inner]
-        out[p + "conv"], out[p + "conv.b"] = sd[frm + "conv_weight"], sd[frm + "conv_bias"]
+        out[p + "conv"], out[p + "conv.b"] = sd[frm + "conv_weight"].t(), sd[frm + "conv_bias"]
         out[p + "A_log"], out[p + "D"] = sd[frm + "a_log"], sd[frm + "d_skip"]
         if L.mlp is None:
             continue

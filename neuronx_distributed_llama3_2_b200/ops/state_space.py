@@ -62,15 +62,16 @@ def conv_silu(x: torch.Tensor, conv_w: torch.Tensor, bias: Optional[torch.Tensor
               q_start: torch.Tensor, n_new: Optional[torch.Tensor] = None, seq_ids: Optional[torch.Tensor] = None,
               out_pitch: Optional[int] = None) -> torch.Tensor:
     """``x [B, T, C]`` (may be a column range of a projection output) -> ``silu(conv(x) + bias) [B, T, C]`` in the same dtype.
-    ``conv_w [C, taps]`` fp32, last column = the current token; ``conv_state [lines, taps - 1, C]`` fp32 is moved to the end
+    ``conv_w [taps, C]`` fp32, last row = the current token; ``conv_state [lines, taps - 1, C]`` fp32 is moved to the end
     of the step in place.  Padding rows come out as zeros.  ``out_pitch``: distance between the output's rows (>= C; the
     result is a view of a buffer that wide)."""
     B, T, C = x.shape
-    taps = conv_w.shape[1]
+    taps = conv_w.shape[0]
     K = taps - 1
     pitch = out_pitch or C
-    assert conv_w.shape[0] == C and conv_state.shape[1:] == (K, C), (x.shape, conv_w.shape, conv_state.shape)
+    assert conv_w.shape[1] == C and conv_state.shape[1:] == (K, C), (x.shape, conv_w.shape, conv_state.shape)
     if _use_kernel(x):
+        assert conv_w.is_contiguous() and conv_w.dtype == torch.float32
         x, ld = _rows(x)
         out = torch.empty(B, T, pitch, dtype=x.dtype, device=x.device)
         qs, nn_, sid = _i32(q_start), _i32(n_new), _i32(seq_ids)
@@ -94,7 +95,7 @@ def conv_silu(x: torch.Tensor, conv_w: torch.Tensor, bias: Optional[torch.Tensor
         seq = torch.cat([past, x[b, :n].float()], dim=0)   # [K + n, C]: position p0 - K + i
         acc = torch.zeros(n, C, dtype=torch.float32, device=x.device)
         for j in range(taps):
-            acc += w[:, j] * seq[j: j + n]
+            acc += w[j] * seq[j: j + n]
         if bias is not None:
             acc += bias.float()
         out[b, :n, :C] = F.silu(acc).to(x.dtype)
@@ -102,16 +103,35 @@ def conv_silu(x: torch.Tensor, conv_w: torch.Tensor, bias: Optional[torch.Tensor
     return out[..., :C]
 
 
-def selective_scan(x: torch.Tensor, dt: torch.Tensor, dt_bias: Optional[torch.Tensor], bc: torch.Tensor, b_offset: int,
+def selective_scan(x: torch.Tensor, dt: Optional[torch.Tensor], dt_bias: Optional[torch.Tensor], bc: torch.Tensor, b_offset: int,
                    c_offset: int, z: torch.Tensor, a_log: torch.Tensor, d: torch.Tensor, S: torch.Tensor,
                    q_start: torch.Tensor, n_new: Optional[torch.Tensor] = None,
-                   seq_ids: Optional[torch.Tensor] = None) -> torch.Tensor:
+                   seq_ids: Optional[torch.Tensor] = None, dt_w: Optional[torch.Tensor] = None) -> torch.Tensor:
     """``x, z [B, T, C]`` (``z`` may be a column range of a projection output), ``dt [B, T, C]`` fp32 pre-activations of the step
     sizes, ``bc [B, T, ld]`` fp32 with the ``N`` columns of B at ``b_offset`` and of C at ``c_offset``; ``a_log [C, N]``,
-    ``d [C]`` fp32; ``S [lines, C, N]`` fp32, updated in place -> ``y * silu(z) [B, T, C]`` in the dtype of ``x``."""
+    ``d [C]`` fp32; ``S [lines, C, N]`` fp32, updated in place -> ``y * silu(z) [B, T, C]`` in the dtype of ``x``.
+    ``dt_w [C, rank]`` instead of ``dt``: the pre-activations are the first ``rank`` columns of ``bc`` times its rows (fp32; of a
+    step of one token per row made inside the recurrence's kernel)."""
     B, T, C = x.shape
     N = a_log.shape[1]
-    assert a_log.shape == (C, N) and S.shape[1:] == (C, N) and dt.dtype == torch.float32 and bc.dtype == torch.float32
+    assert a_log.shape == (C, N) and S.shape[1:] == (C, N) and bc.dtype == torch.float32
+    if dt is None and T == 1 and n_new is None and _use_kernel(x) and dt_w.shape[1] % 8 == 0:
+        assert z.dtype == x.dtype == dt_w.dtype and S.is_contiguous() and a_log.is_contiguous() and dt_w.is_contiguous()
+        (x, ldx), (z, ldz), (bc, ldb) = _rows(x), _rows(z), _rows(bc)
+        out = torch.empty(B, T, C, dtype=x.dtype, device=x.device)
+        qs, sid = _i32(q_start), _i32(seq_ids)
+        L = _lib.lib(GROUP)
+        rc = L.nxd_selective_step(_c.c_int(_code(x.dtype)), _lib.ptr(x), _c.c_longlong(ldx), _lib.ptr(dt_w),
+                                  _c.c_int(dt_w.shape[1]), _lib.ptr(dt_bias), _lib.ptr(bc), _c.c_longlong(ldb),
+                                  _c.c_int(b_offset), _c.c_int(c_offset), _lib.ptr(z), _c.c_longlong(ldz), _lib.ptr(a_log),
+                                  _lib.ptr(d), _lib.ptr(S), _lib.ptr(out), _c.c_longlong(C), _lib.ptr(qs), _lib.ptr(sid),
+                                  _c.c_int(B), _c.c_int(C), _c.c_int(N), _lib.stream_ptr())
+        _lib.check(rc, "nxd_selective_step", L)
+        return out
+    if dt is None:
+        low = bc[..., : dt_w.shape[1]].reshape(B * T, -1).to(dt_w.dtype).contiguous()
+        dt = gemm_nt(low, dt_w, out_dtype=torch.float32).view(B, T, C)
+    assert dt.dtype == torch.float32
     if _use_kernel(x):
         assert z.dtype == x.dtype and S.is_contiguous() and a_log.is_contiguous()
         (x, ldx), (z, ldz), (dt, ldd), (bc, ldb) = _rows(x), _rows(z), _rows(dt), _rows(bc)

@@ -196,7 +196,7 @@ def test_short_convolution_in_portions_with_padding_on_stale_lines(dev, dt, taps
     at = 0
     for n in (2, 1, 7, 70, 20):
         left = [max(0, min(n, L - at)) for L in lens]
-        out = ss.conv_silu(x[:, at: at + n].to(dev)[..., 4: 4 + C], w.to(dev), b.to(dev), state, i32(at, at, dev=dev),
+        out = ss.conv_silu(x[:, at: at + n].to(dev)[..., 4: 4 + C], w.t().contiguous().to(dev), b.to(dev), state, i32(at, at, dev=dev),
                            n_new=i32(*left, dev=dev), seq_ids=lines, out_pitch=(C + 7) // 8 * 8).float().cpu()
         for k in range(2):
             if left[k]:
@@ -407,6 +407,29 @@ def test_step_sizes_of_single_tokens_made_inside_the_recurrence(dev, dt, W):
         outs.append((y, S))
     close(outs[1][0], outs[0][0].cpu(), torch.float32)
     close(outs[1][1], outs[0][1].cpu(), torch.float32)
+
+
+@case
+@pytest.mark.parametrize("C,N,rank,B", [(40, 16, 8, 3), (33, 5, 24, 9), (64, 40, 72, 1), (7, 1, 8, 4)])
+def test_single_tokens_of_the_selective_scan_with_low_rank_step_sizes(dev, dt, C, N, rank, B):
+    torch.manual_seed(C)
+    x, z = torch.randn(B, 1, C).to(dt), torch.randn(B, 1, C + 8).to(dt)
+    p, w = torch.randn(B, 1, rank + 2 * N + 6), (torch.randn(C, rank) * rank ** -0.5).to(dt)
+    bias, a_log, dsk = torch.randn(C) * 0.3 - 1, torch.rand(C, N) * 5 - 4, torch.randn(C)
+    S0, start = torch.randn(B + 2, C, N), torch.tensor([0 if b % 3 == 2 else 4 for b in range(B)], dtype=torch.int32)
+    lines = torch.arange(B, dtype=torch.int32).flip(0) + 1
+    S = S0.clone().to(dev)
+    y = ss.selective_scan(x.to(dev), None, bias.to(dev), p.to(dev), rank + 1, rank + N + 3, z.to(dev)[..., 8:], a_log.to(dev),
+                          dsk.to(dev), S, start.to(dev), seq_ids=lines.to(dev), dt_w=w.to(dev))
+    for b in range(B):
+        ln = int(lines[b])
+        row, xv = p[b, 0].to(F64), x[b, 0].to(F64)
+        step = O.softplus(row[:rank] @ w.to(F64).T + bias.to(F64))
+        s = S0[ln].to(F64) if int(start[b]) else torch.zeros(C, N, dtype=F64)
+        s = torch.exp(step.unsqueeze(1) * -torch.exp(a_log.to(F64))) * s + (step * xv).unsqueeze(1) * row[rank + 1: rank + 1 + N]
+        want = (s @ row[rank + N + 3: rank + 2 * N + 3] + dsk.to(F64) * xv) * O.silu(z[b, 0, 8:].to(F64))
+        close(S[ln], s, torch.float32)
+        close(y[b, 0], want, dt, scale=2.0)
 
 
 def test_scaled_rotation_tables():
