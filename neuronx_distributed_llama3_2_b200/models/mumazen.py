@@ -419,11 +419,19 @@ class MumazenDecoderLayer(nn.Module):
 
 
 class Fp32LogitsHead(ColumnParallelLinear):
-    """An output head of its own whose logits stay in fp32."""
+    """An output head of its own whose logits stay in fp32; its rows are padded to a multiple of 8 with zeros, so that every
+    vocabulary runs on the same kernels."""
+
+    def __init__(self, width: int, vocab: int, **kw):
+        super().__init__(width, _up8(vocab), **kw)
+        self.vocab = vocab
 
     def forward(self, x: torch.Tensor) -> torch.Tensor:
         w = self.weight
-        return gemm_nt(x.reshape(-1, x.shape[-1]).to(w.dtype), w, out_dtype=torch.float32).reshape(x.shape[:-1] + (w.shape[0],))
+        y = gemm_nt(x.reshape(-1, x.shape[-1]).to(w.dtype), w, out_dtype=torch.float32)
+        if w.shape[0] != self.vocab:
+            y = y[:, : self.vocab].contiguous()
+        return y.reshape(x.shape[:-1] + (self.vocab,))
 
 
 class MumazenForCausalLM(nn.Module):
@@ -460,7 +468,7 @@ def convert_mumazen_state_dict(sd: Dict[str, torch.Tensor], config: MumazenConfi
     Constants of the configuration that multiply a vector are folded into it in fp32."""
     W, res = config.hidden_size, config.residual_mult
     out: Dict[str, torch.Tensor] = {"embed_tokens.weight": sd["embed"], "norm": sd["final.norm"].float(),
-                                    "lm_head.weight": sd["head"]}
+                                    "lm_head.weight": _padded(sd["head"], _up8(config.vocab_size))}
     if config.loop is not None:
         out["loop_step"] = sd["loop.step"].float()
     for i, L in enumerate(config.layers):
@@ -530,7 +538,8 @@ def export_mumazen_state_dict(model: MumazenForCausalLM) -> Dict[str, torch.Tens
     """The inverse of ``convert_mumazen_state_dict``: this module's parameters under the checkpoint names."""
     cfg, sd = model.config, model.state_dict()
     W, res = cfg.hidden_size, cfg.residual_mult
-    out: Dict[str, torch.Tensor] = {"embed": sd["embed_tokens.weight"], "final.norm": sd["norm"], "head": sd["lm_head.weight"]}
+    out: Dict[str, torch.Tensor] = {"embed": sd["embed_tokens.weight"], "final.norm": sd["norm"],
+                                    "head": sd["lm_head.weight"][: cfg.vocab_size]}
     if cfg.loop is not None:
         out["loop.step"] = sd["loop_step"]
     for i, L in enumerate(cfg.layers):
