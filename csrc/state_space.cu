@@ -82,6 +82,7 @@ __device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
 template <typename T>
 struct ScanDecay {
     static __device__ __forceinline__ float rate(float a) { return a * LOG2E; }
+    static __device__ __forceinline__ float at(float dt, float rate) { return exp2_ftz(dt * rate); }
     static __device__ __forceinline__ uint64_t at2(uint64_t dt, uint64_t rate) {
         float lo, hi;
         unpair2(mul2(dt, rate), lo, hi);
@@ -91,6 +92,7 @@ struct ScanDecay {
 template <>
 struct ScanDecay<float> {
     static __device__ __forceinline__ float rate(float a) { return a; }
+    static __device__ __forceinline__ float at(float dt, float rate) { return decay_exp(dt * rate); }
     static __device__ __forceinline__ uint64_t at2(uint64_t dt, uint64_t rate) {
         float lo, hi;
         unpair2(mul2(dt, rate), lo, hi);
@@ -620,48 +622,100 @@ selective_step_kernel(const T* __restrict__ x, long long ld_x, const T* __restri
                       const T* __restrict__ z, long long ld_z, const float* __restrict__ a_log, const float* __restrict__ dskip,
                       float* __restrict__ S, T* __restrict__ out, long long ld_out, const int* __restrict__ q_start,
                       const int* __restrict__ seq_ids, int B, int C, int N) {
-    extern __shared__ __align__(16) float smem[];              // [STEP_ROWS][rank + 2 N]
-    const int pitch = rank + 2 * N;
+    extern __shared__ __align__(16) float smem[];              // [STEP_ROWS][rank + 2 N, padded to 4]
+    const int pitch = (rank + 2 * N + 3) & ~3;
     const int tid = threadIdx.x, r = tid & 3, c = blockIdx.x * 32 + (tid >> 2);
     const int b0 = blockIdx.y * STEP_ROWS, nb = min(STEP_ROWS, B - b0);
-    for (int idx = tid; idx < nb * pitch; idx += STEP_THREADS) {
-        const int q = idx / pitch, i = idx - q * pitch;
-        const float* row = p + (long long)(b0 + q) * ld_p;
-        smem[idx] = i < rank ? row[i] : (i < rank + N ? row[b_off + i - rank] : row[c_off + i - rank - N]);
+    const bool ok = c < C;
+    // up to 16 states (one 16-byte piece per lane): they and their decay rates are on their way before anything else
+    const bool small = VEC && N <= 16, mine = small && ok && r * 4 < N;
+    float pre[STEP_ROWS][4], rate[4];
+    if (mine) {
+        ldv<4>(a_log + (long long)c * N + r * 4, rate);
+#pragma unroll
+        for (int q = 0; q < STEP_ROWS; ++q)
+            if (q < nb) ldv<4>(S + ((long long)(seq_ids != nullptr ? seq_ids[b0 + q] : b0 + q) * C + c) * N + r * 4, pre[q]);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) rate[e] = ScanDecay<T>::rate(-expf(rate[e]));
+    }
+    const T* wr = dt_w + (long long)(ok ? c : 0) * rank;       // rank is a multiple of 8
+    constexpr int AHEAD = 4;                                   // pieces of the weights that are asked for up front
+    float w[AHEAD][8];
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j)
+        if (r * 8 + 32 * j < rank) ldv<8>(wr + r * 8 + 32 * j, w[j]);
+    if (VEC && ((ld_p | b_off | c_off) & 3) == 0 && ((uintptr_t)p & 15) == 0) {
+        const int p4 = pitch / 4, r4 = rank / 4, n4 = N / 4;
+        for (int q = tid >> 5; q < nb; q += STEP_THREADS / 32) {          // a warp per row
+            const float* row = p + (long long)(b0 + q) * ld_p;
+#pragma unroll 4
+            for (int i = tid & 31; i < p4; i += 32) {
+                const int at = i < r4 ? 4 * i : (i < r4 + n4 ? b_off + 4 * (i - r4) : c_off + 4 * (i - r4 - n4));
+                *reinterpret_cast<float4*>(smem + q * pitch + 4 * i) = *reinterpret_cast<const float4*>(row + at);
+            }
+        }
+    } else {
+        for (int idx = tid; idx < nb * pitch; idx += STEP_THREADS) {
+            const int q = idx / pitch, i = idx - q * pitch;
+            const float* row = p + (long long)(b0 + q) * ld_p;
+            smem[idx] = i < rank ? row[i] : (i < rank + N ? row[b_off + i - rank] : (i < rank + 2 * N ? row[c_off + i - rank - N] : 0.f));
+        }
     }
     __syncthreads();
-    if (c >= C) return;                                        // whole groups of four lanes
-    const unsigned mask = __activemask();
     float acc[STEP_ROWS];
 #pragma unroll
     for (int q = 0; q < STEP_ROWS; ++q) acc[q] = 0.f;
-    const T* wr = dt_w + (long long)c * rank;                  // rank is a multiple of 8
-    for (int k = r * 8; k < rank; k += 32) {
-        float w[8];
-        ldv<8>(wr + k, w);
+    auto products = [&](int k, const float* v8) {
 #pragma unroll
         for (int q = 0; q < STEP_ROWS; ++q)
             if (q < nb) {
-#pragma unroll
-                for (int i = 0; i < 8; ++i) acc[q] = fmaf(w[i], smem[q * pitch + k + i], acc[q]);
+                const float4 u = *reinterpret_cast<const float4*>(smem + q * pitch + k);
+                const float4 v = *reinterpret_cast<const float4*>(smem + q * pitch + k + 4);
+                acc[q] += fmaf(v8[0], u.x, fmaf(v8[1], u.y, fmaf(v8[2], u.z, v8[3] * u.w))) +
+                          fmaf(v8[4], v.x, fmaf(v8[5], v.y, fmaf(v8[6], v.z, v8[7] * v.w)));
             }
+    };
+#pragma unroll
+    for (int j = 0; j < AHEAD; ++j)
+        if (r * 8 + 32 * j < rank) products(r * 8 + 32 * j, w[j]);
+#pragma unroll 4
+    for (int k = r * 8 + 32 * AHEAD; k < rank; k += 32) {
+        float v8[8];
+        ldv<8>(wr + k, v8);
+        products(k, v8);
     }
-    const float bias = dt_bias != nullptr ? dt_bias[c] : 0.f, dsk = dskip[c];
+    // lane r of a channel takes row r: its sum, its step size, in the end its output
+    const float sum = transpose_sum<STEP_ROWS>(acc, r);
+    const int br = b0 + r;
+    const bool mine_row = ok && r < nb;
+    float step_r = 0.f, x_r = 0.f;
+    if (mine_row) {
+        step_r = ScanMath<T>::softplus(sum + (dt_bias != nullptr ? dt_bias[c] : 0.f));
+        x_r = ldf(x + (long long)br * ld_x + c);
+    }
+    float y[STEP_ROWS];
 #pragma unroll
     for (int q = 0; q < STEP_ROWS; ++q) {
-        if (q >= nb) break;
+        const int src = (tid & 31 & ~3) | q;
+        const float step = __shfl_sync(0xffffffffu, step_r, src), u = step * __shfl_sync(0xffffffffu, x_r, src);
+        y[q] = 0.f;
+        if (!ok || q >= nb) continue;
         const int b = b0 + q, line = seq_ids != nullptr ? seq_ids[b] : b;
         const bool fresh = q_start[b] == 0;
-        float v = acc[q];
-        v += __shfl_xor_sync(mask, v, 1);
-        v += __shfl_xor_sync(mask, v, 2);
-        const float step = softplus_f(v + bias), xv = ldf(x + (long long)b * ld_x + c), u = step * xv;
         const float* Bs = smem + q * pitch + rank;
         const float* Cs = Bs + N;
         float* Sc = S + ((long long)line * C + c) * N;
-        const float* al = a_log + (long long)c * N;
+        if (mine) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                pre[q][e] = fmaf(ScanDecay<T>::at(step, rate[e]), fresh ? 0.f : pre[q][e], u * Bs[r * 4 + e]);
+                y[q] = fmaf(pre[q][e], Cs[r * 4 + e], y[q]);
+            }
+            stv<4>(Sc + r * 4, pre[q]);
+        }
+        if (small) continue;
         constexpr int W = VEC ? 4 : 1;
-        float y = 0.f;
+        const float* al = a_log + (long long)c * N;
         for (int i = r * W; i < N; i += 4 * W) {
             float s[W], a[W];
             if (fresh) {
@@ -673,15 +727,15 @@ selective_step_kernel(const T* __restrict__ x, long long ld_x, const T* __restri
             ldv<W>(al + i, a);
 #pragma unroll
             for (int e = 0; e < W; ++e) {
-                s[e] = fmaf(decay_exp(-expf(a[e]) * step), s[e], u * Bs[i + e]);
-                y = fmaf(s[e], Cs[i + e], y);
+                s[e] = fmaf(ScanDecay<T>::at(step, ScanDecay<T>::rate(-expf(a[e]))), s[e], u * Bs[i + e]);
+                y[q] = fmaf(s[e], Cs[i + e], y[q]);
             }
             stv<W>(Sc + i, s);
         }
-        y += __shfl_xor_sync(mask, y, 1);
-        y += __shfl_xor_sync(mask, y, 2);
-        if (r == 0) stf(out + (long long)b * ld_out + c, fmaf(dsk, xv, y) * silu_f(ldf(z + (long long)b * ld_z + c)));
     }
+    const float yr = transpose_sum<STEP_ROWS>(y, r);
+    if (mine_row)
+        stf(out + (long long)br * ld_out + c, fmaf(dskip[c], x_r, yr) * ScanMath<T>::silu(ldf(z + (long long)br * ld_z + c)));
 }
 
 // ---- state-space heads: one token ------------------------------------------------------------------------------------------
@@ -1279,7 +1333,7 @@ NXD_API int nxd_selective_step(int dtype, const void* x, long long ld_x, const v
     if ((long long)B * C == 0) return 0;
     auto al = [](const void* q) { return ((uintptr_t)q % 16) == 0; };
     NXD_REQUIRE(rank % 8 == 0 && al(dt_w), "selective scan: step sizes of rank %d", rank);
-    const size_t smem = (size_t)STEP_ROWS * (rank + 2 * N) * sizeof(float);
+    const size_t smem = (size_t)STEP_ROWS * ((rank + 2 * N + 3) & ~3) * sizeof(float);
     NXD_REQUIRE(N >= 1 && smem <= 48 * 1024, "selective scan: rank %d, %d states", rank, N);
     dim3 grid((C + 31) / 32, (B + STEP_ROWS - 1) / STEP_ROWS);
     NXD_REQUIRE(grid.y < 65536, "selective scan: %d rows", B);
